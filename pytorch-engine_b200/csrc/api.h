@@ -36,7 +36,8 @@ int pe_attention_decode_noalloc(int dtype, const void* q, long long q_ld, void* 
     const void* v_pages, int split_keys, int max_splits, int* status, cudaStream_t stream);
 
 // attention_mma.cu
-int pe_attention_mma_decode_blocks_per_sm(int head_dim);
+int pe_attention_mma_decode_blocks_per_sm(int head_dim, int v_dim);
+int pe_attention_mma_dims_supported(int head_dim, int v_dim, int n_heads, int n_kv_heads);
 int pe_attention_mma_supported(int head_dim, int n_heads, int n_kv_heads);
 int pe_attention_mma(int decode, const void* q, long long q_ld, void* out, long long out_ld, int n_seqs, int max_q,
     int n_heads, int n_kv_heads, int head_dim, float scale, int window, const int* seq_qstart, const int* seq_past,
@@ -56,6 +57,13 @@ int pe_attention_mma_masked(int decode, const void* q, long long q_ld, void* out
     const void* v_pages, float* scratch, int split_keys, int max_splits, int min_range_keys, int* status,
     cudaStream_t stream);
 
+int pe_attention_mma_gated(int decode, const void* q, long long q_ld, void* out, long long out_ld, int n_seqs, int max_q,
+    int n_heads, int n_kv_heads, int head_dim, int v_dim, float scale, int window, int chunk, int keep_first, int v_heads,
+    int out_f32, int split_p, int sink, const float* out_cos, const float* out_sin, int out_rows, const void* gate,
+    long long gate_ld, const int* seq_qstart, const int* seq_past, const int* seq_slot, const int* page_table,
+    int table_stride, int num_pages, const void* k_pages, const void* v_pages, float* scratch, int split_keys,
+    int max_splits, int min_range_keys, int* status, cudaStream_t stream);
+
 // attention_latent.cu
 int pe_attention_latent_supported(int row, int rank);
 int pe_attention_latent(int decode, const void* q, long long q_ld, void* out, long long out_ld, int n_seqs, int max_q,
@@ -69,6 +77,12 @@ int pe_attention_umma_prefill(const void* q, long long q_ld, long long n_tokens,
     int n_seqs, int max_q, int n_heads, int n_kv_heads, int head_dim, float scale, int window, const int* seq_qstart,
     const int* seq_past, const int* seq_slot, const int* page_table, int table_stride, int num_pages,
     const void* k_pages, const void* v_pages, int n_sms, int* work_counter, int* status, cudaStream_t stream);
+int pe_attention_umma_dims_supported(int head_dim, int v_dim, int n_heads, int n_kv_heads);
+int pe_attention_umma_prefill_gated(const void* q, long long q_ld, long long n_tokens, void* out, long long out_ld,
+    int n_seqs, int max_q, int n_heads, int n_kv_heads, int head_dim, int v_dim, float scale, int window, int sink,
+    const float* out_cos, const float* out_sin, int out_rows, const void* gate, long long gate_ld, const int* seq_qstart,
+    const int* seq_past, const int* seq_slot, const int* page_table, int table_stride, int num_pages, const void* k_pages,
+    const void* v_pages, int n_sms, int* work_counter, int* status, cudaStream_t stream);
 int pe_attention_umma_prefill_ex(const void* q, long long q_ld, long long n_tokens, void* out, long long out_ld,
     int n_seqs, int max_q, int n_heads, int n_kv_heads, int head_dim, float scale, int window, int sink,
     const float* out_cos, const float* out_sin, int out_rows, const int* seq_qstart, const int* seq_past,
@@ -107,6 +121,9 @@ int pe_embed_gather_scaled(int dtype, const void* table, const int* ids, float* 
 
 // gemm_smallm.cu
 int pe_gemm_smallm_supported(int M, int N, int K);
+int pe_gemm_smallm_glu(const void* x, long long ldx, const void* w, void* y, long long ldy, int M, int N, int K,
+    int out_f32, int pair_offset, int kind, float limit, float alpha, const float* bias, int n_sms,
+    cudaStream_t stream);
 int pe_gemm_smallm(const void* x, long long ldx, const void* w, void* y, long long ldy, int M, int N, int K,
     int out_f32, int pair_offset, int n_sms, cudaStream_t stream);
 int pe_gemm_smallm_grouped(const void* x, long long ldx, long long x_group_stride, int groups, int group_rows,
@@ -114,11 +131,17 @@ int pe_gemm_smallm_grouped(const void* x, long long ldx, long long x_group_strid
 
 // gemm_umma.cu
 int pe_gemm_umma_supported(int M, int N, int K, int pair_offset);
+int pe_gemm_umma_glu(const void* x, long long ldx, const void* w, void* y, long long ldy, int M, int N, int K,
+    int out_f32, int pair_offset, int kind, float limit, float alpha, const float* bias, int n_sms, int* status,
+    cudaStream_t stream);
 int pe_gemm_umma(const void* x, long long ldx, const void* w, void* y, long long ldy, int M, int N, int K,
     int out_f32, int pair_offset, int n_sms, int* status, cudaStream_t stream);
 
 // gemm_umma2.cu
 int pe_gemm_umma2_supported(int M, int N, int K, int pair_offset);
+int pe_gemm_umma2_glu(const void* x, long long ldx, const void* w, void* y, long long ldy, int M, int N, int K,
+    int out_f32, int pair_offset, int kind, float limit, float alpha, const float* bias, int n_sms, int* status,
+    cudaStream_t stream);
 int pe_gemm_umma2(const void* x, long long ldx, const void* w, void* y, long long ldy, int M, int N, int K,
     int out_f32, int pair_offset, int n_sms, int* status, cudaStream_t stream);
 int pe_gemm_umma2_qkv_rope_supported(int M, int K, int n_heads, int n_kv_heads, int head_dim, int rotary_dim);
@@ -149,7 +172,14 @@ int pe_qkv_rotate_append(int dtype, void* qkv, long long ld, int n_tokens, int n
     int rotary_dim, int table_rows, int interleaved, int v_unit_norm, const float* v_cos, const float* v_sin,
     int v_rotary_dim, int v_table_rows, int v_interleaved, const int* token_seq, const int* token_pos,
     const int* seq_slot, const int* seq_qstart, const int* page_table, int table_stride, int num_pages, void* k_pages,
-    void* v_pages, int write_cache, const float* bias, int* status, cudaStream_t stream);
+    void* v_pages, int write_cache, const float* bias, int qk_unit, const void* v_mix, float v_lambda, void* v_keep,
+    int* status, cudaStream_t stream);
+
+// streams.cu
+int pe_stream_mix(int dtype, const float* single, float* x, const void* y, const float* bias, const float* mix,
+    const float* write, const float* read, int norm, const float* w, float eps, void* out, const int* rows, int n_rows,
+    int streams, int width, cudaStream_t stream);
+int pe_layernorm(int dtype, const void* x, const float* w, void* out, int n_rows, int width, float eps, cudaStream_t stream);
 
 // sampling.cu
 long long pe_sample_scratch_bytes(int n_rows, int vocab, float temperature, int top_k, float top_p, float min_p);
@@ -219,7 +249,7 @@ int pe_moe_gather_rows(int dtype, const void* x, const int* row_token, const int
 int pe_moe_combine(int dtype, const void* rows, const void* x, const void* shared, const int* pair_row,
     const float* weight, int top, void* out, int n_tokens, int width, cudaStream_t stream);
 int pe_glu_act(int dtype, const void* gate_up, void* out, int n_rows, int inter, int kind, float limit, float alpha,
-    cudaStream_t stream);
+    const float* bias, cudaStream_t stream);
 
 // ssd.cu
 int pe_ssd_recurrence(int dtype, const void* xbc, long long xbc_ld, const void* dt, long long dt_ld, const float* dt_bias,

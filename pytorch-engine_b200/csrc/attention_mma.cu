@@ -1,5 +1,7 @@
 // Causal grouped-query attention over the paged bfloat16 cache on the tensor cores (mma.sync
-// m16n8k16, float32 accumulation), for head sizes 64 and 128 and groups of up to 16 query heads.
+// m16n8k16, float32 accumulation), for groups of up to 16 query heads and head sizes 64 and 128 (values of the
+// same size), or any key size up to 256 and value size up to 128 that are multiples of 8: those run in tiles of the next
+// larger size whose spare columns are zeros (queries: written so; keys and values: TMA fills what lies beyond a row).
 // Other shapes and the float32 mode use attention_generic.cu.
 //
 // Formulas as in attention_generic.cu (pygguf_engine/kv_cache.py:833, 2189-2192 masks; 756 head
@@ -57,7 +59,15 @@ struct Args {
   int split_p;
   // keep_first > 0 (with a window): keys at positions < keep_first stay visible to every later query
   int keep_first;
+  // sizes of a key and of a value row; the kernels' tiles are as large or larger
+  int hd, vd;
+  // each head's output times sigmoid(gate[token, head]) (rows of the step's tokens, gate_ld apart); null: no gate
+  const __nv_bfloat16* gate; long long gate_ld;
 };
+
+__device__ __forceinline__ float gate_of(const Args& a, int token, int head) {
+  return 1.f / (1.f + expf(-__bfloat162float(a.gate[(size_t)token * a.gate_ld + head])));
+}
 
 // What rounding (p0, p1) to bfloat16 left over, as a bfloat16 pair.
 __device__ __forceinline__ uint32_t pack_bf16_rest(float p0, float p1) {
@@ -109,7 +119,7 @@ template <int HD, int ROWS = BN> __device__ __forceinline__ uint32_t tile_off(in
 
 // One elected thread starts the copy of one page (64 keys of kv head `kvh`) of K and V into a stage;
 // `bar` counts the bytes.
-template <int HD>
+template <int HD, int VD>
 __device__ __forceinline__ void issue_page(const Args& a, const CUtensorMap* kmap, const CUtensorMap* vmap, int slot,
                                            int kvh, int k0, char* stage, uint64_t* bar) {
   const int logical = k0 / BN;
@@ -121,11 +131,11 @@ __device__ __forceinline__ void issue_page(const Args& a, const CUtensorMap* kma
   }
   const int y = (page * a.n_kv_heads + kvh) * BN;
   const int yv = (page * a.v_heads + kvh % a.v_heads) * BN;
-  tma::mbar_expect_tx(bar, 2 * BN * HD * 2);
+  tma::mbar_expect_tx(bar, BN * (HD + VD) * 2);
 #pragma unroll
-  for (int sub = 0; sub < HD / 64; ++sub) {
-    tma::load_2d(stage + sub * (BN * 128), kmap, sub * 64, y, bar);
-    tma::load_2d(stage + BN * HD * 2 + sub * (BN * 128), vmap, sub * 64, yv, bar);
+  for (int sub = 0; sub < (HD > VD ? HD : VD) / 64; ++sub) {
+    if (sub < HD / 64) tma::load_2d(stage + sub * (BN * 128), kmap, sub * 64, y, bar);
+    if (sub < VD / 64) tma::load_2d(stage + BN * HD * 2 + sub * (BN * 128), vmap, sub * 64, yv, bar);
   }
 }
 
@@ -143,18 +153,21 @@ __device__ __forceinline__ char* align_1024(char* p) {
 
 // ---- prefill ---------------------------------------------------------------------------------------
 // grid: (row tiles of 64, n_kv_heads, n_seqs); block: 128 threads.
-template <int HD, bool SPLIT_P>
-__global__ void __launch_bounds__(128, SPLIT_P ? 2 : 3) prefill_kernel(Args a, const __grid_constant__ CUtensorMap kmap,
+// PAD: rows are a.hd and a.vd features, fewer than the tiles' HD and VD.
+template <int HD, int VD, bool SPLIT_P, bool PAD>
+__global__ void __launch_bounds__(128, (SPLIT_P || HD > 128) ? 2 : 3) prefill_kernel(Args a, const __grid_constant__ CUtensorMap kmap,
                                                       const __grid_constant__ CUtensorMap vmap) {
   extern __shared__ char smem_raw[];
   __shared__ uint64_t bars[2];
   pdl_wait_block();
   pdl_launch_dependents();
   char* smem = align_1024(smem_raw);
-  constexpr int STAGE = 2 * BN * HD * 2;      // K and V tile
+  constexpr int STAGE = BN * (HD + VD) * 2;   // K and V tile
   constexpr int KS = HD / 16;                 // k-steps of Q.K^T
-  constexpr int NO = HD / 8;                  // n-tiles of the output
-  // Q is staged in the second K/V stage: its fragments are in registers before that stage is first filled
+  constexpr int NO = VD / 8;                  // n-tiles of the output
+  const int hd = PAD ? a.hd : HD, vd = PAD ? a.vd : VD;
+  // Q is staged in the second K/V stage: its fragments are in registers before that stage is first filled (64 rows of
+  // HD features fit there: the stage holds that many of K alone)
   char* q_s = smem + STAGE;                   // [64][HD] swizzled
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t = lane & 3;
@@ -180,16 +193,16 @@ __global__ void __launch_bounds__(128, SPLIT_P ? 2 : 3) prefill_kernel(Args a, c
     tma::mbar_init(&bars[0], 1);
     tma::mbar_init(&bars[1], 1);
     tma::fence_barrier_init();
-    issue_page<HD>(a, &kmap, &vmap, slot, kvh, tile_k0(0), smem, &bars[0]);
+    issue_page<HD, VD>(a, &kmap, &vmap, slot, kvh, tile_k0(0), smem, &bars[0]);
   }
   constexpr int CPR = HD / 8;
   for (int i = tid; i < 64 * CPR; i += 128) {
     const int r = i / CPR, chunk = i % CPR;
     const int row = row0 + r;
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (row < n_rows) {
+    if (row < n_rows && (!PAD || chunk * 8 < hd)) {
       const int tok = row / group, head = kvh * group + row % group;
-      v = *reinterpret_cast<const uint4*>(a.q + (size_t)(q0 + tok) * a.q_ld + (size_t)head * HD + chunk * 8);
+      v = *reinterpret_cast<const uint4*>(a.q + (size_t)(q0 + tok) * a.q_ld + (size_t)head * hd + chunk * 8);
     }
     *reinterpret_cast<uint4*>(q_s + tile_off<HD>(r, chunk)) = v;
   }
@@ -218,7 +231,7 @@ __global__ void __launch_bounds__(128, SPLIT_P ? 2 : 3) prefill_kernel(Args a, c
     char* stage = smem + (it & 1) * STAGE;
     // next page into the other stage (everyone left it at the end of the last round)
     if (tid == 0 && it + 1 < n_tiles)
-      issue_page<HD>(a, &kmap, &vmap, slot, kvh, tile_k0(it + 1), smem + ((it + 1) & 1) * STAGE, &bars[(it + 1) & 1]);
+      issue_page<HD, VD>(a, &kmap, &vmap, slot, kvh, tile_k0(it + 1), smem + ((it + 1) & 1) * STAGE, &bars[(it + 1) & 1]);
     if (!tma::mbar_wait(&bars[it & 1], (it >> 1) & 1)) {
       give_up(a, bars, 2, 1);
       return;
@@ -310,7 +323,7 @@ __global__ void __launch_bounds__(128, SPLIT_P ? 2 : 3) prefill_kernel(Args a, c
         for (int np = 0; np < NO / 2; ++np) {  // pairs of 8-feature n-tiles
           uint32_t vb[4];
           const int key = kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
-          ldmatrix_x4_trans(vb, vs_base + tile_off<HD>(key, np * 2 + (lane >> 4)));
+          ldmatrix_x4_trans(vb, vs_base + tile_off<VD>(key, np * 2 + (lane >> 4)));
           mma_bf16(o[np * 2], pf[kk], vb[0], vb[1]);
           mma_bf16(o[np * 2 + 1], pf[kk], vb[2], vb[3]);
           if (SPLIT_P) {
@@ -332,8 +345,9 @@ __global__ void __launch_bounds__(128, SPLIT_P ? 2 : 3) prefill_kernel(Args a, c
     const int row = half ? r_hi : r_lo;
     if (row >= n_rows) continue;
     const int tok = row / group, head = kvh * group + row % group;
-    __nv_bfloat16* dst = a.out + (size_t)(q0 + tok) * a.out_ld + (size_t)head * HD;
-    const float inv = half ? inv_hi : inv_lo;
+    __nv_bfloat16* dst = a.out + (size_t)(q0 + tok) * a.out_ld + (size_t)head * vd;
+    float inv = half ? inv_hi : inv_lo;
+    if (a.gate) inv *= gate_of(a, q0 + tok, head);
     if (a.out_cos) {
       // a thread's two adjacent features are one interleaved pair: pair n*4 + t turns back by the position's angle
       const int pos = half ? pos_hi : pos_lo;
@@ -341,8 +355,8 @@ __global__ void __launch_bounds__(128, SPLIT_P ? 2 : 3) prefill_kernel(Args a, c
         report(a.status, kStatusPositionOutOfRange, q0 + tok, pos, a.out_rows);
         continue;
       }
-      const float* cs = a.out_cos + (size_t)pos * (HD / 2);
-      const float* sn = a.out_sin + (size_t)pos * (HD / 2);
+      const float* cs = a.out_cos + (size_t)pos * (VD / 2);
+      const float* sn = a.out_sin + (size_t)pos * (VD / 2);
 #pragma unroll
       for (int n = 0; n < NO; ++n) {
         const float c = cs[n * 4 + t], sv = sn[n * 4 + t];
@@ -352,16 +366,16 @@ __global__ void __launch_bounds__(128, SPLIT_P ? 2 : 3) prefill_kernel(Args a, c
       continue;
     }
     if (a.out_f32) {
-      float* dstf = reinterpret_cast<float*>(a.out) + (size_t)(q0 + tok) * a.out_ld + (size_t)head * HD;
+      float* dstf = reinterpret_cast<float*>(a.out) + (size_t)(q0 + tok) * a.out_ld + (size_t)head * vd;
 #pragma unroll
       for (int n = 0; n < NO; ++n)
-        *reinterpret_cast<float2*>(dstf + n * 8 + 2 * t) = make_float2(o[n][half * 2] * inv, o[n][half * 2 + 1] * inv);
+        if (!PAD || n * 8 < vd) *reinterpret_cast<float2*>(dstf + n * 8 + 2 * t) = make_float2(o[n][half * 2] * inv, o[n][half * 2 + 1] * inv);
       continue;
     }
 #pragma unroll
     for (int n = 0; n < NO; ++n) {
       const uint32_t v = pack_bf16(o[n][half * 2] * inv, o[n][half * 2 + 1] * inv);
-      *reinterpret_cast<uint32_t*>(dst + n * 8 + 2 * t) = v;
+      if (!PAD || n * 8 < vd) *reinterpret_cast<uint32_t*>(dst + n * 8 + 2 * t) = v;
     }
   }
 }
@@ -369,14 +383,14 @@ __global__ void __launch_bounds__(128, SPLIT_P ? 2 : 3) prefill_kernel(Args a, c
 // One warp folds its 16 keys (key0 .. key0+15 of the page that starts at position k0) into the
 // running softmax state of the group's rows.  Keys outside [k_first, k_hi) and keys inside [hole_lo, hole_hi) (what lies
 // between the kept first keys and the window) are masked.
-template <int HD, bool SPLIT_P>
+template <int HD, int VD, bool SPLIT_P>
 __device__ __forceinline__ void decode_fold_page(uint32_t ks_base, uint32_t vs_base, int key0, int k0, int k_first,
                                                  int k_hi, int hole_lo, int hole_hi, float scale_log2,
                                                  const uint32_t (&qf)[HD / 16][4],
-                                                 float (&o)[HD / 8][4], float& m_lo, float& m_hi, float& l_lo,
+                                                 float (&o)[VD / 8][4], float& m_lo, float& m_hi, float& l_lo,
                                                  float& l_hi, int lane) {
   constexpr int KS = HD / 16;
-  constexpr int NO = HD / 8;
+  constexpr int NO = VD / 8;
   const int t = lane & 3;
     if (k0 + key0 < k_hi && k0 + key0 + 15 >= k_first && !(k0 + key0 >= hole_lo && k0 + key0 + 15 < hole_hi)) {
   float s[2][4];
@@ -437,7 +451,7 @@ __device__ __forceinline__ void decode_fold_page(uint32_t ks_base, uint32_t vs_b
   for (int np = 0; np < NO / 2; ++np) {
     uint32_t vb[4];
     const int key = key0 + (lane & 7) + ((lane >> 3) & 1) * 8;
-    ldmatrix_x4_trans(vb, vs_base + tile_off<HD>(key, np * 2 + (lane >> 4)));
+    ldmatrix_x4_trans(vb, vs_base + tile_off<VD>(key, np * 2 + (lane >> 4)));
     mma_bf16(o[np * 2], pf, vb[0], vb[1]);
     mma_bf16(o[np * 2 + 1], pf, vb[2], vb[3]);
     if (SPLIT_P) {
@@ -461,7 +475,7 @@ __device__ __forceinline__ int range_keys(const Args& a, int len) {
 }
 
 // grid: (max_splits, n_kv_heads, n_seqs); block: 128 threads; STAGES pages in flight.
-template <int HD, int STAGES, bool SPLIT_P>
+template <int HD, int VD, int STAGES, bool SPLIT_P, bool PAD>
 __global__ void __launch_bounds__(128) decode_split_kernel(Args a, const __grid_constant__ CUtensorMap kmap,
                                                            const __grid_constant__ CUtensorMap vmap) {
   extern __shared__ char smem_raw[];
@@ -470,9 +484,10 @@ __global__ void __launch_bounds__(128) decode_split_kernel(Args a, const __grid_
   // precedes this one started, so they may be read before the dependency wait; the last page (it gets
   // this step's key) and the queries come from that kernel and are read after it.
   char* smem = align_1024(smem_raw);
-  constexpr int STAGE = 2 * BN * HD * 2;
+  constexpr int STAGE = BN * (HD + VD) * 2;
   constexpr int KS = HD / 16;
-  constexpr int NO = HD / 8;
+  constexpr int NO = VD / 8;
+  const int hd = PAD ? a.hd : HD, vd = PAD ? a.vd : VD;
   char* q_s = smem + STAGES * STAGE;  // [16][HD] swizzled
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t = lane & 3;
@@ -505,20 +520,21 @@ __global__ void __launch_bounds__(128) decode_split_kernel(Args a, const __grid_
 #pragma unroll
     for (int s = 0; s < STAGES - 1; ++s)
       if (s < n_tiles && tile_k0(s) != last_page_k0)
-        issue_page<HD>(a, &kmap, &vmap, slot, kvh, tile_k0(s), smem + s * STAGE, &bars[s]);
+        issue_page<HD, VD>(a, &kmap, &vmap, slot, kvh, tile_k0(s), smem + s * STAGE, &bars[s]);
   }
   pdl_wait_block();
   if (tid == 0) {
 #pragma unroll
     for (int s = 0; s < STAGES - 1; ++s)
       if (s < n_tiles && tile_k0(s) == last_page_k0)
-        issue_page<HD>(a, &kmap, &vmap, slot, kvh, tile_k0(s), smem + s * STAGE, &bars[s]);
+        issue_page<HD, VD>(a, &kmap, &vmap, slot, kvh, tile_k0(s), smem + s * STAGE, &bars[s]);
   }
   constexpr int CPR = HD / 8;
   for (int i = tid; i < 16 * CPR; i += 128) {
     const int r = i / CPR, chunk = i % CPR;
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (r < group) v = *reinterpret_cast<const uint4*>(a.q + (size_t)tq * a.q_ld + (size_t)(kvh * group + r) * HD + chunk * 8);
+    if (r < group && (!PAD || chunk * 8 < hd))
+      v = *reinterpret_cast<const uint4*>(a.q + (size_t)tq * a.q_ld + (size_t)(kvh * group + r) * hd + chunk * 8);
     *reinterpret_cast<uint4*>(q_s + tile_off<HD, 16>(r, chunk)) = v;
   }
   __syncthreads();
@@ -537,34 +553,34 @@ __global__ void __launch_bounds__(128) decode_split_kernel(Args a, const __grid_
     // keep STAGES-1 pages in flight (the stage refilled here was released by the last round's barrier)
     const int nxt = it + STAGES - 1;
     if (tid == 0 && nxt < n_tiles)
-      issue_page<HD>(a, &kmap, &vmap, slot, kvh, tile_k0(nxt), smem + (nxt % STAGES) * STAGE, &bars[nxt % STAGES]);
+      issue_page<HD, VD>(a, &kmap, &vmap, slot, kvh, tile_k0(nxt), smem + (nxt % STAGES) * STAGE, &bars[nxt % STAGES]);
     if (!tma::mbar_wait(&bars[it % STAGES], (it / STAGES) & 1)) {
       give_up(a, bars, STAGES, 2);
       return;
     }
     const int k0 = tile_k0(it);
-    decode_fold_page<HD, SPLIT_P>(smem_u32(smem + (it % STAGES) * STAGE), smem_u32(smem + (it % STAGES) * STAGE) + BN * HD * 2,
+    decode_fold_page<HD, VD, SPLIT_P>(smem_u32(smem + (it % STAGES) * STAGE), smem_u32(smem + (it % STAGES) * STAGE) + BN * HD * 2,
                          warp * 16, k0, k_first, k_hi, hole_lo, hole_hi, a.scale_log2, qf, o, m_lo, m_hi, l_lo, l_hi, lane);
     __syncthreads();
   }
   pdl_launch_dependents();
   // merge the four warps (fixed order) through shared memory laid over the stages
   float* ml = reinterpret_cast<float*>(smem);            // [4 warps][16 rows][2]
-  float* acc = ml + 4 * 16 * 2;                          // [4 warps][16 rows][HD]
+  float* acc = ml + 4 * 16 * 2;                          // [4 warps][16 rows][VD]
   if (t == 0) {
     ml[(warp * 16 + g) * 2] = m_lo;     ml[(warp * 16 + g) * 2 + 1] = l_lo;
     ml[(warp * 16 + g + 8) * 2] = m_hi; ml[(warp * 16 + g + 8) * 2 + 1] = l_hi;
   }
 #pragma unroll
   for (int n = 0; n < NO; ++n) {
-    float* r0 = acc + (size_t)(warp * 16 + g) * HD + n * 8 + 2 * t;
-    float* r1 = acc + (size_t)(warp * 16 + g + 8) * HD + n * 8 + 2 * t;
+    float* r0 = acc + (size_t)(warp * 16 + g) * VD + n * 8 + 2 * t;
+    float* r1 = acc + (size_t)(warp * 16 + g + 8) * VD + n * 8 + 2 * t;
     r0[0] = o[n][0]; r0[1] = o[n][1];
     r1[0] = o[n][2]; r1[1] = o[n][3];
   }
   __syncthreads();
-  for (int i = tid; i < group * HD; i += 128) {
-    const int r = i / HD, c = i - r * HD;
+  for (int i = tid; i < group * vd; i += 128) {
+    const int r = i / vd, c = i - r * vd;
     float mm = -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; ++w) mm = fmaxf(mm, ml[(w * 16 + r) * 2]);
@@ -575,22 +591,22 @@ __global__ void __launch_bounds__(128) decode_split_kernel(Args a, const __grid_
         const float mw = ml[(w * 16 + r) * 2];
         const float f = (mw == -INFINITY) ? 0.f : fast_exp2(mw - mm);
         ll += ml[(w * 16 + r) * 2 + 1] * f;
-        aa += acc[(size_t)(w * 16 + r) * HD + c] * f;
+        aa += acc[(size_t)(w * 16 + r) * VD + c] * f;
       }
     }
     const size_t pidx = ((size_t)b * a.n_heads + (kvh * group + r)) * a.max_splits + split;
-    a.part_acc[pidx * HD + c] = (ll > 0.f) ? aa / ll : 0.f;
+    a.part_acc[pidx * vd + c] = (ll > 0.f) ? aa / ll : 0.f;
     // log-sum-exp in natural units, as the merge kernel expects: (m + log2 l) * ln 2
     if (c == 0) a.part_lse[pidx] = (ll > 0.f) ? (mm + log2f(ll)) * 0.6931471805599453f : -INFINITY;
   }
 }
 
 // grid: (n_heads, n_seqs): merge the ranges of one (sequence, head) (pygguf_engine/kv_cache.py:273-282).
-template <int HD>
 __global__ void decode_merge_kernel(Args a) {
   pdl_wait_block();
   pdl_launch_dependents();
   const int b = blockIdx.y, h = blockIdx.x;
+  const int vd = a.vd;
   const int tq = a.seq_qstart[b];
   const int len = a.seq_past[b] + 1;
   const int per_range = range_keys(a, len);
@@ -607,12 +623,13 @@ __global__ void decode_merge_kernel(Args a) {
   const int keep = a.keep_first > 0 ? min(a.keep_first, win_lo) : 0;
   const int kept_ranges = min((keep + per_range - 1) / per_range, first);
   const size_t base = ((size_t)b * a.n_heads + h) * a.max_splits;
-  __nv_bfloat16* o = a.out + (size_t)tq * a.out_ld + (size_t)h * HD;
+  __nv_bfloat16* o = a.out + (size_t)tq * a.out_ld + (size_t)h * vd;
+  const float gate = a.gate ? gate_of(a, tq, h) : 1.f;
   // Ranges are taken eight at a time: all their loads are issued before the first is used (this kernel
   // is short and a decode step waits for it once per layer), then they are folded into a running
   // maximum, denominator and sum, in range order.
   constexpr int G = 8;
-  for (int c = threadIdx.x; c < HD; c += blockDim.x) {
+  for (int c = threadIdx.x; c < vd; c += blockDim.x) {
     // with a sink the fold starts from one more range whose log-sum is 0 and whose output is 0
     float mx = a.sink ? 0.f : -INFINITY, denom = a.sink ? 1.f : 0.f, v = 0.f;
     for (int lot = kept_ranges > 0 ? 0 : 1; lot < 2; ++lot)
@@ -622,7 +639,7 @@ __global__ void decode_merge_kernel(Args a) {
       for (int i = 0; i < G; ++i) {
         const bool live = s0 + i < s_end;
         e[i] = live ? a.part_lse[base + s0 + i] : -INFINITY;
-        acc[i] = live ? a.part_acc[(base + s0 + i) * HD + c] : 0.f;
+        acc[i] = live ? a.part_acc[(base + s0 + i) * vd + c] : 0.f;
       }
       float m_new = mx;
 #pragma unroll
@@ -639,19 +656,20 @@ __global__ void decode_merge_kernel(Args a) {
       }
       mx = m_new;
     }
-    v = v / fmaxf(denom, 1e-20f);
+    v = v / fmaxf(denom, 1e-20f) * gate;
     if (a.out_cos) {
-      // features c and c ^ 1 (adjacent lanes) are one interleaved pair; every lane of the warp is here (HD % 32 == 0)
+      // features c and c ^ 1 (adjacent lanes) are one interleaved pair; every lane of the warp is here (turned outputs: 64 or 128
+      // features)
       const float other = __shfl_xor_sync(0xffffffffu, v, 1);
       const int pos = len - 1;
       if (pos < 0 || pos >= a.out_rows) {
         if (c == 0) report(a.status, kStatusPositionOutOfRange, tq, pos, a.out_rows);
         continue;
       }
-      const float cs = a.out_cos[(size_t)pos * (HD / 2) + (c >> 1)], sn = a.out_sin[(size_t)pos * (HD / 2) + (c >> 1)];
+      const float cs = a.out_cos[(size_t)pos * (vd / 2) + (c >> 1)], sn = a.out_sin[(size_t)pos * (vd / 2) + (c >> 1)];
       v = (c & 1) ? v * cs - other * sn : v * cs + other * sn;
     }
-    if (a.out_f32) reinterpret_cast<float*>(a.out)[(size_t)tq * a.out_ld + (size_t)h * HD + c] = v;
+    if (a.out_f32) reinterpret_cast<float*>(a.out)[(size_t)tq * a.out_ld + (size_t)h * vd + c] = v;
     else o[c] = __float2bfloat16_rn(v);
   }
 }
@@ -666,17 +684,17 @@ static int opt_in(K kernel, size_t bytes) {
   return 0;
 }
 
-template <int HD, bool SPLIT_P>
+template <int HD, int VD, bool SPLIT_P, bool PAD>
 static int launch(const Args& a, bool decode, int n_seqs, int max_q, cudaStream_t stream) {
-  constexpr int STAGE = 2 * BN * HD * 2;
+  constexpr int STAGE = BN * (HD + VD) * 2;
   CUtensorMap kmap, vmap;
   const uint64_t rows = (uint64_t)a.num_pages * a.n_kv_heads * BN;
-  int me = tma::make_map_2d_bf16(&kmap, a.k_pages, HD, rows, HD, 64, BN);
-  if (me == 0) me = tma::make_map_2d_bf16(&vmap, a.v_pages, HD, (uint64_t)a.num_pages * a.v_heads * BN, HD, 64, BN);
+  int me = tma::make_map_2d_bf16(&kmap, a.k_pages, a.hd, rows, a.hd, 64, BN);
+  if (me == 0) me = tma::make_map_2d_bf16(&vmap, a.v_pages, a.vd, (uint64_t)a.num_pages * a.v_heads * BN, a.vd, 64, BN);
   if (me != 0) return me < 0 ? me : PE_ERR_BAD_ARGUMENT;
   if (!decode) {
     const size_t smem = 1024 + 2 * STAGE;
-    auto k = prefill_kernel<HD, SPLIT_P>;
+    auto k = prefill_kernel<HD, VD, SPLIT_P, PAD>;
     int e = opt_in(k, smem);
     if (e) return e;
     const long long tiles = ((long long)max_q * a.group + 63) / 64;
@@ -690,7 +708,7 @@ static int launch(const Args& a, bool decode, int n_seqs, int max_q, cudaStream_
   if (grid.y > 65535 || grid.z > 65535) return PE_ERR_UNSUPPORTED_SIZE;
   auto go = [&](auto kern, int STAGES) -> int {
     size_t smem = STAGES * STAGE + 16 * HD * 2;
-    const size_t merge = (4 * 16 * 2 + 4 * 16 * HD) * sizeof(float);
+    const size_t merge = (4 * 16 * 2 + 4 * 16 * VD) * sizeof(float);
     if (merge > smem) smem = merge;
     smem += 1024;
     int e = opt_in(kern, smem);
@@ -699,7 +717,7 @@ static int launch(const Args& a, bool decode, int n_seqs, int max_q, cudaStream_
     return 0;
   };
   // three stages: two blocks per SM, two pages in flight per block (measured best of 2, 3, 4)
-  const int e = go(decode_split_kernel<HD, 3, SPLIT_P>, 3);
+  const int e = go(decode_split_kernel<HD, VD, 3, SPLIT_P, PAD>, 3);
   if (e) return e;
   PE_LAUNCH_CHECK();
   // The merge starts when the split kernel has completed, not while it drains: with the early start a
@@ -708,7 +726,7 @@ static int launch(const Args& a, bool decode, int n_seqs, int max_q, cudaStream_
   // 1 to 64.  Why its waiting blocks cost that much is not known; switching the early start off for any
   // other kernel of the step gained nothing or lost.
   dim3 mgrid(a.n_heads, n_seqs);
-  pe::launch_after(decode_merge_kernel<HD>, mgrid, HD >= 128 ? 128 : 64, 0, stream, a);
+  pe::launch_after(decode_merge_kernel, mgrid, a.vd > 64 ? 128 : 64, 0, stream, a);
   PE_LAUNCH_CHECK();
   return PE_OK;
 }
@@ -716,11 +734,15 @@ static int launch(const Args& a, bool decode, int n_seqs, int max_q, cudaStream_
 }  // namespace fa
 }  // namespace pe
 
+// The tile sizes that rows of these sizes run in.
+static int tile_of(int dim) { return (dim + 63) / 64 * 64; }
+
 // Decode blocks that one SM holds at a time (shared memory bound): the caller sizes the number of
 // ranges per sequence so that one wave of blocks covers the batch.
-extern "C" int pe_attention_mma_decode_blocks_per_sm(int head_dim) {
-  const size_t stage = 2 * (size_t)pe::fa::BN * head_dim * 2;
-  const size_t smem = 3 * stage + 16 * (size_t)head_dim * 2 + 1024 + 1024;   // + the block's static and reserved part
+extern "C" int pe_attention_mma_decode_blocks_per_sm(int head_dim, int v_dim) {
+  const size_t hd = tile_of(head_dim), vd = tile_of(v_dim);
+  const size_t stage = (size_t)pe::fa::BN * (hd + vd) * 2;
+  const size_t smem = 3 * stage + 16 * hd * 2 + 1024 + 1024;   // + the block's static and reserved part
   const int n = (int)((227 * 1024) / smem);
   return n < 1 ? 1 : n;
 }
@@ -731,6 +753,13 @@ extern "C" int pe_attention_mma_supported(int head_dim, int n_heads, int n_kv_he
   if (n_kv_heads <= 0 || n_heads % n_kv_heads) return 0;
   if (n_heads / n_kv_heads > 16) return 0;
   return 1;
+}
+
+// The same for keys and values of sizes of their own, which run in padded tiles unless they are both 64 or both 128.
+extern "C" int pe_attention_mma_dims_supported(int head_dim, int v_dim, int n_heads, int n_kv_heads) {
+  if (head_dim < 8 || head_dim > 256 || head_dim % 8 || v_dim < 8 || v_dim > 128 || v_dim % 8) return 0;
+  if (n_kv_heads <= 0 || n_heads % n_kv_heads) return 0;
+  return n_heads / n_kv_heads <= 16 ? 1 : 0;
 }
 
 extern "C" int pe_attention_mma(int decode, const void* q, long long q_ld, void* out, long long out_ld, int n_seqs,
@@ -769,11 +798,29 @@ extern "C" int pe_attention_mma_masked(int decode, const void* q, long long q_ld
                                        const int* seq_slot, const int* page_table, int table_stride, int num_pages,
                                        const void* k_pages, const void* v_pages, float* scratch, int split_keys,
                                        int max_splits, int min_range_keys, int* status, cudaStream_t stream) {
+  return pe_attention_mma_gated(decode, q, q_ld, out, out_ld, n_seqs, max_q, n_heads, n_kv_heads, head_dim, head_dim, scale, window,
+                                chunk, keep_first, v_heads, out_f32, split_p, sink, out_cos, out_sin, out_rows, nullptr, 0,
+                                seq_qstart, seq_past, seq_slot, page_table, table_stride, num_pages, k_pages, v_pages, scratch,
+                                split_keys, max_splits, min_range_keys, status, stream);
+}
+
+// The same with values of a size of their own (`v_dim`; the scratch of a decode step then holds v_dim floats per partial
+// row) and, with `gate` (bfloat16, row of token t at gate + t * gate_ld), each head's output times sigmoid(gate[t, head]).
+extern "C" int pe_attention_mma_gated(int decode, const void* q, long long q_ld, void* out, long long out_ld, int n_seqs,
+                                      int max_q, int n_heads, int n_kv_heads, int head_dim, int v_dim, float scale, int window,
+                                      int chunk, int keep_first, int v_heads, int out_f32, int split_p, int sink,
+                                      const float* out_cos, const float* out_sin, int out_rows, const void* gate,
+                                      long long gate_ld, const int* seq_qstart, const int* seq_past, const int* seq_slot,
+                                      const int* page_table, int table_stride, int num_pages, const void* k_pages,
+                                      const void* v_pages, float* scratch, int split_keys, int max_splits, int min_range_keys,
+                                      int* status, cudaStream_t stream) {
   if (n_seqs <= 0) return PE_OK;
+  const bool exact = head_dim == v_dim && (head_dim == 64 || head_dim == 128);
+  if (!exact && (split_p || out_cos)) return PE_ERR_UNSUPPORTED_SIZE;
   if ((out_cos == nullptr) != (out_sin == nullptr)) return PE_ERR_BAD_ARGUMENT;
   if (chunk < 0 || v_heads <= 0 || (out_f32 && out_cos)) return PE_ERR_BAD_ARGUMENT;
   if (keep_first < 0 || (keep_first > 0 && chunk > 0)) return PE_ERR_BAD_ARGUMENT;
-  if (!pe_attention_mma_supported(head_dim, n_heads, n_kv_heads)) return PE_ERR_UNSUPPORTED_SIZE;
+  if (!pe_attention_mma_dims_supported(head_dim, v_dim, n_heads, n_kv_heads)) return PE_ERR_UNSUPPORTED_SIZE;
   // 16-byte vector loads of q rows; 4-byte (bfloat16 pairs) or 8-byte (float pairs) stores of output rows
   const int out_bytes = out_f32 ? 4 : 2;
   if ((q_ld * 2) % 16 || ((uintptr_t)q % 16) || (out_ld * out_bytes) % (2 * out_bytes) || ((uintptr_t)out % (2 * out_bytes)))
@@ -790,17 +837,29 @@ extern "C" int pe_attention_mma_masked(int decode, const void* q, long long q_ld
   a.sink = sink; a.out_cos = out_cos; a.out_sin = out_sin; a.out_rows = out_rows;
   a.chunk = chunk; a.v_heads = v_heads; a.out_f32 = out_f32; a.split_p = split_p;
   a.keep_first = window > 0 ? keep_first : 0;
+  a.hd = head_dim; a.vd = v_dim; a.gate = (const __nv_bfloat16*)gate; a.gate_ld = gate_ld;
   if (decode) {
     if (!scratch || split_keys < 0 || split_keys % pe::fa::BN || max_splits <= 0) return PE_ERR_BAD_ARGUMENT;
     if (min_range_keys < 0 || min_range_keys % pe::fa::BN) return PE_ERR_BAD_ARGUMENT;
     a.split_keys = split_keys; a.max_splits = max_splits; a.min_range_keys = min_range_keys;
     a.part_acc = scratch;
-    a.part_lse = scratch + (size_t)n_seqs * n_heads * max_splits * head_dim;
+    a.part_lse = scratch + (size_t)n_seqs * n_heads * max_splits * v_dim;
   }
-  if (split_p) {
-    if (head_dim == 64) return pe::fa::launch<64, true>(a, decode != 0, n_seqs, max_q, stream);
-    return pe::fa::launch<128, true>(a, decode != 0, n_seqs, max_q, stream);
+  using pe::fa::launch;
+  const bool dec = decode != 0;
+  if (exact) {
+    if (split_p) {
+      if (head_dim == 64) return launch<64, 64, true, false>(a, dec, n_seqs, max_q, stream);
+      return launch<128, 128, true, false>(a, dec, n_seqs, max_q, stream);
+    }
+    if (head_dim == 64) return launch<64, 64, false, false>(a, dec, n_seqs, max_q, stream);
+    return launch<128, 128, false, false>(a, dec, n_seqs, max_q, stream);
   }
-  if (head_dim == 64) return pe::fa::launch<64, false>(a, decode != 0, n_seqs, max_q, stream);
-  return pe::fa::launch<128, false>(a, decode != 0, n_seqs, max_q, stream);
+  const bool wide = v_dim > 64;
+  switch (tile_of(head_dim)) {
+    case 64: return wide ? launch<64, 128, false, true>(a, dec, n_seqs, max_q, stream) : launch<64, 64, false, true>(a, dec, n_seqs, max_q, stream);
+    case 128: return wide ? launch<128, 128, false, true>(a, dec, n_seqs, max_q, stream) : launch<128, 64, false, true>(a, dec, n_seqs, max_q, stream);
+    case 192: return wide ? launch<192, 128, false, true>(a, dec, n_seqs, max_q, stream) : launch<192, 64, false, true>(a, dec, n_seqs, max_q, stream);
+    default: return wide ? launch<256, 128, false, true>(a, dec, n_seqs, max_q, stream) : launch<256, 64, false, true>(a, dec, n_seqs, max_q, stream);
+  }
 }

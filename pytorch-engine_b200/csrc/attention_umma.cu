@@ -1,5 +1,6 @@
-// Prefill attention on the fifth-generation tensor cores (tcgen05.mma), for bfloat16, head size 128
-// and groups of up to 32 query heads per kv head.  Same interface and formulas as
+// Prefill attention on the fifth-generation tensor cores (tcgen05.mma), for bfloat16, head size 128 (or 72 to 120 in
+// steps of 8, the tile's spare columns filled with zeros by TMA), values of 8 to 128 features (in steps of 8; up to 64 a
+// P.V product of half the width), and groups of up to 32 query heads per kv head.  Same interface and formulas as
 // attention_mma.cu (pygguf_engine/kv_cache.py:833, 2189-2192 masks; 756 head mapping; 836-861 online
 // softmax); other shapes keep using that file.
 //
@@ -69,6 +70,9 @@ struct Args {
   // query's position (interleaved pairs over the whole head; tables [out_rows, HD/2]); off: 0 and null
   int sink;
   const float* out_cos; const float* out_sin; int out_rows;
+  int vd, v_halves;       // size of a value row; 64-feature halves of a V page (1 or 2)
+  // each head's output times sigmoid(gate[token, head]) (rows of the step's tokens, gate_ld apart); null: no gate
+  const __nv_bfloat16* gate; long long gate_ld;
 };
 
 // One work item: the rows [row0, row0 + rows_blk) of sequence b's (token, head) rows for kv head kvh.
@@ -417,9 +421,9 @@ prefill_umma_kernel(Args a, const __grid_constant__ CUtensorMap qmap, const __gr
             break;
           }
           char* vd = v_s + vs * kPageBytes;
-          tma::mbar_expect_tx(&kv_full[vs], more ? 2 * kPageBytes : kPageBytes);
+          tma::mbar_expect_tx(&kv_full[vs], (uint32_t)(a.v_halves * (kPageBytes / 2) + (more ? kPageBytes : 0)));
           tma::load_2d(vd, &vmap, 0, y, &kv_full[vs]);
-          tma::load_2d(vd + BN * 128, &vmap, 64, y, &kv_full[vs]);
+          if (a.v_halves > 1) tma::load_2d(vd + BN * 128, &vmap, 64, y, &kv_full[vs]);
           if (more) load_k(g + 1, y_next, &kv_full[vs]);
           y = y_next;
         }
@@ -431,7 +435,7 @@ prefill_umma_kernel(Args a, const __grid_constant__ CUtensorMap qmap, const __gr
     // ---- MMA issuer ----
     if (lane == 0) {
       const uint32_t idesc_qk = instr_desc(BM, BN, false);
-      const uint32_t idesc_pv = instr_desc(BM, HD, true);
+      const uint32_t idesc_pv = instr_desc(BM, 64 * a.v_halves, true);
       const uint32_t q_lo = desc_lo_k_major(tma::smem_addr(q_s));
       const uint32_t k_lo0 = desc_lo_k_major(tma::smem_addr(k_s));               // stage s: + s * (16 KB / 16)
       const uint32_t v_lo0 = desc_lo_mn_major(tma::smem_addr(v_s), BN * 128);
@@ -553,7 +557,7 @@ prefill_umma_kernel(Args a, const __grid_constant__ CUtensorMap qmap, const __gr
           fence_after_sync();
           const float f = (grow && m_ref != -INFINITY) ? fast_exp2(m_ref - mx) : 1.0f;
 #pragma unroll 1
-          for (int c = 0; c < HD; c += 32) {
+          for (int c = 0; c < 64 * a.v_halves; c += 32) {
             uint32_t ov[32];
             tmem_ld32(tmem_o + c + lane_off, ov);
             tmem_ld_wait();
@@ -598,16 +602,17 @@ prefill_umma_kernel(Args a, const __grid_constant__ CUtensorMap qmap, const __gr
         fence_after_sync();
         // the sink's score is 0: its weight relative to the reference that the row's weights were taken against
         if (a.sink) l += fast_exp2(-((m_ref == -INFINITY) ? 0.f : m_ref));
-        const float inv = 1.f / fmaxf(l, 1e-20f);
+        float inv = 1.f / fmaxf(l, 1e-20f);
         const int tok = row / group, head = w.kvh * group + row % group;
-        __nv_bfloat16* dst = a.out + (size_t)(w.q0 + tok) * a.out_ld + (size_t)head * HD;
+        if (a.gate && live) inv /= 1.f + expf(-__bfloat162float(a.gate[(size_t)(w.q0 + tok) * a.gate_ld + head]));
+        __nv_bfloat16* dst = a.out + (size_t)(w.q0 + tok) * a.out_ld + (size_t)head * a.vd;
         const bool turn = a.out_cos != nullptr;
         const bool pos_ok = qpos >= 0 && qpos < a.out_rows;
         if (turn && live && !pos_ok) report(a.status, kStatusPositionOutOfRange, w.q0 + tok, qpos, a.out_rows);
         const float* cs = turn && pos_ok ? a.out_cos + (size_t)qpos * (HD / 2) : nullptr;
         const float* sn = turn && pos_ok ? a.out_sin + (size_t)qpos * (HD / 2) : nullptr;
 #pragma unroll 1
-        for (int c = 0; c < HD; c += 32) {
+        for (int c = 0; c < a.vd; c += 32) {
           uint32_t ov[32];
           tmem_ld32(tmem_o + c + lane_off, ov);
           tmem_ld_wait();
@@ -634,7 +639,7 @@ prefill_umma_kernel(Args a, const __grid_constant__ CUtensorMap qmap, const __gr
               o4.y = pack2(__uint_as_float(ov[8 * i + 2]) * inv, __uint_as_float(ov[8 * i + 3]) * inv);
               o4.z = pack2(__uint_as_float(ov[8 * i + 4]) * inv, __uint_as_float(ov[8 * i + 5]) * inv);
               o4.w = pack2(__uint_as_float(ov[8 * i + 6]) * inv, __uint_as_float(ov[8 * i + 7]) * inv);
-              *reinterpret_cast<uint4*>(dst + c + 8 * i) = o4;
+              if (c + 8 * i < a.vd) *reinterpret_cast<uint4*>(dst + c + 8 * i) = o4;
             }
           }
         }
@@ -668,6 +673,12 @@ extern "C" int pe_attention_umma_supported(int head_dim, int n_heads, int n_kv_h
   return (g >= 1 && g <= 32) ? 1 : 0;
 }
 
+// The same for keys and values of sizes of their own.
+extern "C" int pe_attention_umma_dims_supported(int head_dim, int v_dim, int n_heads, int n_kv_heads) {
+  if (head_dim <= 64 || head_dim > 128 || head_dim % 8 || v_dim < 8 || v_dim > 128 || v_dim % 8) return 0;
+  return pe_attention_umma_supported(128, n_heads, n_kv_heads);
+}
+
 // Prefill form only (decode keeps attention_mma.cu).  q: rows of the fused q|k|v buffer, [n_tokens, q_ld].
 // n_sms: the device's SM count (sizes the persistent grid).  work_counter: two ints, zero before the call (the
 // kernel leaves them zero), not shared with a call that may run at the same time; null: a fixed schedule.
@@ -690,10 +701,26 @@ extern "C" int pe_attention_umma_prefill_ex(const void* q, long long q_ld, long 
                                             const int* page_table, int table_stride, int num_pages, const void* k_pages,
                                             const void* v_pages, int n_sms, int* work_counter, int* status,
                                             cudaStream_t stream) {
+  return pe_attention_umma_prefill_gated(q, q_ld, n_tokens, out, out_ld, n_seqs, max_q, n_heads, n_kv_heads, head_dim, head_dim,
+                                         scale, window, sink, out_cos, out_sin, out_rows, nullptr, 0, seq_qstart, seq_past,
+                                         seq_slot, page_table, table_stride, num_pages, k_pages, v_pages, n_sms, work_counter,
+                                         status, stream);
+}
+
+// The same with values of a size of their own and, with `gate` (bfloat16, row of token t at gate + t * gate_ld), each head's
+// output times sigmoid(gate[t, head]).
+extern "C" int pe_attention_umma_prefill_gated(const void* q, long long q_ld, long long n_tokens, void* out, long long out_ld,
+                                               int n_seqs, int max_q, int n_heads, int n_kv_heads, int head_dim, int v_dim,
+                                               float scale, int window, int sink, const float* out_cos, const float* out_sin,
+                                               int out_rows, const void* gate, long long gate_ld, const int* seq_qstart,
+                                               const int* seq_past, const int* seq_slot, const int* page_table,
+                                               int table_stride, int num_pages, const void* k_pages, const void* v_pages,
+                                               int n_sms, int* work_counter, int* status, cudaStream_t stream) {
   using namespace pe::fau;
   if (n_seqs <= 0) return PE_OK;
   if ((out_cos == nullptr) != (out_sin == nullptr) || ((uintptr_t)out_cos % 16) || ((uintptr_t)out_sin % 16)) return PE_ERR_BAD_ARGUMENT;
-  if (!pe_attention_umma_supported(head_dim, n_heads, n_kv_heads)) return PE_ERR_UNSUPPORTED_SIZE;
+  if (!pe_attention_umma_dims_supported(head_dim, v_dim, n_heads, n_kv_heads)) return PE_ERR_UNSUPPORTED_SIZE;
+  if (out_cos && (head_dim != 128 || v_dim != 128)) return PE_ERR_UNSUPPORTED_SIZE;
   if (((uintptr_t)q % 16) || (q_ld * 2) % 16 || ((uintptr_t)out % 16) || (out_ld * 2) % 16) return PE_ERR_BAD_ARGUMENT;
   Args a;
   a.out = (__nv_bfloat16*)out; a.out_ld = out_ld; a.n_heads = n_heads; a.n_kv_heads = n_kv_heads;
@@ -701,12 +728,13 @@ extern "C" int pe_attention_umma_prefill_ex(const void* q, long long q_ld, long 
   a.seq_qstart = seq_qstart; a.seq_past = seq_past; a.seq_slot = seq_slot;
   a.page_table = page_table; a.table_stride = table_stride; a.num_pages = num_pages; a.status = status;
   a.sink = sink; a.out_cos = out_cos; a.out_sin = out_sin; a.out_rows = out_rows;
+  a.vd = v_dim; a.v_halves = v_dim > 64 ? 2 : 1; a.gate = (const __nv_bfloat16*)gate; a.gate_ld = gate_ld;
   pe::tma::EncodeTiledFn fn = pe::tma::encode_fn();
   if (fn == nullptr) return -5;
   CUtensorMap qmap, kmap, vmap;
   {
-    cuuint64_t dims[3] = {(cuuint64_t)HD, (cuuint64_t)n_heads, (cuuint64_t)n_tokens};
-    cuuint64_t strides[2] = {(cuuint64_t)HD * 2, (cuuint64_t)q_ld * 2};
+    cuuint64_t dims[3] = {(cuuint64_t)head_dim, (cuuint64_t)n_heads, (cuuint64_t)n_tokens};
+    cuuint64_t strides[2] = {(cuuint64_t)head_dim * 2, (cuuint64_t)q_ld * 2};
     cuuint32_t box[3] = {64, (cuuint32_t)a.group, (cuuint32_t)(BM / a.group)};
     cuuint32_t estr[3] = {1, 1, 1};
     CUresult r = fn(&qmap, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(q), dims, strides, box, estr,
@@ -715,8 +743,8 @@ extern "C" int pe_attention_umma_prefill_ex(const void* q, long long q_ld, long 
     if (r != CUDA_SUCCESS) return PE_ERR_BAD_ARGUMENT;
   }
   const uint64_t rows = (uint64_t)num_pages * n_kv_heads * BN;
-  int me = pe::tma::make_map_2d_bf16(&kmap, k_pages, HD, rows, HD, 64, BN);
-  if (me == 0) me = pe::tma::make_map_2d_bf16(&vmap, v_pages, HD, rows, HD, 64, BN);
+  int me = pe::tma::make_map_2d_bf16(&kmap, k_pages, head_dim, rows, head_dim, 64, BN);
+  if (me == 0) me = pe::tma::make_map_2d_bf16(&vmap, v_pages, v_dim, rows, v_dim, 64, BN);
   if (me != 0) return me < 0 ? me : PE_ERR_BAD_ARGUMENT;
   const size_t smem = kQBytes + (kKStages + kVStages) * kPageBytes + 256;   // tiles, then barriers and the two-slot ring
   static bool attr_set = false;

@@ -121,6 +121,38 @@ __device__ __forceinline__ float silu_mul_fast(float g, float u) {
   return __fdividef(g, 1.0f + __expf(-g)) * u;
 }
 
+// What the epilogue of a fused gate|up product does with the two sums of an output: y = act(g, u), with
+//   kind 1: silu(g) u    2: relu(g) u    3: g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit)
+// and, with `bias` (float32: n gate biases, then n up biases), the biases added first.
+struct GluEpilogue {
+  int kind;
+  float limit, alpha;
+  const float* bias;
+};
+__device__ __forceinline__ float glu_fast(const GluEpilogue& e, float g, float u) {
+  if (e.kind == 1) return silu_mul_fast(g, u);
+  if (e.kind == 2) return fmaxf(g, 0.f) * u;
+  g = fminf(g, e.limit);
+  u = fminf(fmaxf(u, -e.limit), e.limit);
+  return __fdividef(g, 1.0f + __expf(-e.alpha * g)) * (u + 1.0f);
+}
+__device__ __forceinline__ float glu_exact(int kind, float g, float u, float limit, float alpha) {
+  if (kind == 1) return g / (1.f + expf(-g)) * u;
+  if (kind == 2) return fmaxf(g, 0.f) * u;
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+}
+// Two neighbouring outputs, packed to bfloat16; `col`: the first one's number, `n`: outputs in all.
+__device__ __forceinline__ uint32_t glu_fast_pair(const GluEpilogue& e, float g0, float g1, float u0, float u1, int col, int n) {
+  if (e.bias) {
+    if (col < n) { g0 += e.bias[col]; u0 += e.bias[n + col]; }
+    if (col + 1 < n) { g1 += e.bias[col + 1]; u1 += e.bias[n + col + 1]; }
+  }
+  const __nv_bfloat162 v = __floats2bfloat162_rn(glu_fast(e, g0, u0), glu_fast(e, g1, u1));
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+
 // ---- reductions --------------------------------------------------------------------------------
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

@@ -33,6 +33,7 @@ struct Args {
   // rows of matrix i multiply an input of their own, x + i * x_group_stride: several projections of several inputs
   // in one launch.  0: one input for all rows.
   int group_rows; long long x_group_stride;
+  GluEpilogue glu;             // PAIR: what is done with the two sums
 };
 
 __device__ __forceinline__ uint4 ldg_stream(const uint4* p) {
@@ -190,8 +191,12 @@ __global__ void __launch_bounds__(WARPS * 32, NT == 1 ? 16 / WARPS : 1) gemm_sma
       if (col >= a.N || m >= a.M) continue;
       float v = c[n][e];
       if (PAIR) {
-        const float up = c[NT + n][e];
-        v = sizeof(OutT) == 2 ? silu_mul_fast(v, up) : v / (1.0f + expf(-v)) * up;   // exact for a float32 result
+        float up = c[NT + n][e];
+        if (a.glu.bias) {
+          v += a.glu.bias[col];
+          up += a.glu.bias[a.N + col];
+        }
+        v = sizeof(OutT) == 2 ? glu_fast(a.glu, v, up) : glu_exact(a.glu.kind, v, up, a.glu.limit, a.glu.alpha);   // exact for a float32 result
       }
       store_out<OutT>(y + (size_t)m * a.ldy + col, v);
     }
@@ -236,12 +241,21 @@ extern "C" int pe_gemm_smallm_supported(int M, int N, int K) {
 // split of K over a block's warps; 0: a B200's).
 extern "C" int pe_gemm_smallm(const void* x, long long ldx, const void* w, void* y, long long ldy, int M, int N, int K,
                               int out_f32, int pair_offset, int n_sms, cudaStream_t stream) {
+  return pe_gemm_smallm_glu(x, ldx, w, y, ldy, M, N, K, out_f32, pair_offset, 1, 0.f, 1.f, nullptr, n_sms, stream);
+}
+
+// The same with another activation on the pair (GluEpilogue's kinds; bias: float32 [2 * N] or null).
+extern "C" int pe_gemm_smallm_glu(const void* x, long long ldx, const void* w, void* y, long long ldy, int M, int N, int K,
+                                  int out_f32, int pair_offset, int kind, float limit, float alpha, const float* bias, int n_sms,
+                                  cudaStream_t stream) {
   if (M <= 0 || N <= 0) return PE_OK;
+  if (kind < 1 || kind > 3 || (pair_offset <= 0 && bias)) return PE_ERR_BAD_ARGUMENT;
   if (!pe_gemm_smallm_supported(M, N, K)) return PE_ERR_UNSUPPORTED_SIZE;
   if (((uintptr_t)x % 16) || ((uintptr_t)w % 16) || (ldx * 2) % 16) return PE_ERR_BAD_ARGUMENT;
   pe::smallm::Args a;
   a.x = (const __nv_bfloat16*)x; a.ldx = ldx; a.w = (const __nv_bfloat16*)w; a.y = y; a.ldy = ldy;
   a.M = M; a.N = N; a.K = K; a.pair_offset = pair_offset;
+  a.glu = pe::GluEpilogue{kind, limit, alpha, bias};
   a.group_rows = 0; a.x_group_stride = 0;
   using namespace pe::smallm;
   if (n_sms <= 0) n_sms = pe::kSMs;
@@ -268,6 +282,7 @@ extern "C" int pe_gemm_smallm_grouped(const void* x, long long ldx, long long x_
   pe::smallm::Args a;
   a.x = (const __nv_bfloat16*)x; a.ldx = ldx; a.w = (const __nv_bfloat16*)w; a.y = y; a.ldy = ldy;
   a.M = M; a.N = N; a.K = K; a.pair_offset = 0;
+  a.glu = pe::GluEpilogue{1, 0.f, 1.f, nullptr};
   a.group_rows = group_rows; a.x_group_stride = x_group_stride;
   using namespace pe::smallm;
   if (n_sms <= 0) n_sms = pe::kSMs;

@@ -36,6 +36,7 @@ struct Params {
   int pair_offset;        // mode 2: row of W that pairs with row 0
   int m_tiles, n_tiles, n_per_tile;
   int* status;
+  GluEpilogue glu;        // mode 2
 };
 
 // ---- tcgen05 wrappers ----------------------------------------------------------------------------
@@ -218,12 +219,19 @@ gemm_umma_kernel(Params p, const __grid_constant__ CUtensorMap amap, const __gri
           tmem_ld_wait();
           if (row < p.M) {
             uint32_t o[16];
+            if (p.glu.kind == 1 && p.glu.bias == nullptr) {
 #pragma unroll
-            for (int j = 0; j < 16; ++j) {
-              const float g0 = __uint_as_float(g[2 * j]), g1 = __uint_as_float(g[2 * j + 1]);
-              const float v0 = silu_mul_fast(g0, __uint_as_float(u[2 * j]));
-              const float v1 = silu_mul_fast(g1, __uint_as_float(u[2 * j + 1]));
-              o[j] = pack2(v0, v1);
+              for (int j = 0; j < 16; ++j) {
+                const float g0 = __uint_as_float(g[2 * j]), g1 = __uint_as_float(g[2 * j + 1]);
+                const float v0 = silu_mul_fast(g0, __uint_as_float(u[2 * j]));
+                const float v1 = silu_mul_fast(g1, __uint_as_float(u[2 * j + 1]));
+                o[j] = pack2(v0, v1);
+              }
+            } else {
+#pragma unroll
+              for (int j = 0; j < 16; ++j)
+                o[j] = glu_fast_pair(p.glu, __uint_as_float(g[2 * j]), __uint_as_float(g[2 * j + 1]), __uint_as_float(u[2 * j]),
+                                     __uint_as_float(u[2 * j + 1]), n0 + c + 2 * j, p.N);
             }
             if (n0 + c + 32 <= p.N && (p.ldy % 8) == 0) {
 #pragma unroll
@@ -297,14 +305,23 @@ extern "C" int pe_gemm_umma_supported(int M, int N, int K, int pair_offset) {
 // y[m, n] = silu(x . gate_n) * (x . up_n), bfloat16.  x rows may be strided (ldx), W rows are dense.
 extern "C" int pe_gemm_umma(const void* x, long long ldx, const void* w, void* y, long long ldy, int M, int N, int K,
                             int out_f32, int pair_offset, int n_sms, int* status, cudaStream_t stream) {
+  return pe_gemm_umma_glu(x, ldx, w, y, ldy, M, N, K, out_f32, pair_offset, 1, 0.f, 1.f, nullptr, n_sms, status, stream);
+}
+
+// The same with another activation on the pair (GluEpilogue's kinds; bias: float32 [2 * N] or null).
+extern "C" int pe_gemm_umma_glu(const void* x, long long ldx, const void* w, void* y, long long ldy, int M, int N, int K,
+                        int out_f32, int pair_offset, int kind, float limit, float alpha, const float* bias, int n_sms, int* status,
+                        cudaStream_t stream) {
   using namespace pe::umma;
   if (M <= 0 || N <= 0) return PE_OK;
+  if (kind < 1 || kind > 3 || (pair_offset <= 0 && bias)) return PE_ERR_BAD_ARGUMENT;
   if (!pe_gemm_umma_supported(M, N, K, pair_offset)) return PE_ERR_UNSUPPORTED_SIZE;
   if (((uintptr_t)x % 16) || ((uintptr_t)w % 16) || (ldx * 2) % 16) return PE_ERR_BAD_ARGUMENT;
   Params p;
   p.M = M; p.N = N; p.K = K; p.y = y; p.ldy = ldy; p.status = status;
   p.mode = pair_offset > 0 ? 2 : (out_f32 ? 1 : 0);
   p.pair_offset = pair_offset;
+  p.glu = pe::GluEpilogue{kind, limit, alpha, bias};
   p.n_per_tile = pair_offset > 0 ? 128 : BN;
   p.m_tiles = (M + BM - 1) / BM;
   p.n_tiles = (N + p.n_per_tile - 1) / p.n_per_tile;

@@ -65,6 +65,7 @@ struct Params {
   int m_tiles, n_tiles, n_per_tile;
   int* status;
   RopeFuse rope;
+  GluEpilogue glu;        // mode 2
 };
 
 __device__ __forceinline__ uint32_t cluster_rank() {
@@ -434,12 +435,19 @@ gemm_umma2_kernel(Params p, const __grid_constant__ CUtensorMap amap, const __gr
           tmem_ld_wait();
           if (row < p.M) {
             uint32_t o[16];
+            if (p.glu.kind == 1 && p.glu.bias == nullptr) {
 #pragma unroll
-            for (int j = 0; j < 16; ++j) {
-              const float g0 = __uint_as_float(g[2 * j]), g1 = __uint_as_float(g[2 * j + 1]);
-              const float v0 = silu_mul_fast(g0, __uint_as_float(u[2 * j]));
-              const float v1 = silu_mul_fast(g1, __uint_as_float(u[2 * j + 1]));
-              o[j] = pack2(v0, v1);
+              for (int j = 0; j < 16; ++j) {
+                const float g0 = __uint_as_float(g[2 * j]), g1 = __uint_as_float(g[2 * j + 1]);
+                const float v0 = silu_mul_fast(g0, __uint_as_float(u[2 * j]));
+                const float v1 = silu_mul_fast(g1, __uint_as_float(u[2 * j + 1]));
+                o[j] = pack2(v0, v1);
+              }
+            } else {
+#pragma unroll
+              for (int j = 0; j < 16; ++j)
+                o[j] = glu_fast_pair(p.glu, __uint_as_float(g[2 * j]), __uint_as_float(g[2 * j + 1]), __uint_as_float(u[2 * j]),
+                                     __uint_as_float(u[2 * j + 1]), n0 + c + 2 * j, p.N);
             }
             if (n0 + c + 32 <= p.N && (p.ldy % 8) == 0) {
 #pragma unroll
@@ -520,14 +528,23 @@ static int launch_pair(Params p, const void* x, long long ldx, const void* w, in
 // The arguments of pe_gemm_umma (gemm_umma.cu); n_sms is rounded down to pairs; K a multiple of 64.
 extern "C" int pe_gemm_umma2(const void* x, long long ldx, const void* w, void* y, long long ldy, int M, int N, int K,
                              int out_f32, int pair_offset, int n_sms, int* status, cudaStream_t stream) {
+  return pe_gemm_umma2_glu(x, ldx, w, y, ldy, M, N, K, out_f32, pair_offset, 1, 0.f, 1.f, nullptr, n_sms, status, stream);
+}
+
+// The same with another activation on the pair (GluEpilogue's kinds; bias: float32 [2 * N] or null).
+extern "C" int pe_gemm_umma2_glu(const void* x, long long ldx, const void* w, void* y, long long ldy, int M, int N, int K,
+                        int out_f32, int pair_offset, int kind, float limit, float alpha, const float* bias, int n_sms, int* status,
+                        cudaStream_t stream) {
   using namespace pe::umma2;
   if (M <= 0 || N <= 0) return PE_OK;
+  if (kind < 1 || kind > 3 || (pair_offset <= 0 && bias)) return PE_ERR_BAD_ARGUMENT;
   if (!pe_gemm_umma2_supported(M, N, K, pair_offset) || n_sms < 2) return PE_ERR_UNSUPPORTED_SIZE;
   if (((uintptr_t)x % 16) || ((uintptr_t)w % 16) || (ldx * 2) % 16) return PE_ERR_BAD_ARGUMENT;
   Params p;
   p.M = M; p.N = N; p.K = K; p.y = y; p.ldy = ldy; p.status = status;
   p.mode = pair_offset > 0 ? 2 : (out_f32 ? 1 : 0);
   p.pair_offset = pair_offset;
+  p.glu = pe::GluEpilogue{kind, limit, alpha, bias};
   p.rope = RopeFuse();
   return launch_pair(p, x, ldx, w, n_sms, stream);
 }
@@ -562,6 +579,7 @@ extern "C" int pe_gemm_umma2_qkv_rope(const void* x, long long ldx, const void* 
   p.M = M; p.N = (n_heads + 2 * n_kv_heads) * head_dim; p.K = K; p.y = qkv; p.ldy = ld; p.status = status;
   p.mode = 3;
   p.pair_offset = 0;
+  p.glu = pe::GluEpilogue{1, 0.f, 1.f, nullptr};
   RopeFuse& r = p.rope;
   r.n_heads = n_heads; r.n_kv_heads = n_kv_heads; r.q_norm_w = q_norm_w; r.k_norm_w = k_norm_w; r.eps = eps;
   r.cos_table = rotary_dim > 0 ? cos_table : nullptr; r.sin_table = rotary_dim > 0 ? sin_table : nullptr;

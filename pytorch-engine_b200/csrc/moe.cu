@@ -218,14 +218,6 @@ __global__ void moe_group_kernel(const int* chosen, int n_pairs, int top, int n_
 constexpr int kMoeRows = 8;
 constexpr int kMoeCols = 32;
 
-__device__ __forceinline__ float glu_value(int kind, float g, float u, float limit, float alpha) {
-  if (kind == 1) return g / (1.f + expf(-g)) * u;
-  if (kind == 2) return fmaxf(g, 0.f) * u;
-  g = fminf(g, limit);
-  u = fminf(fmaxf(u, -limit), limit);
-  return g / (1.f + expf(-alpha * g)) * (u + 1.f);
-}
-
 template <typename T> struct WVec;
 template <> struct WVec<float> {
   static constexpr int N = 4;
@@ -331,7 +323,7 @@ __global__ void __launch_bounds__(256) moe_rows_gemm_kernel(const T* x, long lon
         if (glu) {
           // the two products are rounded as a kernel that writes them would round them
           const float g = to_f32<T>(from_f32<T>(acc[r])), u = to_f32<T>(from_f32<T>(acc2[r]));
-          y = glu_value(glu, g, u, limit, alpha);
+          y = glu_exact(glu, g, u, limit, alpha);
         }
         out[(size_t)(first + r) * out_ld + n] = from_f32<TOut>(y);
       }
@@ -424,17 +416,46 @@ __global__ void moe_combine_vec8_kernel(const __nv_bfloat16* rows, const __nv_bf
   }
 }
 
-// act(gate, up) over the two halves of a row of a [gate | up] product (kinds as above)
+// act(gate, up) over the two halves of a row of a [gate | up] product (kinds as above); bias: [2 * inter] added first, or null
 template <typename T>
-__global__ void glu_act_kernel(const T* gate_up, T* __restrict__ out, int n_rows, int inter, int kind, float limit, float alpha) {
+__global__ void glu_act_kernel(const T* gate_up, T* __restrict__ out, int n_rows, int inter, int kind, float limit, float alpha,
+                               const float* __restrict__ bias) {
   pdl_wait_block();
   pdl_launch_dependents();
   const size_t total = (size_t)n_rows * inter;
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
     const size_t r = i / inter, c = i - r * inter;
-    const float g = to_f32<T>(gate_up[r * 2 * inter + c]);
-    const float u = to_f32<T>(gate_up[r * 2 * inter + inter + c]);
-    out[i] = from_f32<T>(glu_value(kind, g, u, limit, alpha));
+    float g = to_f32<T>(gate_up[r * 2 * inter + c]);
+    float u = to_f32<T>(gate_up[r * 2 * inter + inter + c]);
+    if (bias) {
+      g += bias[c];
+      u += bias[inter + c];
+    }
+    out[i] = from_f32<T>(glu_exact(kind, g, u, limit, alpha));
+  }
+}
+
+// The same for bfloat16 with 16-byte accesses (inter a multiple of 8, everything 16-byte aligned).
+__global__ void __launch_bounds__(256) glu_act_vec8_kernel(const __nv_bfloat16* gate_up, __nv_bfloat16* __restrict__ out, int n_rows,
+                                                           int inter, GluEpilogue e) {
+  pdl_wait_block();
+  pdl_launch_dependents();
+  const int per_row = inter / 8;
+  const size_t total = (size_t)n_rows * per_row;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t r = i / per_row;
+    const int c = (int)(i - r * per_row) * 8;
+    const uint4 graw = *reinterpret_cast<const uint4*>(gate_up + r * 2 * inter + c);
+    const uint4 uraw = *reinterpret_cast<const uint4*>(gate_up + r * 2 * inter + inter + c);
+    const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&graw);
+    const __nv_bfloat162* u2 = reinterpret_cast<const __nv_bfloat162*>(&uraw);
+    uint32_t o[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const float2 g = __bfloat1622float2(g2[k]), u = __bfloat1622float2(u2[k]);
+      o[k] = glu_fast_pair(e, g.x, g.y, u.x, u.y, c + 2 * k, inter);
+    }
+    *reinterpret_cast<uint4*>(out + r * inter + c) = make_uint4(o[0], o[1], o[2], o[3]);
   }
 }
 
@@ -566,18 +587,26 @@ extern "C" int pe_moe_combine(int dtype, const void* rows, const void* x, const 
 }
 
 extern "C" int pe_glu_act(int dtype, const void* gate_up, void* out, int n_rows, int inter, int kind, float limit, float alpha,
-                          cudaStream_t stream) {
+                          const float* bias, cudaStream_t stream) {
   if (n_rows <= 0) return PE_OK;
   if (inter <= 0 || kind < 1 || kind > 3) return PE_ERR_BAD_ARGUMENT;
   const size_t total = (size_t)n_rows * inter;
   const int threads = 256;
   size_t blocks = (total + threads - 1) / threads;
   if (blocks > pe::kSMs * 16) blocks = pe::kSMs * 16;
+  if (dtype == PE_BF16 && inter % 8 == 0 && (uintptr_t)gate_up % 16 == 0 && (uintptr_t)out % 16 == 0) {
+    pe::GluEpilogue e = {kind, limit, alpha, bias};
+    blocks = (total / 8 + threads - 1) / threads;
+    if (blocks > pe::kSMs * 16) blocks = pe::kSMs * 16;
+    pe::launch(pe::glu_act_vec8_kernel, (int)blocks, threads, 0, stream, (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, n_rows, inter, e);
+    PE_LAUNCH_CHECK();
+    return PE_OK;
+  }
   if (dtype == PE_F32)
-    pe::launch(pe::glu_act_kernel<float>, (int)blocks, threads, 0, stream, (const float*)gate_up, (float*)out, n_rows, inter, kind, limit, alpha);
+    pe::launch(pe::glu_act_kernel<float>, (int)blocks, threads, 0, stream, (const float*)gate_up, (float*)out, n_rows, inter, kind, limit, alpha, bias);
   else if (dtype == PE_BF16)
     pe::launch(pe::glu_act_kernel<__nv_bfloat16>, (int)blocks, threads, 0, stream, (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out,
-               n_rows, inter, kind, limit, alpha);
+               n_rows, inter, kind, limit, alpha, bias);
   else
     return PE_ERR_UNSUPPORTED_DTYPE;
   PE_LAUNCH_CHECK();

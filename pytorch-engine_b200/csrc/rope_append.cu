@@ -388,6 +388,11 @@ struct QkvRotateArgs {
   int write_cache;
   int* status;
   const float* bias;   // [q | k | v features] added to the projected rows first (null: none)
+  int qk_unit;         // != 0: q and k are divided by their root mean square over the head after the rotation
+  // Values mixed with another layer's values of the same tokens: v <- (1 - v_lambda) v + v_lambda v_mix, before
+  // anything else but the bias.  v_keep: the (mixed) values are also left there, for layers further on.
+  const void* v_mix; void* v_keep;   // [n_tokens, n_kv_heads * v_dim] run dtype, or null
+  float v_lambda;
 };
 
 template <typename T>
@@ -448,7 +453,7 @@ __global__ void qkv_rotate_append_kernel(QkvRotateArgs a) {
       const float x = to_f32<T>(row[c]) + (bias ? bias[c] : 0.f);
       ss += x * x;
     }
-    inv = rsqrtf(warp_sum(ss) / (float)D + a.eps);
+    inv = rsqrtf(warp_sum(ss) / (float)D + a.eps);     // (values with a norm are not mixed: the launcher refuses that)
   }
   const float* ct = is_v ? a.v_cos : a.cos_table;
   const float* st = is_v ? a.v_sin : a.sin_table;
@@ -460,26 +465,202 @@ __global__ void qkv_rotate_append_kernel(QkvRotateArgs a) {
     if (lane == 0) report(a.status, kStatusPositionOutOfRange, t, pos, rows);
     return;
   }
+  const size_t v_off = is_v ? ((size_t)t * a.n_kv_heads + kv_head) * a.v_dim : 0;
+  const T* v_mix = is_v && a.v_mix ? (const T*)a.v_mix + v_off : nullptr;
+  T* v_keep = is_v && a.v_keep ? (T*)a.v_keep + v_off : nullptr;
   auto value = [&](int c) -> float {
     float x = to_f32<T>(row[c]);
     if (bias) x += bias[c];
+    if (v_mix) x = (1.f - a.v_lambda) * x + a.v_lambda * to_f32<T>(v_mix[c]);
     if (normed) x *= inv;
     if (w) x *= w[c];
     return x;
   };
+  float unit = 1.f;    // what the rotated q or k row is multiplied by
   auto put = [&](int c, float x) {
-    const T o = from_f32<T>(x);
+    const T o = from_f32<T>(x * unit);
     if (!is_v) row[c] = o;
+    if (v_keep) v_keep[c] = o;
     if (cache_row) cache_row[c] = o;
   };
-  for (int j = lane; j < half; j += 32) {
-    const int i0 = inter ? 2 * j : j, i1 = inter ? 2 * j + 1 : j + half;
+  auto turned = [&](int j, int& i0, int& i1, float& y0, float& y1) {
+    i0 = inter ? 2 * j : j;
+    i1 = inter ? 2 * j + 1 : j + half;
     const float x0 = value(i0), x1 = value(i1);
     const float c = ct[(size_t)pos * half + j], s = st[(size_t)pos * half + j];
-    put(i0, x0 * c - x1 * s);
-    put(i1, x1 * c + x0 * s);
+    y0 = x0 * c - x1 * s;
+    y1 = x1 * c + x0 * s;
+  };
+  int i0, i1;
+  float y0, y1;
+  if (a.qk_unit && !is_v) {
+    float ss = 0.f;
+    for (int j = lane; j < half; j += 32) {
+      turned(j, i0, i1, y0, y1);
+      ss += y0 * y0 + y1 * y1;
+    }
+    for (int c = rot + lane; c < D; c += 32) {
+      const float x = value(c);
+      ss += x * x;
+    }
+    unit = rsqrtf(warp_sum(ss) / (float)D + a.eps);
+  }
+  for (int j = lane; j < half; j += 32) {
+    turned(j, i0, i1, y0, y1);
+    put(i0, y0);
+    put(i1, y1);
   }
   for (int c = rot + lane; c < D; c += 32) put(c, value(c));
+}
+
+// The general form for bfloat16 rows with 16-byte accesses and split-half pairs: bias, unit q and k after the rotation, mixed
+// and kept values.  Head and value sizes of their own, multiples of 8 up to 256; half the rotated size a multiple of 8.
+// A head takes size / 8 lanes (a warp holds as many whole heads as fit); a block's first warps take q and k heads, the rest
+// values.  The lane that holds features [8i, 8i + 8) of the first rotated half trades its values with the lane that holds
+// the matching features of the second half.  A block takes TPB tokens and has all their rows in flight before the first use.
+template <int TPB>
+__global__ void __launch_bounds__(256) qkv_rotate_append_halves_kernel(QkvRotateArgs a, int qk_warps) {
+  typedef __nv_bfloat16 T;
+  const int lane = threadIdx.x & 31;
+  const int gw = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const bool is_v = gw >= qk_warps;
+  const int D = is_v ? a.v_dim : a.head_dim;
+  const int lph = D >> 3, per_warp = 32 / lph;
+  const int sub = lane / lph, li = lane - sub * lph;
+  const int idx = (is_v ? gw - qk_warps : gw) * per_warp + sub;       // head among q|k, or value head
+  const bool active = sub < per_warp && idx < (is_v ? a.n_kv_heads : a.n_heads + a.n_kv_heads);
+  const bool is_q = !is_v && idx < a.n_heads;
+  const int kv_head = is_v ? idx : idx - a.n_heads;
+  const size_t row_off = is_v ? (size_t)(a.n_heads + a.n_kv_heads) * a.head_dim + (size_t)idx * D : (size_t)idx * D;
+  const int rot = is_v ? 0 : a.rotary_dim, half = rot >> 1, half_l = half >> 3;
+  const bool turns = active && 8 * li < rot;
+  const bool second = li >= half_l;
+  const int j = 8 * (second ? li - half_l : li);
+  const int partner = turns ? lane + (second ? -half_l : half_l) : lane;
+  const bool pow2 = (lph & (lph - 1)) == 0;
+  float bv[8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) bv[e] = 0.f;
+  if (active && a.bias) {
+    const float4 b0 = *reinterpret_cast<const float4*>(a.bias + row_off + 8 * li), b1 = *reinterpret_cast<const float4*>(a.bias + row_off + 8 * li + 4);
+    bv[0] = b0.x; bv[1] = b0.y; bv[2] = b0.z; bv[3] = b0.w; bv[4] = b1.x; bv[5] = b1.y; bv[6] = b1.z; bv[7] = b1.w;
+  }
+  // the batch description and the page table do not come from the kernel before this one
+  int poss[TPB], page[TPB], qend[TPB], qbeg[TPB];
+#pragma unroll
+  for (int i = 0; i < TPB; ++i) {
+    const int t = blockIdx.x * TPB + i;
+    poss[i] = 0; page[i] = -1; qend[i] = 0; qbeg[i] = 0;
+    if (t < a.n_tokens) {
+      poss[i] = a.token_pos[t];
+      if (active && !is_q && a.write_cache) {
+        const int b = a.token_seq[t];
+        const int slot = a.seq_slot[b];
+        qbeg[i] = a.seq_qstart[b];
+        qend[i] = a.seq_qstart[b + 1];
+        if (poss[i] >= 0 && poss[i] / kPageTokens < a.table_stride) page[i] = a.page_table[(size_t)slot * a.table_stride + poss[i] / kPageTokens];
+      }
+    }
+  }
+  pdl_wait_block();
+  pdl_launch_dependents();
+  uint4 raws[TPB], mixed[TPB];
+#pragma unroll
+  for (int i = 0; i < TPB; ++i) {
+    const int t = blockIdx.x * TPB + i;
+    raws[i] = mixed[i] = make_uint4(0, 0, 0, 0);
+    if (t < a.n_tokens && active) {
+      raws[i] = *reinterpret_cast<const uint4*>((const T*)a.qkv + (size_t)t * a.ld + row_off + 8 * li);
+      if (is_v && a.v_mix) mixed[i] = *reinterpret_cast<const uint4*>((const T*)a.v_mix + ((size_t)t * a.n_kv_heads + idx) * D + 8 * li);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < TPB; ++i) {
+    const int t = blockIdx.x * TPB + i;
+    if (t >= a.n_tokens) break;
+    const int pos = poss[i];
+    T* cache_row = nullptr;
+    if (active && !is_q && a.write_cache) {
+      if (pos < 0 || pos / kPageTokens >= a.table_stride) {
+        if (li == 0) report(a.status, kStatusPositionOutOfRange, t, pos, a.table_stride * kPageTokens);
+      } else if (page[i] < 0 || page[i] >= a.num_pages) {
+        if (li == 0) report(a.status, kStatusPageOutOfRange, t, page[i], a.num_pages);
+      } else {
+        T* base = (T*)(is_v ? a.v_pages : a.k_pages);
+        const int off = pos % kPageTokens;
+        T* head_row = base + (((size_t)page[i] * a.n_kv_heads + kv_head) * kPageTokens + off) * D;
+        cache_row = head_row + 8 * li;
+        if (t + 1 == qend[i] && off + 1 < kPageTokens && (off == 0 || qend[i] - qbeg[i] > 1)) {
+          uint4* r4 = reinterpret_cast<uint4*>(head_row + D);      // clear the rest of the page (see the first kernel)
+          const size_t n4 = (size_t)(kPageTokens - 1 - off) * D / 8;
+          for (size_t x = li; x < n4; x += lph) r4[x] = make_uint4(0, 0, 0, 0);
+        }
+      }
+    }
+    float x[8];
+    {
+      const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raws[i]);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 f = __bfloat1622float2(h2[e]);
+        x[2 * e] = f.x + bv[2 * e];
+        x[2 * e + 1] = f.y + bv[2 * e + 1];
+      }
+    }
+    if (is_v) {       // (whole warps: nothing below shuffles across q|k and value warps)
+      if (a.v_mix) {
+        const __nv_bfloat162* m2 = reinterpret_cast<const __nv_bfloat162*>(&mixed[i]);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 f = __bfloat1622float2(m2[e]);
+          x[2 * e] = (1.f - a.v_lambda) * x[2 * e] + a.v_lambda * f.x;
+          x[2 * e + 1] = (1.f - a.v_lambda) * x[2 * e + 1] + a.v_lambda * f.y;
+        }
+      }
+    } else {
+      float other[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) other[e] = __shfl_sync(0xffffffffu, x[e], partner & 31);
+      bool ok = true;
+      if (turns) {
+        ok = pos >= 0 && pos < a.table_rows;
+        if (!ok && li == 0) report(a.status, kStatusPositionOutOfRange, t, pos, a.table_rows);
+        const int prow = ok ? pos : 0;
+        const float* cs = a.cos_table + (size_t)prow * half + j;     // the tables stay in L2
+        const float* sn = a.sin_table + (size_t)prow * half + j;
+        const float4 c0 = *reinterpret_cast<const float4*>(cs), c1 = *reinterpret_cast<const float4*>(cs + 4);
+        const float4 s0 = *reinterpret_cast<const float4*>(sn), s1 = *reinterpret_cast<const float4*>(sn + 4);
+        const float cv[8] = {c0.x, c0.y, c0.z, c0.w, c1.x, c1.y, c1.z, c1.w};
+        const float sv[8] = {s0.x, s0.y, s0.z, s0.w, s1.x, s1.y, s1.z, s1.w};
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = second ? x[e] * cv[e] + other[e] * sv[e] : x[e] * cv[e] - other[e] * sv[e];
+      }
+      if (a.qk_unit) {
+        float ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
+        if (pow2) {
+          for (int o = lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        } else {
+          float total = 0.f;
+          for (int l = 0; l < lph; ++l) total += __shfl_sync(0xffffffffu, ss, (sub * lph + l) & 31);
+          ss = total;
+        }
+        const float inv = rsqrtf(ss / (float)D + a.eps);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] *= inv;
+      }
+      if (!ok) continue;
+    }
+    if (!active) continue;
+    uint4 out;
+    __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&out);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o2[e] = __floats2bfloat162_rn(x[2 * e], x[2 * e + 1]);
+    if (!is_v) *reinterpret_cast<uint4*>((T*)a.qkv + (size_t)t * a.ld + row_off + 8 * li) = out;
+    else if (a.v_keep) *reinterpret_cast<uint4*>((T*)a.v_keep + ((size_t)t * a.n_kv_heads + idx) * D + 8 * li) = out;
+    if (cache_row) *reinterpret_cast<uint4*>(cache_row) = out;
+  }
 }
 
 // The general form for bfloat16 rows with 16-byte accesses: keys and values of one size that is a multiple of 8 (up to
@@ -680,8 +861,10 @@ extern "C" int pe_qkv_rotate_append(int dtype, void* qkv, long long ld, int n_to
                                     int v_rotary_dim, int v_table_rows, int v_interleaved, const int* token_seq,
                                     const int* token_pos, const int* seq_slot, const int* seq_qstart,
                                     const int* page_table, int table_stride, int num_pages, void* k_pages,
-                                    void* v_pages, int write_cache, const float* bias, int* status, cudaStream_t stream) {
+                                    void* v_pages, int write_cache, const float* bias, int qk_unit, const void* v_mix,
+                                    float v_lambda, void* v_keep, int* status, cudaStream_t stream) {
   if (n_tokens <= 0) return PE_OK;
+  if (v_mix && v_unit_norm) return PE_ERR_BAD_ARGUMENT;
   if (head_dim <= 0 || v_dim <= 0 || n_heads <= 0 || n_kv_heads < 0) return PE_ERR_BAD_ARGUMENT;
   if (rotary_dim < 0 || rotary_dim > head_dim || (rotary_dim & 1)) return PE_ERR_UNSUPPORTED_SIZE;
   if (v_rotary_dim < 0 || v_rotary_dim > v_dim || (v_rotary_dim & 1)) return PE_ERR_UNSUPPORTED_SIZE;
@@ -696,11 +879,33 @@ extern "C" int pe_qkv_rotate_append(int dtype, void* qkv, long long ld, int n_to
   a.token_seq = token_seq; a.token_pos = token_pos; a.seq_slot = seq_slot; a.seq_qstart = seq_qstart;
   a.page_table = page_table; a.table_stride = table_stride; a.num_pages = num_pages;
   a.k_pages = k_pages; a.v_pages = v_pages; a.write_cache = write_cache; a.status = status; a.bias = bias;
+  a.qk_unit = qk_unit; a.v_mix = v_mix; a.v_keep = v_keep; a.v_lambda = v_lambda;
   const int warps = 4;
   dim3 grid(n_tokens, (n_heads + 2 * n_kv_heads + warps - 1) / warps);
   if (grid.y > 65535) return PE_ERR_UNSUPPORTED_SIZE;
   auto al16 = [](const void* p) { return (uintptr_t)p % 16 == 0; };
-  const bool vec8 = dtype == PE_BF16 && bias == nullptr && head_dim == v_dim && head_dim % 8 == 0 && head_dim <= 256 && ld % 8 == 0 &&
+  const bool halves = dtype == PE_BF16 && q_norm_w == nullptr && k_norm_w == nullptr && !v_unit_norm && a.v_rotary_dim == 0 &&
+                      head_dim % 8 == 0 && head_dim <= 256 && v_dim % 8 == 0 && v_dim <= 256 && ld % 8 == 0 &&
+                      (a.rotary_dim == 0 || (!interleaved && a.rotary_dim % 16 == 0)) && al16(qkv) && al16(k_pages) && al16(v_pages) &&
+                      al16(cos_table) && al16(sin_table) && al16(bias) && al16(v_mix) && al16(v_keep);
+  if (halves) {
+    const int qk_per_warp = 32 / (head_dim / 8), v_per_warp = 32 / (v_dim / 8);
+    const int qk_warps = (n_heads + n_kv_heads + qk_per_warp - 1) / qk_per_warp;
+    const int all_warps = qk_warps + (n_kv_heads + v_per_warp - 1) / v_per_warp;
+    if (n_tokens >= 256) {
+      constexpr int kTokensPerBlock = 4;
+      dim3 g((n_tokens + kTokensPerBlock - 1) / kTokensPerBlock, (all_warps + 7) / 8);
+      if (g.y > 65535) return PE_ERR_UNSUPPORTED_SIZE;
+      pe::launch(pe::qkv_rotate_append_halves_kernel<kTokensPerBlock>, g, 256, 0, stream, a, qk_warps);
+    } else {
+      dim3 g(n_tokens, (all_warps + 3) / 4);
+      if (g.y > 65535) return PE_ERR_UNSUPPORTED_SIZE;
+      pe::launch(pe::qkv_rotate_append_halves_kernel<1>, g, 128, 0, stream, a, qk_warps);
+    }
+    PE_LAUNCH_CHECK();
+    return PE_OK;
+  }
+  const bool vec8 = dtype == PE_BF16 && bias == nullptr && !qk_unit && !v_mix && !v_keep && head_dim == v_dim && head_dim % 8 == 0 && head_dim <= 256 && ld % 8 == 0 &&
                     (a.rotary_dim == 0 || (interleaved && a.rotary_dim % 8 == 0)) &&
                     (a.v_rotary_dim == 0 || (v_interleaved && a.v_rotary_dim % 8 == 0)) && al16(qkv) && al16(k_pages) &&
                     al16(v_pages) && al16(cos_table) && al16(sin_table) && al16(v_cos) && al16(v_sin) && al16(q_norm_w) &&

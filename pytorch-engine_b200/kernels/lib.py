@@ -58,7 +58,7 @@ _SIGNATURES = {
     "pe_gemm_umma2_supported": [I, I, I, I],
     "pe_gemm_umma2_qkv_rope_supported": [I, I, I, I, I, I],
     "pe_gemm_umma2_qkv_rope": [P, L, P, P, L, I, I, I, I, I, P, P, F, P, P, I, I, P, P, P, P, P, I, I, P, P, I, I, P, P],
-    "pe_attention_mma_decode_blocks_per_sm": [I],
+    "pe_attention_mma_decode_blocks_per_sm": [I, I],
     "pe_attention_umma_prefill": [P, L, L, P, L, I, I, I, I, I, F, I, P, P, P, P, I, I, P, P, I, P, P, P],
     "pe_attention_umma_supported": [I, I, I],
     "pe_wait_probe": [P, I, P],
@@ -68,7 +68,7 @@ _SIGNATURES = {
     "pe_tanh_inplace": [I, P, L, P],
     "pe_wkv_recurrence": [I, P, P, P, P, L, P, P, P, P, F, P, P, P, P, I, P, P, I, I, I, I, I, I, I, P, P, P],
     "pe_qkv_rotate_append": [I, P, L, I, I, I, I, I, P, P, F, P, P, I, I, I, I, P, P, I, I, I, P, P, P, P, P, I, I, P, P,
-                             I, P, P, P],
+                             I, P, I, P, F, P, P, P],
     "pe_attention_generic_ex": [I, I, P, L, P, L, I, I, I, I, I, I, F, I, I, P, P, I, I, I, P, P, P, P, I, I, P, P, P,
                                 I, I, P, P],
     "pe_attention_mma_ex": [I, P, L, P, L, I, I, I, I, I, F, I, I, P, P, I, P, P, P, P, I, I, P, P, P, I, I, I, P, P],
@@ -88,7 +88,17 @@ _SIGNATURES = {
     "pe_moe_rows_gemm": [I, I, P, L, P, P, I, I, P, L, P, L, I, I, I, F, F, P],
     "pe_moe_gather_rows": [I, P, P, P, I, P, I, I, P],
     "pe_moe_combine": [I, P, P, P, P, P, I, P, I, I, P],
-    "pe_glu_act": [I, P, P, I, I, I, F, F, P],
+    "pe_glu_act": [I, P, P, I, I, I, F, F, P, P],
+    "pe_gemm_smallm_glu": [P, L, P, P, L, I, I, I, I, I, I, F, F, P, I, P],
+    "pe_gemm_umma_glu": [P, L, P, P, L, I, I, I, I, I, I, F, F, P, I, P, P],
+    "pe_gemm_umma2_glu": [P, L, P, P, L, I, I, I, I, I, I, F, F, P, I, P, P],
+    "pe_stream_mix": [I, P, P, P, P, P, P, P, I, P, F, P, P, I, I, I, P],
+    "pe_layernorm": [I, P, P, P, I, I, F, P],
+    "pe_attention_mma_dims_supported": [I, I, I, I],
+    "pe_attention_mma_gated": [I, P, L, P, L, I, I, I, I, I, I, F, I, I, I, I, I, I, I, P, P, I, P, L, P, P, P, P, I, I, P, P, P, I, I, I,
+                               P, P],
+    "pe_attention_umma_dims_supported": [I, I, I, I],
+    "pe_attention_umma_prefill_gated": [P, L, L, P, L, I, I, I, I, I, I, F, I, I, P, P, I, P, L, P, P, P, P, I, I, P, P, I, P, P, P],
     "pe_moe_route_logits": [P, P, I, I, I, P, P, P, I, P],
     "pe_attention_generic_masked": [I, I, P, L, P, L, I, I, I, I, I, I, F, I, I, I, I, I, I, I, P, P, I, I, I, P, P, P, P, I, I,
                                     P, P, P, I, I, P, P],

@@ -182,12 +182,19 @@ def qkv_rotate_append(qkv: torch.Tensor, n_tokens: int, n_heads: int, n_kv_heads
                       v_interleaved: bool, token_seq: torch.Tensor, token_pos: torch.Tensor, seq_slot: torch.Tensor,
                       seq_qstart: torch.Tensor, page_table: Optional[torch.Tensor], num_pages: int,
                       k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor], write_cache: bool,
-                      status: torch.Tensor, bias: Optional[torch.Tensor] = None) -> None:
+                      status: torch.Tensor, bias: Optional[torch.Tensor] = None, qk_unit: bool = False,
+                      v_mix: Optional[torch.Tensor] = None, v_lambda: float = 0.0, v_keep: Optional[torch.Tensor] = None) -> None:
     """The general form of ``qk_norm_rope_append`` (csrc/rope_append.cu): either layout of rotated pairs, values of
     their own size that may be divided by their root mean square and rotated by their position on the way to the
-    cache.  ``qkv`` rows: q heads | k heads | v heads.  ``bias`` (float32, one per q|k|v feature) is added first."""
+    cache.  ``qkv`` rows: q heads | k heads | v heads.  ``bias`` (float32, one per q|k|v feature) is added first.
+    ``qk_unit``: q and k are divided by their root mean square over the head after the rotation.  ``v_mix`` (run dtype, ``[n,
+    n_kv_heads * v_dim]``): the values become ``(1 - v_lambda) v + v_lambda v_mix``; ``v_keep`` (the same shape) gets the values
+    that go to the cache."""
     _need(qkv.stride(-1) == 1, "qkv_rotate_append: rows of qkv must be contiguous")
     _need(bias is None or bias.numel() == (n_heads + n_kv_heads) * head_dim + n_kv_heads * v_dim, "qkv_rotate_append: bias size")
+    for t in (v_mix, v_keep):
+        _need(t is None or (t.dtype == qkv.dtype and t.is_contiguous() and t.numel() >= n_tokens * n_kv_heads * v_dim),
+              "qkv_rotate_append: v_mix and v_keep are [n, n_kv_heads * v_dim] in the run dtype")
     for t in (cos, sin, v_cos, v_sin, q_norm_w, k_norm_w, bias):
         _need(t is None or (t.dtype == torch.float32 and t.is_contiguous()), "qkv_rotate_append: float32 tables and weights")
     check(library().pe_qkv_rotate_append(
@@ -197,7 +204,8 @@ def qkv_rotate_append(qkv: torch.Tensor, n_tokens: int, n_heads: int, n_kv_heads
         v_rotary_dim if v_cos is not None else 0, 0 if v_cos is None else v_cos.shape[0], 1 if v_interleaved else 0,
         _ptr(token_seq), _ptr(token_pos), _ptr(seq_slot), _ptr(seq_qstart), _ptr(page_table),
         0 if page_table is None else page_table.shape[1], num_pages, _ptr(k_pages), _ptr(v_pages),
-        1 if write_cache else 0, _ptr(bias), _ptr(status), _stream()), "qkv_rotate_append")
+        1 if write_cache else 0, _ptr(bias), 1 if qk_unit else 0, _ptr(v_mix), float(v_lambda), _ptr(v_keep), _ptr(status),
+        _stream()), "qkv_rotate_append")
     _count(1)
 
 
@@ -292,6 +300,32 @@ def attention_mma_supported(dtype: torch.dtype, head_dim: int, n_heads: int, n_k
     return dtype == torch.bfloat16 and bool(library().pe_attention_mma_supported(head_dim, n_heads, n_kv_heads))
 
 
+def attention_mma_dims_supported(dtype: torch.dtype, head_dim: int, v_dim: int, n_heads: int, n_kv_heads: int) -> bool:
+    """Whether the tensor-core attention kernels take keys and values of these sizes (``attention_mma_gated``)."""
+    return dtype == torch.bfloat16 and bool(library().pe_attention_mma_dims_supported(head_dim, v_dim, n_heads, n_kv_heads))
+
+
+def attention_mma_gated(decode: bool, q: torch.Tensor, out: torch.Tensor, n_seqs: int, max_q: int, n_heads: int,
+                        n_kv_heads: int, head_dim: int, v_dim: int, scale: float, window: int, seq_qstart: torch.Tensor,
+                        seq_past: torch.Tensor, seq_slot: torch.Tensor, page_table: torch.Tensor, num_pages: int,
+                        k_pages: torch.Tensor, v_pages: torch.Tensor, scratch: Optional[torch.Tensor], split_keys: int,
+                        max_splits: int, status: torch.Tensor, min_range_keys: int = 0, sink: bool = False,
+                        gate: Optional[torch.Tensor] = None, keep_first: int = 0) -> None:
+    """``attention_mma`` for values of a size of their own (keys up to 256 features, values up to 128, multiples of 8; decode
+    scratch: ``attention_generic_scratch_floats(.., v_dim, ..)``), optionally with each head's output multiplied by
+    ``sigmoid(gate[token, head])`` (``gate``: bfloat16 rows, ``[n, n_heads]``, rows may be strided)."""
+    _need(q.stride(-1) == 1 and out.stride(-1) == 1, "attention: rows must be contiguous")
+    _need(q.dtype == out.dtype == k_pages.dtype == v_pages.dtype == torch.bfloat16, "attention_mma: bfloat16 tensors only")
+    _need(gate is None or (gate.dtype == torch.bfloat16 and gate.stride(-1) == 1 and gate.shape[-1] >= n_heads), "attention_mma: gate rows")
+    check(library().pe_attention_mma_gated(
+        1 if decode else 0, _ptr(q), q.stride(0), _ptr(out), out.stride(0), n_seqs, max_q, n_heads, n_kv_heads, head_dim, v_dim,
+        float(scale), int(window), 0, int(keep_first), n_kv_heads, 0, 0, 1 if sink else 0, None, None, 0, _ptr(gate),
+        0 if gate is None else gate.stride(0), _ptr(seq_qstart), _ptr(seq_past), _ptr(seq_slot), _ptr(page_table),
+        page_table.shape[1], num_pages, _ptr(k_pages), _ptr(v_pages), _ptr(scratch), split_keys, max_splits,
+        int(min_range_keys), _ptr(status), _stream()), "attention_mma_gated")
+    _count(2 if decode else 1)
+
+
 def attention_mma(decode: bool, q: torch.Tensor, out: torch.Tensor, n_seqs: int, max_q: int, n_heads: int,
                   n_kv_heads: int, head_dim: int, scale: float, window: int, seq_qstart: torch.Tensor,
                   seq_past: torch.Tensor, seq_slot: torch.Tensor, page_table: torch.Tensor, num_pages: int,
@@ -367,6 +401,15 @@ def attention_latent(decode: bool, q: torch.Tensor, out: torch.Tensor, n_seqs: i
     _count(2 if decode else 1)
 
 
+def _glu_args(glu, n: int) -> tuple:
+    """(kind, limit, alpha, bias pointer) of a fused gate|up product's activation; ``glu`` = (kind name, limit, alpha, bias)."""
+    if glu is None:
+        return 1, 0.0, 1.0, None
+    kind, limit, alpha, bias = glu
+    _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == 2 * n), "glu: bias float32 [2 * n]")
+    return GLU_KINDS[kind], float(limit), float(alpha), _ptr(bias)
+
+
 def gemm_smallm_supported(x: torch.Tensor, weight: torch.Tensor) -> bool:
     """Whether csrc/gemm_smallm.cu takes ``x [M, K] @ weight [N, K]^T``: bfloat16, M <= 16, K % 8 == 0."""
     return (x.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16 and x.dim() == 2 and x.shape[0] <= 16
@@ -374,9 +417,10 @@ def gemm_smallm_supported(x: torch.Tensor, weight: torch.Tensor) -> bool:
             and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0)
 
 
-def gemm_smallm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, pair_offset: int = 0) -> None:
+def gemm_smallm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, pair_offset: int = 0, glu=None) -> None:
     """``out[M, N] = x @ weight^T`` (out bfloat16 or float32).  With ``pair_offset`` = I the weight holds
-    gate rows then up rows and ``out[M, I] = silu(x @ gate^T) * (x @ up^T)``."""
+    gate rows then up rows and ``out[M, I] = silu(x @ gate^T) * (x @ up^T)``, or another activation of the two with
+    ``glu`` = (kind of ``GLU_KINDS``, limit, alpha, float32 bias ``[2 * I]`` or None)."""
     _need(gemm_smallm_supported(x, weight), "gemm_smallm: needs bfloat16, M <= 16, K % 8 == 0, contiguous rows")
     _need(out.stride(-1) == 1 and out.dtype in (torch.bfloat16, torch.float32), "gemm_smallm: out bfloat16 or float32")
     m, k = x.shape
@@ -384,8 +428,8 @@ def gemm_smallm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, pair_o
     _need(weight.shape[1] == k and weight.shape[0] == (2 * n if pair_offset else n) and out.shape[0] == m,
           "gemm_smallm: shapes do not match")
     _need(pair_offset in (0, n), "gemm_smallm: pair_offset must be 0 or the output width")
-    check(library().pe_gemm_smallm(_ptr(x), x.stride(0), _ptr(weight), _ptr(out), out.stride(0), m, n, k,
-                                   1 if out.dtype == torch.float32 else 0, pair_offset, sm_count(x.device), _stream()), "gemm_smallm")
+    check(library().pe_gemm_smallm_glu(_ptr(x), x.stride(0), _ptr(weight), _ptr(out), out.stride(0), m, n, k,
+                                   1 if out.dtype == torch.float32 else 0, pair_offset, *_glu_args(glu, n), sm_count(x.device), _stream()), "gemm_smallm")
     _count(1)
 
 
@@ -431,9 +475,10 @@ def gemm_umma_supported(x: torch.Tensor, weight: torch.Tensor, pair_offset: int 
     return bool(library().pe_gemm_umma_supported(x.shape[0], n, x.shape[1], pair_offset))
 
 
-def gemm_umma(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, status: torch.Tensor, pair_offset: int = 0) -> None:
+def gemm_umma(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, status: torch.Tensor, pair_offset: int = 0, glu=None) -> None:
     """``out[M, N] = x @ weight^T`` on the tcgen05 tensor cores (out bfloat16 or float32); with
-    ``pair_offset`` = I: ``out[M, I] = silu(x @ gate^T) * (x @ up^T)`` for weight = [gate; up]."""
+    ``pair_offset`` = I: ``out[M, I] = silu(x @ gate^T) * (x @ up^T)`` for weight = [gate; up] (``glu``: as for
+    ``gemm_smallm``)."""
     _need(gemm_umma_supported(x, weight, pair_offset), "gemm_umma: needs bfloat16, K % 8 == 0, dense weight rows")
     _need(out.stride(-1) == 1 and out.dtype in (torch.bfloat16, torch.float32), "gemm_umma: out bfloat16 or float32")
     m, k = x.shape
@@ -441,8 +486,8 @@ def gemm_umma(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, status: 
     _need(weight.shape[1] == k and weight.shape[0] == (2 * n if pair_offset else n) and out.shape[0] == m,
           "gemm_umma: shapes do not match")
     _need(not pair_offset or out.dtype == torch.bfloat16, "gemm_umma: the fused gate writes bfloat16")
-    check(library().pe_gemm_umma(_ptr(x), x.stride(0), _ptr(weight), _ptr(out), out.stride(0), m, n, k,
-                                 1 if out.dtype == torch.float32 else 0, pair_offset, sm_count(x.device), _ptr(status),
+    check(library().pe_gemm_umma_glu(_ptr(x), x.stride(0), _ptr(weight), _ptr(out), out.stride(0), m, n, k,
+                                 1 if out.dtype == torch.float32 else 0, pair_offset, *_glu_args(glu, n), sm_count(x.device), _ptr(status),
                                  _stream()), "gemm_umma")
     _count(1)
 
@@ -455,7 +500,7 @@ def gemm_umma2_supported(x: torch.Tensor, weight: torch.Tensor, pair_offset: int
     return bool(library().pe_gemm_umma2_supported(x.shape[0], n, x.shape[1], pair_offset))
 
 
-def gemm_umma2(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, status: torch.Tensor, pair_offset: int = 0) -> None:
+def gemm_umma2(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, status: torch.Tensor, pair_offset: int = 0, glu=None) -> None:
     """``gemm_umma`` with two SMs per 256 x 256 output tile (csrc/gemm_umma2.cu, tcgen05 cta_group::2)."""
     _need(gemm_umma2_supported(x, weight, pair_offset), "gemm_umma2: needs bfloat16, K % 64 == 0, dense weight rows")
     _need(out.stride(-1) == 1 and out.dtype in (torch.bfloat16, torch.float32), "gemm_umma2: out bfloat16 or float32")
@@ -464,8 +509,8 @@ def gemm_umma2(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, status:
     _need(weight.shape[1] == k and weight.shape[0] == (2 * n if pair_offset else n) and out.shape[0] == m,
           "gemm_umma2: shapes do not match")
     _need(not pair_offset or out.dtype == torch.bfloat16, "gemm_umma2: the fused gate writes bfloat16")
-    check(library().pe_gemm_umma2(_ptr(x), x.stride(0), _ptr(weight), _ptr(out), out.stride(0), m, n, k,
-                                  1 if out.dtype == torch.float32 else 0, pair_offset, sm_count(x.device), _ptr(status),
+    check(library().pe_gemm_umma2_glu(_ptr(x), x.stride(0), _ptr(weight), _ptr(out), out.stride(0), m, n, k,
+                                  1 if out.dtype == torch.float32 else 0, pair_offset, *_glu_args(glu, n), sm_count(x.device), _ptr(status),
                                   _stream()), "gemm_umma2")
     _count(1)
 
@@ -521,9 +566,9 @@ def decode_ranges(slots: int, pairs: int, max_kv_len: int, split_keys: int) -> t
 
 
 def attention_mma_decode_ranges(device: torch.device, head_dim: int, n_seqs: int, n_kv_heads: int, max_kv_len: int,
-                                split_keys: int) -> tuple:
+                                split_keys: int, v_dim: Optional[int] = None) -> tuple:
     """``decode_ranges`` for csrc/attention_mma.cu on this device."""
-    slots = sm_count(device) * int(library().pe_attention_mma_decode_blocks_per_sm(head_dim))
+    slots = sm_count(device) * int(library().pe_attention_mma_decode_blocks_per_sm(head_dim, head_dim if v_dim is None else v_dim))
     return decode_ranges(slots, n_seqs * n_kv_heads, max_kv_len, split_keys)
 
 
@@ -533,6 +578,11 @@ def attention_umma_supported(dtype: torch.dtype, head_dim: int, n_heads: int, n_
 
 
 _WORK_COUNTERS = {}
+
+
+def attention_umma_dims_supported(dtype: torch.dtype, head_dim: int, v_dim: int, n_heads: int, n_kv_heads: int) -> bool:
+    """Whether the tcgen05 prefill attention takes keys and values of these sizes."""
+    return dtype == torch.bfloat16 and bool(library().pe_attention_umma_dims_supported(head_dim, v_dim, n_heads, n_kv_heads))
 
 
 def _work_counter(device: torch.device) -> torch.Tensor:
@@ -550,17 +600,20 @@ def attention_umma_prefill(q: torch.Tensor, out: torch.Tensor, n_seqs: int, max_
                            head_dim: int, scale: float, window: int, seq_qstart: torch.Tensor, seq_past: torch.Tensor,
                            seq_slot: torch.Tensor, page_table: torch.Tensor, num_pages: int, k_pages: torch.Tensor,
                            v_pages: torch.Tensor, status: torch.Tensor, sink: bool = False,
-                           out_cos: Optional[torch.Tensor] = None, out_sin: Optional[torch.Tensor] = None) -> None:
-    """Prefill attention on tcgen05 (bfloat16, head size 128, groups up to 32); ``q`` holds the step's
+                           out_cos: Optional[torch.Tensor] = None, out_sin: Optional[torch.Tensor] = None,
+                           v_dim: Optional[int] = None, gate: Optional[torch.Tensor] = None) -> None:
+    """Prefill attention on tcgen05 (bfloat16, head size 128, groups up to 32; or key and value sizes that
+    ``attention_umma_dims_supported`` takes, with ``gate`` as for ``attention_mma_gated``); ``q`` holds the step's
     query rows (the first ``n_heads * head_dim`` features of each row of the fused q|k|v buffer).  ``sink``,
     ``out_cos``, ``out_sin``: as for ``attention_mma``."""
     _need(q.stride(-1) == 1 and out.stride(-1) == 1, "attention: rows must be contiguous")
     _need(q.dtype == out.dtype == k_pages.dtype == torch.bfloat16, "attention_umma: bfloat16 tensors only")
     _check_out_tables(out_cos, out_sin, head_dim)
-    check(library().pe_attention_umma_prefill_ex(
+    _need(gate is None or (gate.dtype == torch.bfloat16 and gate.stride(-1) == 1 and gate.shape[-1] >= n_heads), "attention_umma: gate rows")
+    check(library().pe_attention_umma_prefill_gated(
         _ptr(q), q.stride(0), q.shape[0], _ptr(out), out.stride(0), n_seqs, max_q, n_heads, n_kv_heads, head_dim,
-        float(scale), int(window), 1 if sink else 0, _ptr(out_cos), _ptr(out_sin),
-        0 if out_cos is None else out_cos.shape[0], _ptr(seq_qstart), _ptr(seq_past), _ptr(seq_slot), _ptr(page_table),
+        head_dim if v_dim is None else int(v_dim), float(scale), int(window), 1 if sink else 0, _ptr(out_cos), _ptr(out_sin),
+        0 if out_cos is None else out_cos.shape[0], _ptr(gate), 0 if gate is None else gate.stride(0), _ptr(seq_qstart), _ptr(seq_past), _ptr(seq_slot), _ptr(page_table),
         page_table.shape[1], num_pages, _ptr(k_pages), _ptr(v_pages), sm_count(q.device), _ptr(_work_counter(q.device)), _ptr(status), _stream()),
         "attention_umma_prefill")
     _count(1)
@@ -772,12 +825,14 @@ def moe_combine(rows: torch.Tensor, x: torch.Tensor, shared: Optional[torch.Tens
     _count(1)
 
 
-def glu_act(gate_up: torch.Tensor, out: torch.Tensor, kind: str, limit: float = 0.0, alpha: float = 1.0) -> None:
+def glu_act(gate_up: torch.Tensor, out: torch.Tensor, kind: str, limit: float = 0.0, alpha: float = 1.0,
+            bias: Optional[torch.Tensor] = None) -> None:
     """``out = act(gate, up)`` over the halves of ``gate_up [N, 2 * I]``: "silu", "relu", or "clamped_swish"
-    (``g' sigmoid(alpha g') (u' + 1)`` with ``g' = min(g, limit)``, ``u' = clamp(u, -limit, limit)``)."""
+    (``g' sigmoid(alpha g') (u' + 1)`` with ``g' = min(g, limit)``, ``u' = clamp(u, -limit, limit)``); ``bias`` (float32 ``[2 * I]``) is added first."""
+    _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == gate_up.shape[1]), "glu_act: bias")
     _need(gate_up.is_contiguous() and out.is_contiguous() and gate_up.shape[1] == 2 * out.shape[1], "glu_act: shapes")
     check(library().pe_glu_act(dtype_tag(gate_up.dtype), _ptr(gate_up), _ptr(out), out.shape[0], out.shape[1], GLU_KINDS[kind],
-                               float(limit), float(alpha), _stream()), "glu_act")
+                               float(limit), float(alpha), _ptr(bias), _stream()), "glu_act")
     _count(1)
 
 
@@ -1052,4 +1107,44 @@ def rmsnorm_pair_mix_dyt_add(a: torch.Tensor, b: torch.Tensor, wa: torch.Tensor,
     check(library().pe_rmsnorm_pair_mix_dyt_add(dtype_tag(a.dtype), _ptr(a), _ptr(b), _ptr(wa), _ptr(wb), float(eps), float(sa),
                                                 float(sb), _ptr(stream), _ptr(w1), _ptr(b1), float(a1), _ptr(w2), _ptr(b2), float(a2),
                                                 _ptr(out), n, dim, _stream()), "rmsnorm_pair_mix_dyt_add")
+    _count(1)
+
+
+# ---- residual streams side by side, layer norm -----------------------------------------------------------------------
+STREAM_NORMS = {None: 0, "layer": 1, "rms": 2}
+MAX_STREAMS = 32
+
+
+def stream_mix(single: Optional[torch.Tensor], x: Optional[torch.Tensor], y: Optional[torch.Tensor], bias: Optional[torch.Tensor],
+               mix: Optional[torch.Tensor], write: Optional[torch.Tensor], read: torch.Tensor, norm: Optional[str],
+               weight: Optional[torch.Tensor], eps: float, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+    """Streams ``x [n, s, width]`` (float32): ``x_t <- sum_i mix[i, t] x_i + write[t] (y + bias)`` if ``y`` is given, then ``out =
+    norm(sum_i read[i] x_i)`` (csrc/streams.cu).  ``single [n, width]``: the streams are all equal to it and do not exist yet.
+    ``norm``: "layer", "rms" (times ``weight``; ``out`` in ``y``'s dtype) or None (``out`` float32).  ``rows`` (int32): output row
+    r is stream row rows[r], and nothing is written back."""
+    s = read.numel()
+    base = single if single is not None else x
+    width = base.shape[-1]
+    for t in (single, x, bias, mix, write, read, weight):
+        _need(t is None or (t.dtype == torch.float32 and t.is_contiguous()), "stream_mix: streams, coefficients and weights float32")
+    _need(x is None or x.numel() == base.shape[0] * s * width, "stream_mix: x is [n, s, width]")
+    _need(y is None or (y.is_contiguous() and y.shape == (base.shape[0], width) and mix.numel() == s * s and write.numel() == s),
+          "stream_mix: y [n, width], mix [s, s], write [s]")
+    _need(out.is_contiguous() and out.shape[-1] == width and out.shape[0] == (base.shape[0] if rows is None else rows.numel()), "stream_mix: out")
+    _need(norm is not None or out.dtype == torch.float32, "stream_mix: without a norm out is float32")
+    _need(norm is None or y is None or y.dtype == out.dtype, "stream_mix: y and out share a dtype")
+    _need(rows is None or rows.dtype == torch.int32, "stream_mix: rows int32")
+    dtype = y.dtype if y is not None else out.dtype
+    check(library().pe_stream_mix(dtype_tag(dtype), _ptr(single), _ptr(x), _ptr(y), _ptr(bias), _ptr(mix), _ptr(write), _ptr(read),
+                                  STREAM_NORMS[norm], _ptr(weight), float(eps), _ptr(out), _ptr(rows), out.shape[0], s, width,
+                                  _stream()), "stream_mix")
+    _count(1)
+
+
+def layernorm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float) -> None:
+    """``(x - mean) / sqrt(mean of squared deviations + eps) * weight`` over the last dimension."""
+    _need(x.is_contiguous() and out.is_contiguous() and x.dtype == out.dtype and weight.dtype == torch.float32, "layernorm: contiguous, weight f32")
+    dim = x.shape[-1]
+    check(library().pe_layernorm(dtype_tag(x.dtype), _ptr(x), _ptr(weight), _ptr(out), x.numel() // dim, dim, float(eps), _stream()),
+          "layernorm")
     _count(1)

@@ -60,7 +60,11 @@ class GQAttention:
         if params.get("bias", False):
             decls.update({"q_bias": WeightDecl((nh * d,)), "k_bias": WeightDecl((nkv * d,)), "v_bias": WeightDecl((nkv * dv,))})
         if params.get("output_gate"):
-            decls["g_proj"] = WeightDecl((nh * dv, h))
+            decls["g_proj"] = WeightDecl((nh if params["output_gate"] == "sigmoid_head" else nh * dv, h))
+        if params.get("value_mix") == "mix":
+            decls["v_lambda"] = WeightDecl((), "unit")
+        if params.get("out_bias", False):
+            decls["o_bias"] = WeightDecl((h,))
         return decls
 
     @classmethod
@@ -94,8 +98,18 @@ class GQAttention:
         if self.keep_first and (self.sink or params.get("value_position") is not None):
             raise ValueError("keep_first is not built together with a sink or turned values")
         self.output_gate = params.get("output_gate")
-        if self.output_gate not in (None, "sigmoid"):
-            raise ValueError(f"output_gate {self.output_gate!r} is not built (None or 'sigmoid')")
+        if self.output_gate not in (None, "sigmoid", "sigmoid_head"):
+            raise ValueError(f"output_gate {self.output_gate!r} is not built (None, 'sigmoid' or 'sigmoid_head')")
+        self.qk_unit = bool(params.get("qk_unit", False))
+        self.value_mix = params.get("value_mix")
+        if self.value_mix not in (None, "keep", "mix"):
+            raise ValueError(f"value_mix {self.value_mix!r} is not built (None, 'keep' or 'mix')")
+        if self.value_mix == "mix" and self.v_norm:
+            raise ValueError("value_mix is not built together with a norm on the values")
+        # a single number, read once when the model is built
+        self.v_lambda = float(weights["v_lambda"].to(torch.float32).reshape(-1)[0].item()) if self.value_mix == "mix" else 0.0
+        self.out_bias = runtime.adopt(weights["o_bias"], torch.float32) if params.get("out_bias", False) else None
+        self.out_bias_deferred = False
         self.bias = None
         if params.get("bias", False):
             self.bias = torch.cat([weights[n].to(device=runtime.device, dtype=torch.float32).reshape(-1)
@@ -103,6 +117,10 @@ class GQAttention:
         fused = [weights["q_proj"], weights["k_proj"], weights["v_proj"]]
         if self.output_gate:
             fused.append(weights["g_proj"])       # q | k | v | gate: one product over the mixer's input
+        if self.output_gate == "sigmoid_head":    # rows of the product stay 16-byte aligned
+            rows = sum(t.shape[0] for t in fused)
+            if rows % 8:
+                fused.append(torch.zeros((8 - rows % 8, self.hidden), dtype=fused[0].dtype, device=fused[0].device))
         self.qkv = fuse_rows(runtime, fused)
         self.o_proj = runtime.adopt(weights["o_proj"])
         self.q_norm = self.k_norm = None
@@ -130,13 +148,14 @@ class GQAttention:
         interleaved = self.fused_position and getattr(self.position, "interleaved", False)
         # what the kernels of the plain softmax attention do not do
         self.general = bool(self.sink or self.v_norm or self.value_position is not None or self.v_dim != self.head_dim
-                            or interleaved or self.bias is not None or self.keep_first or self.output_gate)
+                            or interleaved or self.bias is not None or self.keep_first or self.output_gate or self.qk_unit
+                            or self.value_mix or self.out_bias is not None)
         if self.general and self.position is not None and not self.fused_position:
             raise ValueError("the general attention path takes a rotary position encoding with tables(), or none")
         self.qkv_dim = (self.n_heads + self.n_kv_heads) * self.head_dim + self.n_kv_heads * self.v_dim
         self.gate_col = self.qkv_dim               # the gate's columns follow q | k | v in the fused product
         if self.output_gate:
-            self.qkv_dim += self.n_heads * self.v_dim
+            self.qkv_dim = int(self.qkv.shape[0])
         # tensor-core kernels where they take the shape (bfloat16, head size 64 or 128, group <= 16);
         # the generic float32-arithmetic kernels otherwise
         # (with a sink or turned values too, if keys and values have one size and the values turn in interleaved pairs
@@ -149,6 +168,11 @@ class GQAttention:
         # prefill on tcgen05 where that kernel takes the shape (bfloat16, head size 128, groups up to 32)
         self.use_umma_prefill = (fast_ok and runtime.is_cuda and not self.keep_first
                                  and ops.attention_umma_supported(runtime.dtype, self.head_dim, self.n_heads, self.n_kv_heads))
+        # sizes that run in padded tiles, and a gate per head (no turned values)
+        if self.general and vp is None and runtime.is_cuda:
+            dims = (runtime.dtype, self.head_dim, self.v_dim, self.n_heads, self.n_kv_heads)
+            self.use_mma = ops.attention_mma_dims_supported(*dims)
+            self.use_umma_prefill = not self.keep_first and ops.attention_umma_dims_supported(*dims)
         self.generic_attention = bool(getattr(runtime, "generic_attention", False))   # comparisons: the general kernels only
 
     def forward(self, x: torch.Tensor, ctx, view, writes_cache: bool = True) -> torch.Tensor:
@@ -162,12 +186,14 @@ class GQAttention:
             self.rotate_append_general(qkv, n, ctx, view, writes_cache)
             out = ctx.buffer("attn.out", (n, self.n_heads * self.v_dim), rt.dtype)
             self.attend_general(qkv, out, ctx, view)
-            if self.output_gate:
+            if self.output_gate == "sigmoid" or (self.output_gate and not self.gate_in_kernel(ctx)):
                 gated = ctx.buffer("attn.gated", (n, self.n_heads * self.v_dim), rt.dtype)
-                ops.sigmoid_gate(out.view(n, self.n_heads, self.v_dim).transpose(0, 1), qkv[:, self.gate_col:], gated)
+                ops.sigmoid_gate(out.view(n, self.n_heads, self.v_dim).transpose(0, 1), self.gate_columns(qkv), gated)
                 out = gated
             delta = ctx.buffer("attn.delta", (n, self.hidden), rt.dtype)
             rt.linear(out, self.o_proj, out=delta)
+            if self.out_bias is not None and not self.out_bias_deferred:
+                delta.add_(self.out_bias)
             return delta
         if self.fuses_rope_into_product(x, rt):
             # many rows: q/k-norm, rotation and the cache append ride in the epilogue of the q|k|v product (its
@@ -187,6 +213,12 @@ class GQAttention:
         rt.linear(out, self.o_proj, out=delta)
         return delta
 
+    def defer_out_bias(self) -> Optional[torch.Tensor]:
+        """For an arrangement that adds the output projection's bias itself: the bias (float32, or None), which ``forward`` then
+        leaves out."""
+        self.out_bias_deferred = True
+        return self.out_bias
+
     # ---- the general path ---------------------------------------------------------------------------------
     def rotate_append_general(self, qkv: torch.Tensor, n: int, ctx, view, writes_cache: bool) -> None:
         """q/k-norm, rotation of q and k, the values' norm and rotation, and the append, in one kernel."""
@@ -199,10 +231,25 @@ class GQAttention:
         if self.value_position is not None:
             vcos, vsin, vrot = self.value_position.tables()
             vinter = bool(getattr(self.value_position, "interleaved", False))
+        kept = None
+        if self.value_mix:
+            kept = ctx.buffer("attn.kept_values", (n, self.n_kv_heads * self.v_dim), self.runtime.dtype)
         ops.qkv_rotate_append(qkv, n, self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim, self.q_norm, self.k_norm,
                               self.eps, cos, sin, rot, inter, self.v_norm == "unit", vcos, vsin, vrot, vinter,
                               ctx.token_seq, ctx.token_pos, ctx.seq_slot, ctx.seq_qstart, view.page_table, view.num_pages,
-                              view.k_pages, view.v_pages, writes_cache, self.runtime.status, self.bias)
+                              view.k_pages, view.v_pages, writes_cache, self.runtime.status, self.bias, qk_unit=self.qk_unit,
+                              v_mix=kept if self.value_mix == "mix" else None, v_lambda=self.v_lambda,
+                              v_keep=kept if self.value_mix == "keep" else None)
+
+    def gate_columns(self, qkv: torch.Tensor) -> torch.Tensor:
+        width = self.n_heads if self.output_gate == "sigmoid_head" else self.n_heads * self.v_dim
+        return qkv[:, self.gate_col:self.gate_col + width]
+
+    def gate_in_kernel(self, ctx) -> bool:
+        """Whether the step's attention kernel multiplies the heads' gates in (the general kernels leave it to one behind)."""
+        if self.output_gate != "sigmoid_head" or self.generic_attention:
+            return False
+        return self.use_mma or (self.use_umma_prefill and not ctx.decode)
 
     def attend_general(self, q: torch.Tensor, out: torch.Tensor, ctx, view) -> None:
         vcos = vsin = None
@@ -213,23 +260,25 @@ class GQAttention:
             vinter = bool(getattr(self.value_position, "interleaved", False))
         where = (ctx.seq_qstart, ctx.seq_past, ctx.seq_slot, view.page_table, view.num_pages, view.k_pages, view.v_pages)
         extra = dict(sink=self.sink, out_cos=vcos, out_sin=vsin)
+        gate = self.gate_columns(q) if self.gate_in_kernel(ctx) else None
         if self.use_umma_prefill and not ctx.decode and not self.generic_attention:
             ops.attention_umma_prefill(q, out, ctx.n_seqs, ctx.max_q, self.n_heads, self.n_kv_heads, self.head_dim, self.scale,
-                                       self.window, *where, self.runtime.status, **extra)
+                                       self.window, *where, self.runtime.status, v_dim=self.v_dim, gate=gate, **extra)
             return
         if self.use_mma and not self.generic_attention:
             scratch = None
             split_keys, max_splits, floor = SPLIT_KEYS, 0, 0
             if ctx.decode:
                 split_keys, max_splits, floor = ops.attention_mma_decode_ranges(
-                    q.device, self.head_dim, ctx.n_seqs, self.n_kv_heads, ctx.max_kv_len, SPLIT_KEYS)
+                    q.device, self.head_dim, ctx.n_seqs, self.n_kv_heads, ctx.max_kv_len, SPLIT_KEYS, v_dim=self.v_dim)
                 scratch = ctx.buffer(
                     "attn.scratch",
-                    (ops.attention_generic_scratch_floats(ctx.n_seqs, self.n_heads, self.head_dim, max_splits),), torch.float32)
-            if self.keep_first:        # (not with a sink or turned values: the constructor refuses that pair)
-                ops.attention_mma_masked(ctx.decode, q, out, ctx.n_seqs, ctx.max_q, self.n_heads, self.n_kv_heads, self.head_dim,
-                                         self.scale, *where, scratch, split_keys, max_splits, self.runtime.status,
-                                         min_range_keys=floor, window=self.window, keep_first=self.keep_first)
+                    (ops.attention_generic_scratch_floats(ctx.n_seqs, self.n_heads, self.v_dim, max_splits),), torch.float32)
+            if self.value_position is None:
+                ops.attention_mma_gated(ctx.decode, q, out, ctx.n_seqs, ctx.max_q, self.n_heads, self.n_kv_heads, self.head_dim,
+                                        self.v_dim, self.scale, self.window, *where, scratch, split_keys, max_splits,
+                                        self.runtime.status, min_range_keys=floor, sink=self.sink, gate=gate,
+                                        keep_first=self.keep_first)
                 return
             ops.attention_mma(ctx.decode, q, out, ctx.n_seqs, ctx.max_q, self.n_heads, self.n_kv_heads, self.head_dim,
                               self.scale, self.window, *where, scratch, split_keys, max_splits, self.runtime.status,

@@ -37,11 +37,46 @@ class NormedDelta:
         self.norm.add_after(stream, self.delta, None)
 
 
+class StreamsDelta:
+    """A sublayer output that is still to be written back into several residual streams: what a block of the ``streams``
+    arrangement hands on.  ``single`` is the row that all streams are equal to while they do not exist yet (else None)."""
+
+    def __init__(self, streams: torch.Tensor, single: Optional[torch.Tensor], delta: torch.Tensor, bias: Optional[torch.Tensor],
+                 bundle, ones: torch.Tensor, stream: torch.Tensor) -> None:
+        self.streams, self.single, self.delta, self.bias, self.bundle = streams, single, delta, bias, bundle
+        self.ones = ones          # reads the sum of the streams
+        self.stream = stream
+
+    def write_and_read(self, read: torch.Tensor, norm, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+        """Write the output back, then ``out = norm(sum_i read[i] X_i)``, in one pass where the norm is one that the kernel
+        knows.  ``rows``: only those rows, and the streams are left as they are."""
+        b = self.bundle
+        args = (self.single, self.streams, self.delta, self.bias, b.mix, b.write, read)
+        if norm is None or getattr(norm, "stream_norm", None):
+            kind, w, eps = (None, None, 0.0) if norm is None else (norm.stream_norm, norm.weight, norm.eps)
+            ops.stream_mix(*args, kind, w, eps, out, rows)
+            return
+        ops.stream_mix(*args, None, None, 0.0, self.stream)
+        norm.add_forward(self.stream, None, out, rows)
+
+    def finish(self, norm, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+        """The norm of the sum of the streams (the model's last norm, or the first norm of a block of another arrangement)."""
+        if rows is None:
+            self.settle(self.stream)
+            norm.add_forward(self.stream, None, out)
+        else:
+            self.write_and_read(self.ones, norm, out, rows)
+
+    def settle(self, stream: torch.Tensor) -> None:
+        """``stream`` becomes the sum of the streams."""
+        self.write_and_read(self.ones, None, stream)
+
+
 def settle_pending(stream: torch.Tensor, pending) -> None:
     """Add what the block before left to be added (nothing, one delta, several scaled ones, one behind a norm)."""
     if pending is None:
         return
-    if isinstance(pending, NormedDelta):
+    if hasattr(pending, "settle"):
         pending.settle(stream)
     elif isinstance(pending, DeltaSum):
         pending.add_into(stream, stream)
@@ -302,3 +337,58 @@ class SandwichBlock:
     def fuses(post_norm, next_norm) -> bool:
         import inspect
         return type(post_norm) is type(next_norm) and "then" in inspect.signature(post_norm.add_after).parameters
+
+
+@register("arrangement", "streams")
+class StreamsBlock:
+    """Several residual streams side by side instead of one (all equal to the stream where the first such block begins; their
+    sum is the stream where another arrangement or the model's last norm follows).  For each sublayer with its numbers
+    ``read``, ``mix``, ``write``:
+
+        y = sublayer(norm(sum_i read[i] X_i)) ;   X_t <- sum_i mix[i, t] X_i + write[t] y      (all t from the old X)
+
+    Parts by name: ``mixer_norm, mixer, mixer_streams`` and optionally ``ffn_norm, ffn, ffn_streams`` (``*_streams``: kind
+    ``stream_bundle``).  A sublayer's output is written back in the pass that reads the next sublayer's input and norms it,
+    across blocks too: the block hands its last output on as a ``StreamsDelta``.  A bias of a sublayer's output projection
+    is added in that pass."""
+
+    graph_safe = True  # launches only; nothing in forward() waits for the device
+
+    def __init__(self, spec, parts, runtime) -> None:
+        self.runtime = runtime
+        self.name = spec.name
+        self.steps = [(parts["mixer_norm"], parts["mixer"], parts["mixer_streams"], True)]
+        if "ffn" in parts:
+            self.steps.append((parts["ffn_norm"], parts["ffn"], parts["ffn_streams"], False))
+        self.biases = [part.defer_out_bias() if hasattr(part, "defer_out_bias") else None for _, part, _, _ in self.steps]
+        self.ones = torch.ones(self.steps[0][2].streams, dtype=torch.float32, device=runtime.device)
+
+    def forward(self, stream: torch.Tensor, pending, ctx, view, writes_cache: bool = True):
+        rt = self.runtime
+        n, hidden = stream.shape
+        s = self.ones.numel()
+        if pending is not None and not (isinstance(pending, StreamsDelta) and pending.bundle.streams == s):
+            settle_pending(stream, pending)
+            pending = None
+        streams = ctx.buffer("streams.rows", (n, s, hidden), torch.float32)
+        normed = ctx.buffer("block.normed", (n, hidden), rt.dtype)
+        for (norm, part, bundle, is_mixer), bias in zip(self.steps, self.biases):
+            single = None
+            if pending is not None:
+                pending.write_and_read(bundle.read, norm, normed)
+            else:
+                single = stream          # the streams do not exist yet: all of them are this row
+                if getattr(norm, "stream_norm", None):
+                    ops.stream_mix(single, None, None, None, None, None, bundle.read, norm.stream_norm, norm.weight, norm.eps, normed)
+                else:
+                    work = ctx.buffer("streams.read", (n, hidden), torch.float32)
+                    ops.stream_mix(single, None, None, None, None, None, bundle.read, None, None, 0.0, work)
+                    norm.add_forward(work, None, normed)
+            if is_mixer:
+                mview = view["mixer"] if isinstance(view, dict) else view
+                delta = part.forward(normed, ctx, mview) if writes_cache else part.forward(normed, ctx, mview, writes_cache=False)
+            else:
+                delta = part.forward(normed, ctx)
+            pending = StreamsDelta(streams, single, delta, bias, bundle, self.ones, stream)
+        ctx.stream_copy = None
+        return pending

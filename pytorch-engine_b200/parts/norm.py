@@ -1,4 +1,4 @@
-"""RMSNorm and Dynamic Tanh.  RMSNorm's formula: ``x * rsqrt(mean(x^2) + eps) * w`` in float32
+"""RMSNorm, layer norm and Dynamic Tanh.  RMSNorm's formula: ``x * rsqrt(mean(x^2) + eps) * w`` in float32
 (pygguf_engine/quant_kernels.py:831-833, 1548; fused with the residual add 1595-1596)."""
 from __future__ import annotations
 
@@ -17,6 +17,7 @@ class RMSNorm:
     ``offset + weight``; random weights then lie around zero).  weights: ``weight [dim]`` (kept in float32)."""
 
     graph_safe = True  # launches only; nothing in forward() waits for the device
+    stream_norm = "rms"     # the kernel over several streams (csrc/streams.cu) can end in this norm
 
     @classmethod
     def weight_decls(cls, params) -> Dict[str, WeightDecl]:
@@ -32,6 +33,9 @@ class RMSNorm:
 
     def add_forward(self, residual: torch.Tensor, delta: Optional[torch.Tensor], out: torch.Tensor,
                     rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if hasattr(delta, "finish"):      # several streams whose sum is the stream
+            delta.finish(self, out, rows)
+            return out
         if hasattr(delta, "settle"):      # an output that goes through a norm of its own before it is added
             delta.settle(residual)
             delta = None
@@ -49,6 +53,45 @@ class RMSNorm:
     def add_after(self, stream: torch.Tensor, delta: torch.Tensor, cast: Optional[torch.Tensor] = None) -> None:
         """The norm on what is added: ``stream += rmsnorm(delta) * w``; ``cast`` gets the new rows in the run dtype."""
         ops.rmsnorm_add(stream, delta, self.weight, self.eps, cast)
+
+
+@register("norm", "layer_norm")
+class LayerNorm:
+    """``(x - mean) / sqrt(mean((x - mean)^2) + eps) * weight``, no bias, in float32 (csrc/streams.cu).  params: ``dim``,
+    ``eps``.  weights: ``weight [dim]``."""
+
+    graph_safe = True  # launches only; nothing in forward() waits for the device
+    stream_norm = "layer"
+
+    @classmethod
+    def weight_decls(cls, params) -> Dict[str, WeightDecl]:
+        return {"weight": WeightDecl((int(params["dim"]),), "norm")}
+
+    def __init__(self, params, weights, runtime) -> None:
+        self.dim = int(params["dim"])
+        self.eps = float(params["eps"])
+        self.runtime = runtime
+        self.weight = runtime.adopt(weights["weight"], torch.float32)
+        self.one = torch.ones(1, dtype=torch.float32, device=runtime.device)
+
+    def add_forward(self, residual: torch.Tensor, delta, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if hasattr(delta, "finish"):      # several streams whose sum is the stream
+            delta.finish(self, out, rows)
+            return out
+        if hasattr(delta, "settle"):
+            delta.settle(residual)
+            delta = None
+        elif hasattr(delta, "deltas"):
+            delta.add_into(residual, self.weight)
+            delta = None
+        one = self.one                    # the usual residual add is the case of one stream
+        ops.stream_mix(None, residual, delta, None, one, one, one, "layer", self.weight, self.eps, out, rows)
+        return out
+
+    def forward(self, x: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        out = torch.empty_like(x) if out is None else out
+        ops.layernorm(x, self.weight, out, self.eps)
+        return out
 
 
 @register("norm", "dynamic_tanh")
@@ -74,7 +117,7 @@ class DynamicTanh:
     def add_forward(self, residual: torch.Tensor, delta, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         if delta is not None:
             if hasattr(delta, "settle"):
-                if rows is None and type(delta.norm) is type(self):
+                if rows is None and type(getattr(delta, "norm", None)) is type(self):
                     delta.norm.add_after(residual, delta.delta, out, then=self)     # its norm, the add and this norm in one pass
                     return out
                 delta.settle(residual)

@@ -1,11 +1,13 @@
 """Rotary position encoding with precomputed float32 cos/sin tables, in either layout of pairs (split-half "neox":
-feature j with j + rotary_dim/2; "interleaved": 2j with 2j + 1), optionally with YaRN-scaled frequencies.
+feature j with j + rotary_dim/2; "interleaved": 2j with 2j + 1), optionally with frequencies scaled linearly or by YaRN.
 
 Formulas: ``inv_freq_j = 1 / theta^(2j / rotary_dim)`` (pygguf_engine/model.py:147-156),
 ``angle = position * inv_freq`` with float32 positions, then cos and sin (183-185); rotation of the
 first ``rotary_dim`` features ``[x1*cos - x2*sin, x2*cos + x1*sin]``, the rest passing through
 (232-251).  ``inv_freq`` is computed on the host so that it is bit-identical everywhere; the
 product and cos/sin are taken on the device in float32.
+
+Linear scaling (``scaling`` with ``factor`` alone): every frequency is divided by the factor.
 
 YaRN (``scaling`` = factor, original, fast, slow): with ``turn(t) = rotary_dim * ln(original / (2 pi t)) / (2 ln theta)``
 the pair index at which a pair makes ``t`` turns over ``original`` positions, ``lo = max(floor(turn(fast)), 0)``,
@@ -27,7 +29,7 @@ from .spec import WeightDecl
 @register("position", "rope")
 class RotaryPosition:
     """params: ``rotary_dim`` (even, <= head size), ``theta``, ``max_positions``, ``style`` ("neox" or
-    "interleaved"), ``scaling`` (None, or a mapping with factor, original, fast, slow), ``exact`` (true: the tables are
+    "interleaved"), ``scaling`` (None, a mapping with factor, original, fast, slow, or one with factor alone), ``exact`` (true: the tables are
     computed in float64 and rounded once; otherwise the angle is a float32 product, as the reference has it).  The tables hold
     ``max_positions`` rows, or as many as the engine can hold in one sequence if that is fewer
     (``runtime.position_limit``)."""
@@ -55,16 +57,19 @@ class RotaryPosition:
             raise ValueError(f"rotary_dim must be positive and even, got {self.rotary_dim}")
         scaling = params.get("scaling")
         mult = 1.0
+        linear = 1.0
+        if scaling and "original" not in scaling:
+            linear, scaling = float(scaling["factor"]), None
         if params.get("exact") and not scaling:
             # frequencies, angles, cos and sin in float64 on the host, each table entry rounded once to float32
             idx = torch.arange(0, self.rotary_dim, 2, dtype=torch.float64)
-            ang = torch.outer(torch.arange(0, self.max_positions, dtype=torch.float64), self.theta ** (-idx / self.rotary_dim))
+            ang = torch.outer(torch.arange(0, self.max_positions, dtype=torch.float64), self.theta ** (-idx / self.rotary_dim) / linear)
             self.cos = torch.cos(ang).to(torch.float32).to(runtime.device).contiguous()
             self.sin = torch.sin(ang).to(torch.float32).to(runtime.device).contiguous()
             return
         if not scaling:
             idx = torch.arange(0, self.rotary_dim, 2, dtype=torch.float32)
-            inv_freq = (1.0 / (self.theta ** (idx / self.rotary_dim))).to(runtime.device)
+            inv_freq = (1.0 / (self.theta ** (idx / self.rotary_dim)) / linear).to(runtime.device)
         else:
             inv_freq, mult = yarn_frequencies(self.rotary_dim, self.theta, scaling)
             inv_freq = inv_freq.to(runtime.device)

@@ -125,7 +125,7 @@ class WeightDecl:
     """What a part expects of one of its weights: shape, and the ``role`` that decides how a
     random model fills it and what the part converts it to (``matrix``/``embedding``: normal
     with the given std, run dtype; ``norm``: one plus normal, float32; ``table_int``: int32;
-    ``unit``: uniform in (0, 1), a mixing coefficient).  ``any_dims`` lists the dimensions whose size the
+    ``unit``: uniform in (0, 1), a mixing coefficient; ``near_identity``: the identity plus normal).  ``any_dims`` lists the dimensions whose size the
     checkpoint decides (a projection's rank that no configuration key names): the loader accepts any size
     there, ``shape`` holds the size that random weights get, and the part reads the tensor's own shape."""
 

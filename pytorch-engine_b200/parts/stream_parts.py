@@ -17,6 +17,9 @@ with the results kept for the length of a step in one float32 buffer.
 ``input_mix``: the stream is replaced by a learned mix of itself and the embedding's output, ``x <- W [x ; x0]`` (a block that
 runs several times over takes the model's input in again in front of every pass).
 
+``stream_bundle``: how a sublayer reads several residual streams and writes its output back into them (learned numbers per
+stream and per pair of streams; the ``streams`` arrangement of ``parts/block.py`` runs it fused with the norms).
+
 ``normed_mean``: two sublayer outputs side by side become one, ``(unit(a) * w_a + unit(b) * w_b) / 2``, each divided by its own
 root mean square over the row first.
 """
@@ -149,3 +152,25 @@ class NormedMean:
         nxt = None if then is None or out is None else (then.weight, then.bias, then.alpha)
         ops.rmsnorm_pair_mix_dyt_add(a, b, self.weight_a, self.weight_b, self.eps, self.scale, self.scale, stream,
                                      (post.weight, post.bias, post.alpha), nxt, out if nxt else None)
+
+
+@register("stream", "stream_bundle")
+class StreamBundle:
+    """``u = sum_i read[i] X_i`` and ``X_t <- sum_i mix[i, t] X_i + write[t] y`` over ``streams`` residual streams
+    (csrc/streams.cu).  params: ``streams``.  weights: ``read [s]``, ``mix [s, s]`` (from, to), ``write [s]``."""
+
+    graph_safe = True  # launches only; nothing in forward() waits for the device
+
+    @classmethod
+    def weight_decls(cls, params) -> Dict[str, WeightDecl]:
+        s = int(params["streams"])
+        return {"read": WeightDecl((s,), "unit"), "mix": WeightDecl((s, s), "near_identity"), "write": WeightDecl((s,), "unit")}
+
+    def __init__(self, params, weights, runtime) -> None:
+        self.runtime = runtime
+        self.streams = int(params["streams"])
+        if self.streams > ops.MAX_STREAMS:
+            raise ValueError(f"{self.streams} residual streams are more than the kernel takes ({ops.MAX_STREAMS})")
+        self.read = runtime.adopt(weights["read"], torch.float32)
+        self.mix = runtime.adopt(weights["mix"], torch.float32)
+        self.write = runtime.adopt(weights["write"], torch.float32)

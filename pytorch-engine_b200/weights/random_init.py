@@ -49,6 +49,8 @@ def random_weights(plan: ModelPlan, seed: int, device="cpu", norm_dtype: torch.d
         x = torch.randn(decl.shape, generator=gen, device=device, dtype=torch.float32) * WEIGHT_STD
         if decl.role == "unit":
             out[name] = torch.rand(decl.shape, generator=gen, device=device, dtype=torch.float32).to(torch.bfloat16)
+        elif decl.role == "near_identity":
+            out[name] = (torch.eye(decl.shape[0], decl.shape[1], device=device) + x).to(torch.bfloat16)
         elif decl.role == "norm":
             out[name] = (1.0 + x).to(torch.bfloat16).to(norm_dtype)
         else:
