@@ -1,6 +1,6 @@
-"""``python bench.py --archs``: the Vabelorn, Lunadra and Vemepel architectures beside the Qwen3 dense decoder at equal layer
-sizes (``--arch-names`` picks among them; Lunadra's own kernels stand beside the like kernels of the Vabelorn path, Vemepel's
-beside those of the Qwen3 path).
+"""``python bench.py --archs``: the Vabelorn, Lunadra, Vemepel, Zonevik and Bobasun architectures beside the Qwen3 dense decoder
+at equal layer sizes (``--arch-names`` picks among them; Lunadra's own kernels stand beside the like kernels of the Vabelorn
+path, Zonevik's beside those of the Lunadra path, Vemepel's and Bobasun's beside those of the Qwen3 path).
 
 Random weights, bfloat16, one B200.  For each size: tokens/s of a 2,048-token prompt and of decode steps at batch 8
 (context 2,048) through ``ModelRunner.step``, for both architectures; then the kernels that only the new
@@ -747,6 +747,133 @@ def zonevik_kernel_pairs(pe, torch, s, peaks, prompt, batch, context):
     return out
 
 
+def bobasun_config(pe, s):
+    """Bobasun at the same width, attention heads, feed-forward and vocabulary: four residual streams, every layer mixes its
+    values with the first one's, rotation over the whole head with halved frequencies."""
+    layer = {"type": "attention",
+             "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": 1.0 / math.sqrt(s["dim"]),
+                       "v_mix": True, "rot": {"base": 1e6, "dims": s["dim"], "scaling": {"factor": 2.0}}},
+             "mlp": {"kind": "dense", "ff": s["ff"], "limit": 7.0}}
+    return pe.BobasunConfig.from_dict({"architecture": "Bobasun", "vocab": s["vocab"], "width": s["width"], "streams": 4,
+                                       "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "layers": [layer] * s["layers"]})
+
+
+def bobasun_kernel_pairs(pe, torch, s, peaks, prompt, batch, context):
+    """The kernels that Bobasun runs in place of the Qwen3 path's (the closest model: a dense softmax-attention decoder), each
+    beside the like kernel at the same shape, warm: bytes over the copy bandwidth or operations over the matrix products' rate,
+    whichever takes longer, is the roofline time."""
+    ops = pe.kernels.ops
+    dev = torch.device("cuda:0")
+    bf = torch.bfloat16
+    H, G, d, width, ff = s["heads"], s["kv_heads"], s["dim"], s["width"], s["ff"]
+    hbm_gbs, tflops = peaks["hbm_gbs"], peaks.get("bf16_tflops") or 1590.0
+    flush = torch.zeros(96 * 2 ** 20, device=dev)
+    status = torch.zeros(4, dtype=torch.int32, device=dev)
+    rt = pe.parts.Runtime(dev, bf)
+    cos, sin, _ = pe.parts.lookup("position", "rope")({"rotary_dim": d, "theta": 1e6, "max_positions": context + 64, "style": "neox",
+                                                       "scaling": {"factor": 2.0}, "exact": True}, {}, rt).tables()
+    out = {}
+
+    def us_of(fn):
+        return 1e3 * timed(torch, fn, 20, 5, flush, graph=True)
+
+    def roof_us(nbytes, flops=0.0):
+        return max(nbytes / (hbm_gbs * 1e9), flops / (tflops * 1e12)) * 1e6
+
+    def entry(name, us_new, roof_new, like, us_like, roof_like):
+        out[name] = {"us": round(us_new, 2), "roofline_us": round(roof_new, 2), "of_roofline": round(roof_new / us_new, 3),
+                     "like_kernel": like, "like_us": round(us_like, 2), "like_of_roofline": round(roof_like / us_like, 3),
+                     "times_as_far_from_roofline": round((us_new / roof_new) / (us_like / roof_like), 2)}
+
+    for what, n_seqs, q_len, past in (("prompt", 1, prompt, 0), ("decode", batch, 1, context - 1)):
+        n, decode, length = n_seqs * q_len, q_len == 1, past + q_len
+        # ---- streams: write, read, layer norm
+        delta = torch.randn(n, width, device=dev).to(bf)
+        w, bias = torch.ones(width, device=dev), torch.zeros(width, device=dev)
+        normed = torch.empty(n, width, dtype=bf, device=dev)
+        stream = torch.randn(n, width, device=dev)
+        us_like = us_of(lambda: ops.rmsnorm_residual(stream, delta, w, normed, 1e-6))
+        roof_like = roof_us(n * width * 12)
+        for k in (2, 4):
+            X = torch.randn(n, k, width, device=dev)
+            mix, wr, rd = torch.eye(k, device=dev), torch.rand(k, device=dev), torch.rand(k, device=dev)
+            us = us_of(lambda: ops.stream_mix(None, X, delta, bias, mix, wr, rd, "layer", w, 1e-6, normed))
+            entry(f"{what}: output written into {k} streams, read, layer norm", us, roof_us(n * width * (8 * k + 4)), "rmsnorm_residual",
+                  us_like, roof_like)
+        # ---- q|k|v rows: bias, rotation, unit norm, mixed values, append
+        pages_per = -(-length // 64)
+        n_pages = n_seqs * pages_per
+        table = torch.arange(n_pages, dtype=torch.int32, device=dev).view(n_seqs, pages_per).contiguous()
+        qstart = torch.arange(0, n + 1, q_len, dtype=torch.int32, device=dev)
+        pasts = torch.full((n_seqs,), past, dtype=torch.int32, device=dev)
+        slots = torch.arange(n_seqs, dtype=torch.int32, device=dev)
+        token_seq = torch.arange(n_seqs, dtype=torch.int32, device=dev).repeat_interleave(q_len).contiguous()
+        token_pos = (torch.arange(q_len, dtype=torch.int32, device=dev)[None] + past).repeat(n_seqs, 1).view(-1).contiguous()
+        kp = torch.randn(n_pages, G, 64, d, device=dev).to(bf)
+        vp = torch.randn(n_pages, G, 64, d, device=dev).to(bf)
+        where = (token_seq, token_pos, slots, qstart, table, n_pages, kp, vp)
+        qw = torch.ones(d, device=dev)
+        plain_rows = torch.randn(n, (H + 2 * G) * d, device=dev).to(bf)
+        us_like = us_of(lambda: ops.qk_norm_rope_append(plain_rows, n, H, G, d, qw, qw, 1e-6, cos, sin, d, *where, True, status))
+        nbytes = n * (H + 2 * G) * d * 2 + n * (H + G) * d * 2 + n * 2 * G * d * 2
+        rows = torch.randn(n, (H + 2 * G) * d + H, device=dev).to(bf)
+        qb = torch.zeros((H + 2 * G) * d, device=dev)
+        kept = torch.randn(n, G * d, device=dev).to(bf)
+        us = us_of(lambda: ops.qkv_rotate_append(rows, n, H, G, d, d, None, None, 1e-6, cos, sin, d, False, False, None, None, 0, False,
+                                                 *where, True, status, qb, qk_unit=True, v_mix=kept, v_lambda=0.3))
+        entry(f"{what}: bias, rotation, unit norm, mixed values, append", us, roof_us(nbytes + n * G * d * 2), "qk_norm_rope_append",
+              us_like, roof_us(nbytes))
+        # ---- attention with a sink and a gate per head; the same sizes, and values or keys of another size
+        def attention(hd, vd, gated):
+            q = (torch.randn(n, H * hd + H, device=dev) * 0.5).to(bf)
+            k = (torch.randn(n_pages, G, 64, hd, device=dev) * 0.5).to(bf)
+            v = (torch.randn(n_pages, G, 64, vd, device=dev) * 0.5).to(bf)
+            o = torch.empty(n, H * vd, dtype=bf, device=dev)
+            gate = q[:, H * hd:] if gated else None
+            at = (qstart, pasts, slots, table, n_pages, k, v)
+            if not decode and ops.attention_umma_dims_supported(bf, hd, vd, H, G):
+                us = us_of(lambda: ops.attention_umma_prefill(q, o, n_seqs, q_len, H, G, hd, hd ** -0.5, 0, *at, status, sink=gated, v_dim=vd,
+                                                              gate=gate))
+            else:
+                sk, ms, fl = ops.attention_mma_decode_ranges(dev, hd, n_seqs, G, context + 64, 512, v_dim=vd) if decode else (512, 0, 0)
+                scr = torch.empty(ops.attention_generic_scratch_floats(n_seqs, H, vd, max(ms, 1)), device=dev)
+                us = us_of(lambda: ops.attention_mma_gated(decode, q, o, n_seqs, q_len, H, G, hd, vd, hd ** -0.5, 0, *at, scr, sk, ms, status,
+                                                           min_range_keys=fl, sink=gated, gate=gate))
+            nbytes = n * H * (hd + vd) * 2 + n_seqs * length * G * (hd + vd) * 2
+            flops = 2.0 * n * H * (hd + vd) * (length if decode else length / 2)
+            return us, roof_us(nbytes, flops)
+
+        us_like, roof_like = attention(d, d, False)
+        for hd, vd in ((d, d), (d, d // 2), (3 * d // 4, d // 2), (3 * d // 2, d)):
+            us, roof = attention(hd, vd, True)
+            entry(f"{what}: attention with sink and gates, keys of {hd}, values of {vd}", us, roof, f"attention, {d} and {d}", us_like, roof_like)
+        # ---- products: q|k|v with the gates' rows beside q|k|v, gate|up with biases and clamps beside silu
+        x = torch.randn(n, width, device=dev).to(bf)
+        wq = (torch.randn((H + 2 * G) * d, width, device=dev) * 0.02).to(bf)
+        wg = (torch.randn((H + 2 * G) * d + H, width, device=dev) * 0.02).to(bf)
+        oq, og = torch.empty(n, wq.shape[0], dtype=bf, device=dev), torch.empty(n, wg.shape[0], dtype=bf, device=dev)
+        product = lambda rows_out: roof_us((width * rows_out + n * (width + rows_out)) * 2, 2.0 * n * width * rows_out)
+        us = us_of(lambda: rt.linear(x, wg, out=og))
+        us_like = us_of(lambda: rt.linear(x, wq, out=oq))
+        entry(f"{what}: q|k|v|gates product", us, product(wg.shape[0]), "q|k|v product", us_like, product(wq.shape[0]))
+        wgu = (torch.randn(2 * ff, width, device=dev) * 0.02).to(bf)
+        gub = torch.zeros(2 * ff, device=dev)
+        act = torch.empty(n, ff, dtype=bf, device=dev)
+        if rt.takes_small_gemm(x, wgu):
+            run = lambda **kw: ops.gemm_smallm(x, wgu, act, pair_offset=ff, **kw)
+        else:
+            run = lambda **kw: ops.gemm_umma2(x, wgu, act, status, pair_offset=ff, **kw)
+        us = us_of(lambda: run(glu=("clamped_swish", 7.0, 1.702, gub)))
+        us_like = us_of(lambda: run())
+        roof = roof_us((width * 2 * ff + n * (width + ff)) * 2, 4.0 * n * width * ff)
+        entry(f"{what}: gate|up product with biases and clamped gate", us, roof, "gate|up product with silu gate", us_like, roof)
+        gu = torch.randn(n, 2 * ff, device=dev).to(bf)
+        us = us_of(lambda: ops.glu_act(gu, act, "clamped_swish", 7.0, 1.702, gub))
+        us_like = us_of(lambda: ops.silu_mul(gu, act))
+        entry(f"{what}: biases and clamped gate behind a library product", us, roof_us(n * ff * 6), "silu_mul", us_like, roof_us(n * ff * 6))
+    return out
+
+
 def main(args):
     import torch
 
@@ -763,9 +890,9 @@ def main(args):
     for name in names:
         s = SIZES[name]
         row = {"shape": s}
-        wanted = [a for a in (args.arch_names or "vabelorn,qwen3,lunadra,vemepel,zonevik").split(",") if a]
+        wanted = [a for a in (args.arch_names or "vabelorn,qwen3,lunadra,vemepel,zonevik,bobasun").split(",") if a]
         for arch, make in (("vabelorn", vabelorn_config), ("qwen3", qwen3_config), ("lunadra", lunadra_config),
-                           ("vemepel", vemepel_config), ("zonevik", zonevik_config)):
+                           ("vemepel", vemepel_config), ("zonevik", zonevik_config), ("bobasun", bobasun_config)):
             if arch not in wanted:
                 continue
             row[arch] = model_speeds(pe, torch, make(pe, s), prompt, batch, context, args.steps, max(args.warmup, 3))
@@ -785,6 +912,10 @@ def main(args):
         if "zonevik" in wanted:
             row["zonevik_kernels"] = zonevik_kernel_pairs(pe, torch, s, peaks, prompt, batch, context)
             for k, v in row["zonevik_kernels"].items():
+                print(f"[{name}] {k}: {v}", file=sys.stderr, flush=True)
+        if "bobasun" in wanted:
+            row["bobasun_kernels"] = bobasun_kernel_pairs(pe, torch, s, peaks, prompt, batch, context)
+            for k, v in row["bobasun_kernels"].items():
                 print(f"[{name}] {k}: {v}", file=sys.stderr, flush=True)
         result["sizes"][name] = row
     result["gpu_launches"] = pe.kernels.ops.launch_count()

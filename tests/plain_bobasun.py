@@ -185,3 +185,52 @@ def greedy(cfg: dict, weights: Dict[str, torch.Tensor], prompt: List[int], n: in
     for _ in range(n):
         tokens.append(int(forward(cfg, weights, tokens, dtype)[-1].argmax()))
     return tokens[len(prompt):]
+
+
+def random_weights(cfg: dict, seed: int) -> Dict[str, torch.Tensor]:
+    """Random weights by checkpoint name, rounded to bfloat16: biases and mixing numbers large enough to matter, stream mixes
+    that are far from the identity (but not growing), a different set of numbers for every sublayer."""
+    gen = torch.Generator().manual_seed(seed)
+    out: Dict[str, torch.Tensor] = {}
+
+    def put(name, t):
+        out[name] = t.to(torch.bfloat16).to(torch.float32)
+
+    def mat(name, *shape, s):
+        put(name, torch.randn(*shape, generator=gen) * s)
+
+    def norm(name):
+        put(name, 1.0 + 0.2 * torch.randn(W, generator=gen))
+
+    V, W, S = int(cfg["vocab"]), int(cfg["width"]), int(cfg.get("streams", 1))
+    mat("embed", V, W, s=1.0)
+    mat("head", V, W, s=1.0 / math.sqrt(W))
+    norm("final.norm")
+    s_in = 1.0 / math.sqrt(W)
+    for i, entry in enumerate(cfg["layers"]):
+        p, m = f"l{i}", entry["mixer"]
+        H, G, d, dv = (int(m[k]) for k in ("heads", "kv_heads", "dim", "vdim"))
+        for q in ("1", "2"):
+            if q == "2" and entry.get("mlp") is None:
+                continue
+            norm(f"{p}.norm{q}")
+            mat(f"{p}.hc{q}.in", S, s=1.0)
+            mat(f"{p}.hc{q}.out", S, s=1.0)
+            put(f"{p}.hc{q}.mix", 0.6 * torch.eye(S) + 0.5 / math.sqrt(S) * torch.randn(S, S, generator=gen))
+        for name, rows in (("q", H * d), ("k", G * d), ("v", G * dv)):
+            mat(f"{p}.mix.{name}", rows, W, s=s_in)
+            mat(f"{p}.mix.{name}.b", rows, s=0.5)
+        if m.get("v_mix"):
+            put(f"{p}.mix.vmix", torch.rand((), generator=gen) * 0.8 + 0.1)
+        mat(f"{p}.mix.g", H, W, s=2.0 * s_in)
+        mat(f"{p}.mix.o", W, H * dv, s=1.0 / math.sqrt(H * dv))
+        mat(f"{p}.mix.o.b", W, s=0.3)
+        mlp = entry.get("mlp")
+        if mlp is not None:
+            ff = int(mlp["ff"])
+            for name in ("gate", "up"):
+                mat(f"{p}.mlp.{name}", ff, W, s=s_in)
+                mat(f"{p}.mlp.{name}.b", ff, s=0.5)
+            mat(f"{p}.mlp.down", W, ff, s=1.0 / math.sqrt(ff))
+            mat(f"{p}.mlp.down.b", W, s=0.3)
+    return out
