@@ -856,6 +856,12 @@ def bobasun_kernel_pairs(pe, torch, s, peaks, prompt, batch, context):
         us = us_of(lambda: rt.linear(x, wg, out=og))
         us_like = us_of(lambda: rt.linear(x, wq, out=oq))
         entry(f"{what}: q|k|v|gates product", us, product(wg.shape[0]), "q|k|v product", us_like, product(wq.shape[0]))
+        if not decode:       # many rows: everything on q|k|v in the product's epilogue
+            like = lambda: ops.gemm_umma2_qkv_rope(x, wq, oq, H, G, d, qw, qw, 1e-6, cos, sin, d, *where, True, status)
+            new = lambda: ops.gemm_umma2_qkv_rope(x, wg, og, H, G, d, None, None, 1e-6, cos, sin, d, *where, True, status, qb, qk_unit=True,
+                                                  v_mix=kept, v_lambda=0.3)
+            entry(f"{what}: q|k|v|gates product with biases, rotation, unit norm, mixed values, append", us_of(new), product(wg.shape[0]),
+                  "q|k|v product with norm, rotation, append", us_of(like), product(wq.shape[0]))
         wgu = (torch.randn(2 * ff, width, device=dev) * 0.02).to(bf)
         gub = torch.zeros(2 * ff, device=dev)
         act = torch.empty(n, ff, dtype=bf, device=dev)

@@ -1,5 +1,6 @@
-// Prefill attention on the fifth-generation tensor cores (tcgen05.mma), for bfloat16, head size 128 (or 72 to 120 in
-// steps of 8, the tile's spare columns filled with zeros by TMA), values of 8 to 128 features (in steps of 8; up to 64 a
+// Prefill attention on the fifth-generation tensor cores (tcgen05.mma), for bfloat16, head size 128 (or 72 to 256 in
+// steps of 8: tiles of 128, 192 or 256 features, their spare columns filled with zeros by TMA; beyond 128 one block
+// fits on an SM instead of two), values of 8 to 128 features (in steps of 8; up to 64 a
 // P.V product of half the width), and groups of up to 32 query heads per kv head.  Same interface and formulas as
 // attention_mma.cu (pygguf_engine/kv_cache.py:833, 2189-2192 masks; 756 head mapping; 836-861 online
 // softmax); other shapes keep using that file.
@@ -47,11 +48,12 @@
 namespace pe {
 namespace fau {
 
-constexpr int HD = 128;        // head size
+constexpr int HD = 128;        // features of a value row's tile, and of a head whose output is turned
 constexpr int BM = 128;        // rows per block
 constexpr int BN = 64;         // keys per page
-constexpr int kQBytes = BM * HD * 2;          // 32 KB: two 64-feature halves of [128 rows][128 B]
-constexpr int kPageBytes = BN * HD * 2;        // 16 KB: a K or V page, two halves of [64][128 B]
+constexpr int kQPart = BM * 64 * 2;           // 16 KB: 64 features of Q, [128 rows][128 B]
+constexpr int kKPart = BN * 64 * 2;           // 8 KB: 64 features of a page, [64][128 B]
+constexpr int kPageBytes = 2 * kKPart;        // 16 KB: a V page (a K page: KH parts)
 constexpr int kKStages = 2, kVStages = 3;     // K is spent once S is there, V only after P.V: V needs the deeper ring
 constexpr int kTmemCols = 256;                // S0 [0,64) S1 [64,128) O [128,256)
 constexpr float kRescaleThreshold = 8.0f;     // in log2 units
@@ -174,7 +176,7 @@ __device__ __forceinline__ uint32_t desc_lo_mn_major(uint32_t saddr, uint32_t lb
   return ((saddr >> 4) & 0x3FFF) | (((lbo_bytes >> 4) & 0x3FFF) << 16);
 }
 
-// S = Q.K^T of one page: eight k-steps of 16 features.  Both operands are two 64-feature halves of [rows][128 B]:
+// S = Q.K^T of one page of 128 features: eight k-steps of 16 features.  Both operands are two 64-feature halves of [rows][128 B]:
 // a k-step moves 32 bytes (2 units) inside a half, the second half lies rows * 128 bytes further (A: 128 rows,
 // 1,024 units; B: 64 keys, 512 units).
 #define PE_QK_STEP(A, B)                                                                       \
@@ -196,6 +198,17 @@ __device__ __forceinline__ void umma_qk_page(uint32_t d_tmem, uint32_t a_lo, uin
       "tcgen05.mma.cta_group::1.kind::f16 [%0], da, db, %4, pf;\n"
       PE_QK_STEP(2, 2) PE_QK_STEP(4, 4) PE_QK_STEP(6, 6)
       PE_QK_STEP(1024, 512) PE_QK_STEP(1026, 514) PE_QK_STEP(1028, 516) PE_QK_STEP(1030, 518)
+      "}\n" ::"r"(d_tmem), "r"(a_lo), "r"(b_lo), "r"(kDescHi), "r"(idesc) : "memory");
+}
+// Another 64 features of the same S: four more k-steps that accumulate.
+__device__ __forceinline__ void umma_qk_more(uint32_t d_tmem, uint32_t a_lo, uint32_t b_lo, uint32_t idesc) {
+  asm volatile(
+      "{\n"
+      ".reg .pred pt;\n"
+      ".reg .b64 da, db;\n"
+      ".reg .b32 al, bl;\n"
+      "setp.eq.b32 pt, %4, %4;\n"
+      PE_QK_STEP(0, 0) PE_QK_STEP(2, 2) PE_QK_STEP(4, 4) PE_QK_STEP(6, 6)
       "}\n" ::"r"(d_tmem), "r"(a_lo), "r"(b_lo), "r"(kDescHi), "r"(idesc) : "memory");
 }
 #undef PE_QK_STEP
@@ -260,16 +273,18 @@ __device__ __forceinline__ void load_3d(void* dst, const CUtensorMap* map, int x
       ::"r"(tma::smem_addr(dst)), "l"(map), "r"(x), "r"(y), "r"(z), "r"(tma::smem_addr(bar)) : "memory");
 }
 
-// grid: G persistent blocks (see the file's head); block: 192 threads.
-__global__ void __launch_bounds__(192, 2)
+// grid: G persistent blocks (see the file's head); block: 192 threads.  KH: 64-feature parts of a Q or K tile.
+template <int KH>
+__global__ void __launch_bounds__(192, KH > 2 ? 1 : 2)
 prefill_umma_kernel(Args a, const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap kmap,
                     const __grid_constant__ CUtensorMap vmap) {
   // All shared memory is dynamic and starts on a 1,024-byte boundary (there are no static shared
   // variables in front of it), so that two blocks fit on an SM: tiles first, barriers behind them.
   extern __shared__ __align__(1024) char smem[];
-  char* q_s = smem;                       // [2 halves][128 rows][128 B]
-  char* k_s = q_s + kQBytes;              // kKStages K pages
-  char* v_s = k_s + kKStages * kPageBytes;   // kVStages V pages
+  constexpr int kKPage = KH * kKPart;
+  char* q_s = smem;                       // [KH parts][128 rows][128 B]
+  char* k_s = q_s + KH * kQPart;          // kKStages K pages
+  char* v_s = k_s + kKStages * kKPage;    // kVStages V pages
   uint64_t* bars = reinterpret_cast<uint64_t*>(v_s + kVStages * kPageBytes);
   uint64_t& q_full = bars[0];
   // The MMA thread's commits are few on purpose: that thread issues one instruction after the other, a commit costs
@@ -327,11 +342,11 @@ prefill_umma_kernel(Args a, const __grid_constant__ CUtensorMap qmap, const __gr
     failed = 0;
     tma::fence_barrier_init();
   }
-  // the Q rows beyond the block's whole tokens are no copy's target: zero them (both feature halves)
+  // the Q rows beyond the block's whole tokens are no copy's target: zero them (all feature parts)
   // so that the MMA's rows there stay finite; they are never stored
-  for (int i = tid; i < (BM - rows_blk) * 2 * 8; i += blockDim.x) {
-    const int rr = rows_blk + i / 16, half = (i / 8) & 1, chunk = i & 7;
-    *reinterpret_cast<uint4*>(q_s + half * (kQBytes / 2) + rr * 128 + chunk * 16) = make_uint4(0, 0, 0, 0);
+  for (int i = tid; i < (BM - rows_blk) * KH * 8; i += blockDim.x) {
+    const int rr = rows_blk + i / (KH * 8), part = (i / 8) % KH, chunk = i & 7;
+    *reinterpret_cast<uint4*>(q_s + part * kQPart + rr * 128 + chunk * 16) = make_uint4(0, 0, 0, 0);
   }
   tma::fence_proxy_async();
   if (warp == 4) tmem_alloc(&tmem_holder, kTmemCols);
@@ -376,9 +391,9 @@ prefill_umma_kernel(Args a, const __grid_constant__ CUtensorMap qmap, const __gr
           failed = 1;
           continue;              // the loop's head then tells the other warps that nothing follows
         }
-        tma::mbar_expect_tx(&q_full, (uint32_t)(rows_blk * HD * 2));
-        load_3d(q_s, &qmap, 0, w.kvh * group, w.q0 + w.tok0, &q_full);
-        load_3d(q_s + kQBytes / 2, &qmap, 64, w.kvh * group, w.q0 + w.tok0, &q_full);
+        tma::mbar_expect_tx(&q_full, (uint32_t)(rows_blk * KH * 64 * 2));
+#pragma unroll
+        for (int h = 0; h < KH; ++h) load_3d(q_s + h * kQPart, &qmap, 64 * h, w.kvh * group, w.q0 + w.tok0, &q_full);
         // Row of the page table's page for the item's page j in the K and V tensors' 2-D views.
         auto page_row = [&](int j) -> int {
           const int k0 = w.k_begin + j * BN;
@@ -397,9 +412,9 @@ prefill_umma_kernel(Args a, const __grid_constant__ CUtensorMap qmap, const __gr
           return tma::mbar_wait(&s_full[g % kKStages], ((g / kKStages) & 1) ^ 1);
         };
         auto load_k = [&](uint32_t g, int y, uint64_t* bar) {
-          char* kd = k_s + (g % kKStages) * kPageBytes;
-          tma::load_2d(kd, &kmap, 0, y, bar);
-          tma::load_2d(kd + BN * 128, &kmap, 64, y, bar);
+          char* kd = k_s + (g % kKStages) * kKPage;
+#pragma unroll
+          for (int h = 0; h < KH; ++h) tma::load_2d(kd + h * kKPart, &kmap, 64 * h, y, bar);
         };
         int y = page_row(0);
         // the first page's K alone; every later K page travels with the V page before it
@@ -408,7 +423,7 @@ prefill_umma_kernel(Args a, const __grid_constant__ CUtensorMap qmap, const __gr
           failed = 1;
           continue;
         }
-        tma::mbar_expect_tx(&k0_full, kPageBytes);
+        tma::mbar_expect_tx(&k0_full, kKPage);
         load_k(n, y, &k0_full);
         for (int j = 0; j < w.n_tiles && !failed; ++j) {
           const uint32_t g = n + j;
@@ -421,7 +436,7 @@ prefill_umma_kernel(Args a, const __grid_constant__ CUtensorMap qmap, const __gr
             break;
           }
           char* vd = v_s + vs * kPageBytes;
-          tma::mbar_expect_tx(&kv_full[vs], (uint32_t)(a.v_halves * (kPageBytes / 2) + (more ? kPageBytes : 0)));
+          tma::mbar_expect_tx(&kv_full[vs], (uint32_t)(a.v_halves * kKPart + (more ? kKPage : 0)));
           tma::load_2d(vd, &vmap, 0, y, &kv_full[vs]);
           if (a.v_halves > 1) tma::load_2d(vd + BN * 128, &vmap, 64, y, &kv_full[vs]);
           if (more) load_k(g + 1, y_next, &kv_full[vs]);
@@ -437,7 +452,7 @@ prefill_umma_kernel(Args a, const __grid_constant__ CUtensorMap qmap, const __gr
       const uint32_t idesc_qk = instr_desc(BM, BN, false);
       const uint32_t idesc_pv = instr_desc(BM, 64 * a.v_halves, true);
       const uint32_t q_lo = desc_lo_k_major(tma::smem_addr(q_s));
-      const uint32_t k_lo0 = desc_lo_k_major(tma::smem_addr(k_s));               // stage s: + s * (16 KB / 16)
+      const uint32_t k_lo0 = desc_lo_k_major(tma::smem_addr(k_s));               // stage s: + s * (a K page / 16)
       const uint32_t v_lo0 = desc_lo_mn_major(tma::smem_addr(v_s), BN * 128);
       bool ok = true;
       for (uint32_t f = 0; ok && !failed; ++f) {
@@ -453,7 +468,11 @@ prefill_umma_kernel(Args a, const __grid_constant__ CUtensorMap qmap, const __gr
           const uint32_t g = n + j;
           const int st = g & 1, ks = g % kKStages;
           fence_after_sync();
-          umma_qk_page(tmem_base + st * BN, q_lo, k_lo0 + ((uint32_t)ks << 10), idesc_qk);
+          const uint32_t k_lo = k_lo0 + (uint32_t)ks * (kKPage >> 4);
+          umma_qk_page(tmem_base + st * BN, q_lo, k_lo, idesc_qk);
+#pragma unroll
+          for (int h = 2; h < KH; ++h)
+            umma_qk_more(tmem_base + st * BN, q_lo + h * (kQPart >> 4), k_lo + h * (kKPart >> 4), idesc_qk);
           umma_commit(&s_full[st]);     // S is there, and the K stage is spent
           if (j == n_tiles - 1) umma_commit(&q_empty);   // ... and so is Q, after the item's last S product
         };
@@ -675,7 +694,7 @@ extern "C" int pe_attention_umma_supported(int head_dim, int n_heads, int n_kv_h
 
 // The same for keys and values of sizes of their own.
 extern "C" int pe_attention_umma_dims_supported(int head_dim, int v_dim, int n_heads, int n_kv_heads) {
-  if (head_dim <= 64 || head_dim > 128 || head_dim % 8 || v_dim < 8 || v_dim > 128 || v_dim % 8) return 0;
+  if (head_dim <= 64 || head_dim > 256 || head_dim % 8 || v_dim < 8 || v_dim > 128 || v_dim % 8) return 0;
   return pe_attention_umma_supported(128, n_heads, n_kv_heads);
 }
 
@@ -746,22 +765,25 @@ extern "C" int pe_attention_umma_prefill_gated(const void* q, long long q_ld, lo
   int me = pe::tma::make_map_2d_bf16(&kmap, k_pages, head_dim, rows, head_dim, 64, BN);
   if (me == 0) me = pe::tma::make_map_2d_bf16(&vmap, v_pages, v_dim, rows, v_dim, 64, BN);
   if (me != 0) return me < 0 ? me : PE_ERR_BAD_ARGUMENT;
-  const size_t smem = kQBytes + (kKStages + kVStages) * kPageBytes + 256;   // tiles, then barriers and the two-slot ring
-  static bool attr_set = false;
-  if (!attr_set) {
-    cudaError_t ce = cudaFuncSetAttribute(prefill_umma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  const int kh = head_dim <= 128 ? 2 : (head_dim + 63) / 64;
+  // tiles, then barriers and the two-slot ring
+  const size_t smem = (size_t)kh * kQPart + kKStages * (size_t)kh * kKPart + kVStages * kPageBytes + 256;
+  auto kern = kh == 2 ? prefill_umma_kernel<2> : (kh == 3 ? prefill_umma_kernel<3> : prefill_umma_kernel<4>);
+  static bool attr_set[5] = {};
+  if (!attr_set[kh]) {
+    cudaError_t ce = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (ce != cudaSuccess) return (int)ce;
-    attr_set = true;
+    attr_set[kh] = true;
   }
   const int rows_blk = (BM / a.group) * a.group;
   const long long tiles = ((long long)max_q * a.group + rows_blk - 1) / rows_blk;
   const long long total = tiles * n_kv_heads * n_seqs;
   if (total <= 0 || total > (1ll << 30)) return PE_ERR_UNSUPPORTED_SIZE;
   a.tiles = (int)tiles; a.n_seqs = n_seqs; a.work_counter = work_counter;
-  // two blocks fit on an SM (shared memory, tensor memory columns); no more blocks than items
-  const long long slots = 2ll * (n_sms > 0 ? n_sms : pe::kSMs);
+  // two blocks fit on an SM (shared memory, tensor memory columns), or one with wider keys; no more blocks than items
+  const long long slots = (kh > 2 ? 1ll : 2ll) * (n_sms > 0 ? n_sms : pe::kSMs);
   dim3 grid((unsigned)(total < slots ? total : slots));
-  pe::launch(prefill_umma_kernel, grid, 192, smem, stream, a, qmap, kmap, vmap);
+  pe::launch(kern, grid, 192, smem, stream, a, qmap, kmap, vmap);
   PE_LAUNCH_CHECK();
   return PE_OK;
 }

@@ -143,14 +143,36 @@ __device__ __forceinline__ float glu_exact(int kind, float g, float u, float lim
   u = fminf(fmaxf(u, -limit), limit);
   return g / (1.f + expf(-alpha * g)) * (u + 1.f);
 }
-// Two neighbouring outputs, packed to bfloat16; `col`: the first one's number, `n`: outputs in all.
-__device__ __forceinline__ uint32_t glu_fast_pair(const GluEpilogue& e, float g0, float g1, float u0, float u1, int col, int n) {
-  if (e.bias) {
-    if (col < n) { g0 += e.bias[col]; u0 += e.bias[n + col]; }
-    if (col + 1 < n) { g1 += e.bias[col + 1]; u1 += e.bias[n + col + 1]; }
-  }
+// Two neighbouring outputs, packed to bfloat16.
+__device__ __forceinline__ uint32_t glu_fast_pair(const GluEpilogue& e, float g0, float g1, float u0, float u1) {
   const __nv_bfloat162 v = __floats2bfloat162_rn(glu_fast(e, g0, u0), glu_fast(e, g1, u1));
   return *reinterpret_cast<const uint32_t*>(&v);
+}
+// 32 neighbouring outputs from column `col` of `n` (both multiples of 32; the bias is 16-byte aligned), float32 sums as bits:
+// the kind of activation is decided once, not per output.
+template <int KIND>
+__device__ __forceinline__ void glu_fast_32_of(const GluEpilogue& e, const uint32_t (&g)[32], const uint32_t (&u)[32], int col, int n,
+                                               uint32_t (&o)[16]) {
+#pragma unroll
+  for (int q = 0; q < 8; ++q) {
+    float4 bg = make_float4(0.f, 0.f, 0.f, 0.f), bu = bg;
+    if (e.bias) {
+      bg = __ldg(reinterpret_cast<const float4*>(e.bias + col) + q);
+      bu = __ldg(reinterpret_cast<const float4*>(e.bias + n + col) + q);
+    }
+    GluEpilogue k = e;
+    k.kind = KIND;
+    o[2 * q] = glu_fast_pair(k, __uint_as_float(g[4 * q]) + bg.x, __uint_as_float(g[4 * q + 1]) + bg.y,
+                             __uint_as_float(u[4 * q]) + bu.x, __uint_as_float(u[4 * q + 1]) + bu.y);
+    o[2 * q + 1] = glu_fast_pair(k, __uint_as_float(g[4 * q + 2]) + bg.z, __uint_as_float(g[4 * q + 3]) + bg.w,
+                                 __uint_as_float(u[4 * q + 2]) + bu.z, __uint_as_float(u[4 * q + 3]) + bu.w);
+  }
+}
+__device__ __forceinline__ void glu_fast_32(const GluEpilogue& e, const uint32_t (&g)[32], const uint32_t (&u)[32], int col, int n,
+                                            uint32_t (&o)[16]) {
+  if (e.kind == 3) glu_fast_32_of<3>(e, g, u, col, n, o);
+  else if (e.kind == 2) glu_fast_32_of<2>(e, g, u, col, n, o);
+  else glu_fast_32_of<1>(e, g, u, col, n, o);
 }
 
 // ---- reductions --------------------------------------------------------------------------------

@@ -228,10 +228,7 @@ gemm_umma_kernel(Params p, const __grid_constant__ CUtensorMap amap, const __gri
                 o[j] = pack2(v0, v1);
               }
             } else {
-#pragma unroll
-              for (int j = 0; j < 16; ++j)
-                o[j] = glu_fast_pair(p.glu, __uint_as_float(g[2 * j]), __uint_as_float(g[2 * j + 1]), __uint_as_float(u[2 * j]),
-                                     __uint_as_float(u[2 * j + 1]), n0 + c + 2 * j, p.N);
+              glu_fast_32(p.glu, g, u, n0 + c, p.N, o);
             }
             if (n0 + c + 32 <= p.N && (p.ldy % 8) == 0) {
 #pragma unroll
@@ -314,7 +311,7 @@ extern "C" int pe_gemm_umma_glu(const void* x, long long ldx, const void* w, voi
                         cudaStream_t stream) {
   using namespace pe::umma;
   if (M <= 0 || N <= 0) return PE_OK;
-  if (kind < 1 || kind > 3 || (pair_offset <= 0 && bias)) return PE_ERR_BAD_ARGUMENT;
+  if (kind < 1 || kind > 3 || (pair_offset <= 0 && bias) || (uintptr_t)bias % 16) return PE_ERR_BAD_ARGUMENT;
   if (!pe_gemm_umma_supported(M, N, K, pair_offset)) return PE_ERR_UNSUPPORTED_SIZE;
   if (((uintptr_t)x % 16) || ((uintptr_t)w % 16) || (ldx * 2) % 16) return PE_ERR_BAD_ARGUMENT;
   Params p;

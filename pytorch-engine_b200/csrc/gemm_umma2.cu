@@ -55,6 +55,13 @@ struct RopeFuse {
   const int* page_table; int table_stride, num_pages;
   __nv_bfloat16* k_pages; __nv_bfloat16* v_pages;   // [num_pages, n_kv_heads, 64, 128]
   int write_cache;
+  // What a plain layer does not have (defaults: null, 0): biases of q|k|v ([features], added first); q and k divided by their
+  // root mean square over the head (no weight; after a rotation that leaves lengths as they are it is the same before it);
+  // values mixed with another layer's of the same tokens, (1 - v_lambda) v + v_lambda v_mix, or left in v_keep for layers
+  // further on ([M, n_kv_heads * 128]).  Columns behind q|k|v (a gate's) go to the output rows as they are.
+  const float* bias;
+  int qk_unit;
+  const __nv_bfloat16* v_mix; __nv_bfloat16* v_keep; float v_lambda;
 };
 
 struct Params {
@@ -197,11 +204,33 @@ __device__ __forceinline__ void rope_epilogue(const Params& p, int row, int n0, 
     const int col0 = n0 + h * D;
     if (col0 >= p.N) break;
     const int head = col0 / D;
+    if (head >= r.n_heads + 2 * r.n_kv_heads) {           // columns behind q|k|v
+#pragma unroll 1
+      for (int c = 0; c < D && col0 + c < p.N; c += 32) {
+        uint32_t v[32];
+        __syncwarp();
+        tmem_ld32(t_row + h * D + c, v);
+        tmem_ld_wait();
+        if (live) {
+          __nv_bfloat16* yrow = reinterpret_cast<__nv_bfloat16*>(p.y) + (size_t)row * p.ldy + col0 + c;
+#pragma unroll
+          for (int j = 0; j < 32; ++j)
+            if (col0 + c + j < p.N) yrow[j] = __float2bfloat16_rn(__uint_as_float(v[j]));
+        }
+      }
+      continue;
+    }
     const bool is_q = head < r.n_heads;
     const bool is_k = !is_q && head < r.n_heads + r.n_kv_heads;
     const int kv_head = is_q ? 0 : (is_k ? head - r.n_heads : head - r.n_heads - r.n_kv_heads);
     const uint32_t t_head = t_row + h * D;
     const float* w = is_q ? r.q_norm_w : (is_k ? r.k_norm_w : nullptr);
+    const bool is_v = !is_q && !is_k;
+    const bool unit = r.qk_unit != 0 && !is_v;
+    const float4* bias = r.bias ? reinterpret_cast<const float4*>(r.bias + col0) : nullptr;
+    const size_t v_off = ((size_t)row * r.n_kv_heads + kv_head) * D;
+    const __nv_bfloat16* mix = is_v && r.v_mix && live ? r.v_mix + v_off : nullptr;
+    __nv_bfloat16* keep = is_v && r.v_keep && live ? r.v_keep + v_off : nullptr;
     const bool wanted = is_q || r.write_cache;            // k and v of a layer that only reads a cache go nowhere
     // where the row goes: q into the output rows, k and v into their page of the cache
     __nv_bfloat16* dst = nullptr;
@@ -235,7 +264,7 @@ __device__ __forceinline__ void rope_epilogue(const Params& p, int row, int n0, 
     }
     // the norm's scale: sum of squares over the head, in four chains added up in a fixed order
     float inv = 1.f;
-    if (w != nullptr) {
+    if (w != nullptr || unit) {
       float ss[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll 1
       for (int c = 0; c < D; c += 32) {
@@ -244,9 +273,14 @@ __device__ __forceinline__ void rope_epilogue(const Params& p, int row, int n0, 
         tmem_ld32(t_head + c, v);
         tmem_ld_wait();
 #pragma unroll
-        for (int j = 0; j < 32; ++j) {
-          const float x = bf16_round(v[j]);
-          ss[j & 3] = fmaf(x, x, ss[j & 3]);
+        for (int j = 0; j < 8; ++j) {
+          const float4 b = bias ? bias[c / 4 + j] : make_float4(0.f, 0.f, 0.f, 0.f);
+          const float bb[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float x = bf16_round(v[4 * j + e]) + bb[e];
+            ss[e] = fmaf(x, x, ss[e]);
+          }
         }
       }
       inv = rsqrtf(((ss[0] + ss[1]) + (ss[2] + ss[3])) / (float)D + r.eps);
@@ -259,7 +293,7 @@ __device__ __forceinline__ void rope_epilogue(const Params& p, int row, int n0, 
       tmem_ld32(t_head + c, a);
       tmem_ld32(t_head + HALF + c, b);
       tmem_ld_wait();
-      if (dst != nullptr) {
+      if (dst != nullptr || keep != nullptr) {
         uint32_t o1[16], o2[16];
         const bool rot = rotates && !(!is_q && !is_k);
         const float4* cs = rot ? reinterpret_cast<const float4*>(r.cos_table + (size_t)pos * HALF + c) : nullptr;
@@ -273,6 +307,27 @@ __device__ __forceinline__ void rope_epilogue(const Params& p, int row, int n0, 
           for (int e = 0; e < 4; ++e) {
             x1[e] = bf16_round(a[4 * q4 + e]);
             x2[e] = bf16_round(b[4 * q4 + e]);
+          }
+          if (bias) {
+            const float4 b1 = bias[c / 4 + q4], b2 = bias[HALF / 4 + c / 4 + q4];
+            x1[0] += b1.x; x1[1] += b1.y; x1[2] += b1.z; x1[3] += b1.w;
+            x2[0] += b2.x; x2[1] += b2.y; x2[2] += b2.z; x2[3] += b2.w;
+          }
+          if (mix) {
+            const float lam = r.v_lambda, rest = 1.f - r.v_lambda;
+            const uint2 m1 = *reinterpret_cast<const uint2*>(mix + c + 4 * q4), m2 = *reinterpret_cast<const uint2*>(mix + HALF + c + 4 * q4);
+            const uint32_t mm[4] = {m1.x, m1.y, m2.x, m2.y};
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              const float2 f1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&mm[e]));
+              const float2 f2 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&mm[2 + e]));
+              x1[2 * e] = rest * x1[2 * e] + lam * f1.x; x1[2 * e + 1] = rest * x1[2 * e + 1] + lam * f1.y;
+              x2[2 * e] = rest * x2[2 * e] + lam * f2.x; x2[2 * e + 1] = rest * x2[2 * e + 1] + lam * f2.y;
+            }
+          }
+          if (unit && !w) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) { x1[e] *= inv; x2[e] *= inv; }
           }
           if (w) {
             const float4 wa = w1[q4], wb = w2[q4];
@@ -297,8 +352,16 @@ __device__ __forceinline__ void rope_epilogue(const Params& p, int row, int n0, 
         }
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-          reinterpret_cast<uint4*>(dst + c)[j] = make_uint4(o1[4 * j], o1[4 * j + 1], o1[4 * j + 2], o1[4 * j + 3]);
-          reinterpret_cast<uint4*>(dst + HALF + c)[j] = make_uint4(o2[4 * j], o2[4 * j + 1], o2[4 * j + 2], o2[4 * j + 3]);
+          const uint4 v1 = make_uint4(o1[4 * j], o1[4 * j + 1], o1[4 * j + 2], o1[4 * j + 3]);
+          const uint4 v2 = make_uint4(o2[4 * j], o2[4 * j + 1], o2[4 * j + 2], o2[4 * j + 3]);
+          if (dst != nullptr) {
+            reinterpret_cast<uint4*>(dst + c)[j] = v1;
+            reinterpret_cast<uint4*>(dst + HALF + c)[j] = v2;
+          }
+          if (keep != nullptr) {
+            reinterpret_cast<uint4*>(keep + c)[j] = v1;
+            reinterpret_cast<uint4*>(keep + HALF + c)[j] = v2;
+          }
         }
       }
     }
@@ -444,10 +507,7 @@ gemm_umma2_kernel(Params p, const __grid_constant__ CUtensorMap amap, const __gr
                 o[j] = pack2(v0, v1);
               }
             } else {
-#pragma unroll
-              for (int j = 0; j < 16; ++j)
-                o[j] = glu_fast_pair(p.glu, __uint_as_float(g[2 * j]), __uint_as_float(g[2 * j + 1]), __uint_as_float(u[2 * j]),
-                                     __uint_as_float(u[2 * j + 1]), n0 + c + 2 * j, p.N);
+              glu_fast_32(p.glu, g, u, n0 + c, p.N, o);
             }
             if (n0 + c + 32 <= p.N && (p.ldy % 8) == 0) {
 #pragma unroll
@@ -537,7 +597,7 @@ extern "C" int pe_gemm_umma2_glu(const void* x, long long ldx, const void* w, vo
                         cudaStream_t stream) {
   using namespace pe::umma2;
   if (M <= 0 || N <= 0) return PE_OK;
-  if (kind < 1 || kind > 3 || (pair_offset <= 0 && bias)) return PE_ERR_BAD_ARGUMENT;
+  if (kind < 1 || kind > 3 || (pair_offset <= 0 && bias) || (uintptr_t)bias % 16) return PE_ERR_BAD_ARGUMENT;
   if (!pe_gemm_umma2_supported(M, N, K, pair_offset) || n_sms < 2) return PE_ERR_UNSUPPORTED_SIZE;
   if (((uintptr_t)x % 16) || ((uintptr_t)w % 16) || (ldx * 2) % 16) return PE_ERR_BAD_ARGUMENT;
   Params p;
@@ -566,21 +626,38 @@ extern "C" int pe_gemm_umma2_qkv_rope(const void* x, long long ldx, const void* 
                                       const int* seq_slot, const int* seq_qstart, const int* page_table, int table_stride,
                                       int num_pages, void* k_pages, void* v_pages, int write_cache, int n_sms, int* status,
                                       cudaStream_t stream) {
+  return pe_gemm_umma2_qkv_rope_ex(x, ldx, w, qkv, ld, M, K, n_heads, n_kv_heads, head_dim, 0, q_norm_w, k_norm_w, eps, cos_table,
+                                   sin_table, rotary_dim, table_rows, nullptr, 0, nullptr, 0.f, nullptr, token_seq, token_pos,
+                                   seq_slot, seq_qstart, page_table, table_stride, num_pages, k_pages, v_pages, write_cache, n_sms,
+                                   status, stream);
+}
+
+// The same with the rest of RopeFuse and `extra_cols` weight rows behind q|k|v, whose results go to qkv's columns behind them.
+extern "C" int pe_gemm_umma2_qkv_rope_ex(const void* x, long long ldx, const void* w, void* qkv, long long ld, int M, int K,
+                                         int n_heads, int n_kv_heads, int head_dim, int extra_cols, const float* q_norm_w,
+                                         const float* k_norm_w, float eps, const float* cos_table, const float* sin_table,
+                                         int rotary_dim, int table_rows, const float* bias, int qk_unit, const void* v_mix,
+                                         float v_lambda, void* v_keep, const int* token_seq, const int* token_pos,
+                                         const int* seq_slot, const int* seq_qstart, const int* page_table, int table_stride,
+                                         int num_pages, void* k_pages, void* v_pages, int write_cache, int n_sms, int* status,
+                                         cudaStream_t stream) {
   using namespace pe::umma2;
   if (M <= 0) return PE_OK;
   if (cos_table == nullptr) rotary_dim = 0;
   if (!pe_gemm_umma2_qkv_rope_supported(M, K, n_heads, n_kv_heads, head_dim, rotary_dim) || n_sms < 2) return PE_ERR_UNSUPPORTED_SIZE;
   if (((uintptr_t)x % 16) || ((uintptr_t)w % 16) || (ldx * 2) % 16 || ((uintptr_t)qkv % 16) || (ld * 2) % 16 ||
       ((uintptr_t)k_pages % 16) || ((uintptr_t)v_pages % 16) || ((uintptr_t)q_norm_w % 16) || ((uintptr_t)k_norm_w % 16) ||
-      ((uintptr_t)cos_table % 16) || ((uintptr_t)sin_table % 16))
+      ((uintptr_t)cos_table % 16) || ((uintptr_t)sin_table % 16) || ((uintptr_t)bias % 16) || ((uintptr_t)v_mix % 16) ||
+      ((uintptr_t)v_keep % 16) || extra_cols < 0)
     return PE_ERR_BAD_ARGUMENT;
   if (write_cache && (page_table == nullptr || k_pages == nullptr || v_pages == nullptr)) return PE_ERR_BAD_ARGUMENT;
   Params p;
-  p.M = M; p.N = (n_heads + 2 * n_kv_heads) * head_dim; p.K = K; p.y = qkv; p.ldy = ld; p.status = status;
+  p.M = M; p.N = (n_heads + 2 * n_kv_heads) * head_dim + extra_cols; p.K = K; p.y = qkv; p.ldy = ld; p.status = status;
   p.mode = 3;
   p.pair_offset = 0;
   p.glu = pe::GluEpilogue{1, 0.f, 1.f, nullptr};
   RopeFuse& r = p.rope;
+  r.bias = bias; r.qk_unit = qk_unit; r.v_mix = (const __nv_bfloat16*)v_mix; r.v_keep = (__nv_bfloat16*)v_keep; r.v_lambda = v_lambda;
   r.n_heads = n_heads; r.n_kv_heads = n_kv_heads; r.q_norm_w = q_norm_w; r.k_norm_w = k_norm_w; r.eps = eps;
   r.cos_table = rotary_dim > 0 ? cos_table : nullptr; r.sin_table = rotary_dim > 0 ? sin_table : nullptr;
   r.table_rows = table_rows; r.token_seq = token_seq; r.token_pos = token_pos; r.seq_slot = seq_slot;

@@ -452,8 +452,12 @@ __global__ void __launch_bounds__(256) glu_act_vec8_kernel(const __nv_bfloat16* 
     uint32_t o[4];
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
-      const float2 g = __bfloat1622float2(g2[k]), u = __bfloat1622float2(u2[k]);
-      o[k] = glu_fast_pair(e, g.x, g.y, u.x, u.y, c + 2 * k, inter);
+      float2 g = __bfloat1622float2(g2[k]), u = __bfloat1622float2(u2[k]);
+      if (e.bias) {
+        const float2 bg = __ldg(reinterpret_cast<const float2*>(e.bias + c) + k), bu = __ldg(reinterpret_cast<const float2*>(e.bias + inter + c) + k);
+        g.x += bg.x; g.y += bg.y; u.x += bu.x; u.y += bu.y;
+      }
+      o[k] = glu_fast_pair(e, g.x, g.y, u.x, u.y);
     }
     *reinterpret_cast<uint4*>(out + r * inter + c) = make_uint4(o[0], o[1], o[2], o[3]);
   }
@@ -594,7 +598,7 @@ extern "C" int pe_glu_act(int dtype, const void* gate_up, void* out, int n_rows,
   const int threads = 256;
   size_t blocks = (total + threads - 1) / threads;
   if (blocks > pe::kSMs * 16) blocks = pe::kSMs * 16;
-  if (dtype == PE_BF16 && inter % 8 == 0 && (uintptr_t)gate_up % 16 == 0 && (uintptr_t)out % 16 == 0) {
+  if (dtype == PE_BF16 && inter % 8 == 0 && (uintptr_t)gate_up % 16 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)bias % 16 == 0) {
     pe::GluEpilogue e = {kind, limit, alpha, bias};
     blocks = (total / 8 + threads - 1) / threads;
     if (blocks > pe::kSMs * 16) blocks = pe::kSMs * 16;

@@ -519,7 +519,7 @@ __global__ void qkv_rotate_append_kernel(QkvRotateArgs a) {
 // values.  The lane that holds features [8i, 8i + 8) of the first rotated half trades its values with the lane that holds
 // the matching features of the second half.  A block takes TPB tokens and has all their rows in flight before the first use.
 template <int TPB>
-__global__ void __launch_bounds__(256) qkv_rotate_append_halves_kernel(QkvRotateArgs a, int qk_warps) {
+__global__ void __launch_bounds__(256, TPB > 1 ? 5 : 1) qkv_rotate_append_halves_kernel(QkvRotateArgs a, int qk_warps) {
   typedef __nv_bfloat16 T;
   const int lane = threadIdx.x & 31;
   const int gw = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -530,135 +530,168 @@ __global__ void __launch_bounds__(256) qkv_rotate_append_halves_kernel(QkvRotate
   const int idx = (is_v ? gw - qk_warps : gw) * per_warp + sub;       // head among q|k, or value head
   const bool active = sub < per_warp && idx < (is_v ? a.n_kv_heads : a.n_heads + a.n_kv_heads);
   const bool is_q = !is_v && idx < a.n_heads;
+  const bool to_cache = active && !is_q && a.write_cache;
   const int kv_head = is_v ? idx : idx - a.n_heads;
-  const size_t row_off = is_v ? (size_t)(a.n_heads + a.n_kv_heads) * a.head_dim + (size_t)idx * D : (size_t)idx * D;
-  const int rot = is_v ? 0 : a.rotary_dim, half = rot >> 1, half_l = half >> 3;
-  const bool turns = active && 8 * li < rot;
-  const bool second = li >= half_l;
-  const int j = 8 * (second ? li - half_l : li);
-  const int partner = turns ? lane + (second ? -half_l : half_l) : lane;
-  const bool pow2 = (lph & (lph - 1)) == 0;
+  const int row_off = (is_v ? (a.n_heads + a.n_kv_heads) * a.head_dim + idx * D : idx * D) + 8 * li;
+  const int t0 = blockIdx.x * TPB;
+  // the batch description and the page table do not come from the kernel before this one; with one token a block they are
+  // fetched while it may still run
+  int pos0 = 0, page0 = -1, seq0 = 0;
+  auto find_page = [&](int t, int pos) -> int {
+    if (pos < 0 || pos / kPageTokens >= a.table_stride) return -1;
+    return a.page_table[(size_t)a.seq_slot[a.token_seq[t]] * a.table_stride + pos / kPageTokens];
+  };
+  if (TPB == 1 && t0 < a.n_tokens) {
+    pos0 = a.token_pos[t0];
+    if (to_cache) {
+      page0 = find_page(t0, pos0);
+      seq0 = a.token_seq[t0];
+    }
+  }
   float bv[8];
 #pragma unroll
   for (int e = 0; e < 8; ++e) bv[e] = 0.f;
   if (active && a.bias) {
-    const float4 b0 = *reinterpret_cast<const float4*>(a.bias + row_off + 8 * li), b1 = *reinterpret_cast<const float4*>(a.bias + row_off + 8 * li + 4);
+    const float4 b0 = *reinterpret_cast<const float4*>(a.bias + row_off), b1 = *reinterpret_cast<const float4*>(a.bias + row_off + 4);
     bv[0] = b0.x; bv[1] = b0.y; bv[2] = b0.z; bv[3] = b0.w; bv[4] = b1.x; bv[5] = b1.y; bv[6] = b1.z; bv[7] = b1.w;
-  }
-  // the batch description and the page table do not come from the kernel before this one
-  int poss[TPB], page[TPB], qend[TPB], qbeg[TPB];
-#pragma unroll
-  for (int i = 0; i < TPB; ++i) {
-    const int t = blockIdx.x * TPB + i;
-    poss[i] = 0; page[i] = -1; qend[i] = 0; qbeg[i] = 0;
-    if (t < a.n_tokens) {
-      poss[i] = a.token_pos[t];
-      if (active && !is_q && a.write_cache) {
-        const int b = a.token_seq[t];
-        const int slot = a.seq_slot[b];
-        qbeg[i] = a.seq_qstart[b];
-        qend[i] = a.seq_qstart[b + 1];
-        if (poss[i] >= 0 && poss[i] / kPageTokens < a.table_stride) page[i] = a.page_table[(size_t)slot * a.table_stride + poss[i] / kPageTokens];
-      }
-    }
   }
   pdl_wait_block();
   pdl_launch_dependents();
-  uint4 raws[TPB], mixed[TPB];
+  auto unpack = [&](const uint4& raw, float (&x)[8]) {
+    const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
 #pragma unroll
-  for (int i = 0; i < TPB; ++i) {
-    const int t = blockIdx.x * TPB + i;
-    raws[i] = mixed[i] = make_uint4(0, 0, 0, 0);
-    if (t < a.n_tokens && active) {
-      raws[i] = *reinterpret_cast<const uint4*>((const T*)a.qkv + (size_t)t * a.ld + row_off + 8 * li);
-      if (is_v && a.v_mix) mixed[i] = *reinterpret_cast<const uint4*>((const T*)a.v_mix + ((size_t)t * a.n_kv_heads + idx) * D + 8 * li);
+    for (int e = 0; e < 4; ++e) {
+      const float2 f = __bfloat1622float2(h2[e]);
+      x[2 * e] = f.x;
+      x[2 * e + 1] = f.y;
     }
-  }
-#pragma unroll
-  for (int i = 0; i < TPB; ++i) {
-    const int t = blockIdx.x * TPB + i;
-    if (t >= a.n_tokens) break;
-    const int pos = poss[i];
-    T* cache_row = nullptr;
-    if (active && !is_q && a.write_cache) {
-      if (pos < 0 || pos / kPageTokens >= a.table_stride) {
-        if (li == 0) report(a.status, kStatusPositionOutOfRange, t, pos, a.table_stride * kPageTokens);
-      } else if (page[i] < 0 || page[i] >= a.num_pages) {
-        if (li == 0) report(a.status, kStatusPageOutOfRange, t, page[i], a.num_pages);
-      } else {
-        T* base = (T*)(is_v ? a.v_pages : a.k_pages);
-        const int off = pos % kPageTokens;
-        T* head_row = base + (((size_t)page[i] * a.n_kv_heads + kv_head) * kPageTokens + off) * D;
-        cache_row = head_row + 8 * li;
-        if (t + 1 == qend[i] && off + 1 < kPageTokens && (off == 0 || qend[i] - qbeg[i] > 1)) {
-          uint4* r4 = reinterpret_cast<uint4*>(head_row + D);      // clear the rest of the page (see the first kernel)
-          const size_t n4 = (size_t)(kPageTokens - 1 - off) * D / 8;
-          for (size_t x = li; x < n4; x += lph) r4[x] = make_uint4(0, 0, 0, 0);
-        }
-      }
+  };
+  // where this lane's piece of token t goes in the cache (null: nowhere); clears the rest of a page where the first kernel does
+  auto cache_place = [&](int t, int pos, int page) -> T* {
+    if (!to_cache) return nullptr;
+    if (pos < 0 || pos / kPageTokens >= a.table_stride) {
+      if (li == 0) report(a.status, kStatusPositionOutOfRange, t, pos, a.table_stride * kPageTokens);
+      return nullptr;
     }
-    float x[8];
-    {
-      const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raws[i]);
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float2 f = __bfloat1622float2(h2[e]);
-        x[2 * e] = f.x + bv[2 * e];
-        x[2 * e + 1] = f.y + bv[2 * e + 1];
-      }
+    if (page < 0 || page >= a.num_pages) {
+      if (li == 0) report(a.status, kStatusPageOutOfRange, t, page, a.num_pages);
+      return nullptr;
     }
-    if (is_v) {       // (whole warps: nothing below shuffles across q|k and value warps)
-      if (a.v_mix) {
-        const __nv_bfloat162* m2 = reinterpret_cast<const __nv_bfloat162*>(&mixed[i]);
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float2 f = __bfloat1622float2(m2[e]);
-          x[2 * e] = (1.f - a.v_lambda) * x[2 * e] + a.v_lambda * f.x;
-          x[2 * e + 1] = (1.f - a.v_lambda) * x[2 * e + 1] + a.v_lambda * f.y;
-        }
-      }
-    } else {
-      float other[8];
-#pragma unroll
-      for (int e = 0; e < 8; ++e) other[e] = __shfl_sync(0xffffffffu, x[e], partner & 31);
-      bool ok = true;
-      if (turns) {
-        ok = pos >= 0 && pos < a.table_rows;
-        if (!ok && li == 0) report(a.status, kStatusPositionOutOfRange, t, pos, a.table_rows);
-        const int prow = ok ? pos : 0;
-        const float* cs = a.cos_table + (size_t)prow * half + j;     // the tables stay in L2
-        const float* sn = a.sin_table + (size_t)prow * half + j;
-        const float4 c0 = *reinterpret_cast<const float4*>(cs), c1 = *reinterpret_cast<const float4*>(cs + 4);
-        const float4 s0 = *reinterpret_cast<const float4*>(sn), s1 = *reinterpret_cast<const float4*>(sn + 4);
-        const float cv[8] = {c0.x, c0.y, c0.z, c0.w, c1.x, c1.y, c1.z, c1.w};
-        const float sv[8] = {s0.x, s0.y, s0.z, s0.w, s1.x, s1.y, s1.z, s1.w};
-#pragma unroll
-        for (int e = 0; e < 8; ++e) x[e] = second ? x[e] * cv[e] + other[e] * sv[e] : x[e] * cv[e] - other[e] * sv[e];
-      }
-      if (a.qk_unit) {
-        float ss = 0.f;
-#pragma unroll
-        for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
-        if (pow2) {
-          for (int o = lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-        } else {
-          float total = 0.f;
-          for (int l = 0; l < lph; ++l) total += __shfl_sync(0xffffffffu, ss, (sub * lph + l) & 31);
-          ss = total;
-        }
-        const float inv = rsqrtf(ss / (float)D + a.eps);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) x[e] *= inv;
-      }
-      if (!ok) continue;
+    const int off = pos % kPageTokens;
+    T* head_row = (T*)(is_v ? a.v_pages : a.k_pages) + (((size_t)page * a.n_kv_heads + kv_head) * kPageTokens + off) * D;
+    const int b = TPB == 1 ? seq0 : a.token_seq[t];
+    const int q_end = a.seq_qstart[b + 1];
+    if (t + 1 == q_end && off + 1 < kPageTokens && (off == 0 || q_end - a.seq_qstart[b] > 1)) {
+      uint4* r4 = reinterpret_cast<uint4*>(head_row + D);
+      const int n4 = (kPageTokens - 1 - off) * D / 8;
+      for (int x = li; x < n4; x += lph) r4[x] = make_uint4(0, 0, 0, 0);
     }
-    if (!active) continue;
+    return head_row + 8 * li;
+  };
+  auto pack = [&](const float (&x)[8]) -> uint4 {
     uint4 out;
     __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&out);
 #pragma unroll
     for (int e = 0; e < 4; ++e) o2[e] = __floats2bfloat162_rn(x[2 * e], x[2 * e + 1]);
-    if (!is_v) *reinterpret_cast<uint4*>((T*)a.qkv + (size_t)t * a.ld + row_off + 8 * li) = out;
-    else if (a.v_keep) *reinterpret_cast<uint4*>((T*)a.v_keep + ((size_t)t * a.n_kv_heads + idx) * D + 8 * li) = out;
+    return out;
+  };
+  uint4 raws[TPB];
+  int poss[TPB], pages[TPB];
+#pragma unroll
+  for (int i = 0; i < TPB; ++i) {
+    const int t = t0 + i;
+    raws[i] = make_uint4(0, 0, 0, 0);
+    poss[i] = pos0;
+    pages[i] = page0;
+    if (t < a.n_tokens) {
+      if (active) raws[i] = *reinterpret_cast<const uint4*>((const T*)a.qkv + (size_t)t * a.ld + row_off);
+      if (TPB > 1) {
+        poss[i] = a.token_pos[t];
+        if (to_cache) pages[i] = find_page(t, poss[i]);
+      }
+    }
+  }
+  if (is_v) {                               // (whole warps: nothing below shuffles across q|k and value warps)
+    const size_t v_off = (size_t)idx * D + 8 * li;
+    uint4 mixed[TPB];
+#pragma unroll
+    for (int i = 0; i < TPB; ++i) {
+      mixed[i] = make_uint4(0, 0, 0, 0);
+      if (active && a.v_mix && t0 + i < a.n_tokens)
+        mixed[i] = *reinterpret_cast<const uint4*>((const T*)a.v_mix + (size_t)(t0 + i) * a.n_kv_heads * D + v_off);
+    }
+    if (!active) return;
+#pragma unroll
+    for (int i = 0; i < TPB; ++i) {
+      const int t = t0 + i;
+      if (t >= a.n_tokens) break;
+      T* cache_row = cache_place(t, poss[i], pages[i]);
+      float x[8], f[8];
+      unpack(raws[i], x);
+      unpack(mixed[i], f);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        x[e] += bv[e];
+        if (a.v_mix) x[e] = (1.f - a.v_lambda) * x[e] + a.v_lambda * f[e];
+      }
+      const uint4 out = pack(x);
+      if (a.v_keep) *reinterpret_cast<uint4*>((T*)a.v_keep + (size_t)t * a.n_kv_heads * D + v_off) = out;
+      if (cache_row) *reinterpret_cast<uint4*>(cache_row) = out;
+    }
+    return;
+  }
+  const int rot = a.rotary_dim, half = rot >> 1, half_l = half >> 3;
+  const bool turns = active && 8 * li < rot;
+  const bool second = li >= half_l;
+  const int j = 8 * (second ? li - half_l : li);
+  const int partner = (turns ? lane + (second ? -half_l : half_l) : lane) & 31;
+  const float sign = second ? 1.f : -1.f;
+  const bool pow2 = (lph & (lph - 1)) == 0;
+#pragma unroll
+  for (int i = 0; i < TPB; ++i) {
+    const int t = t0 + i;
+    if (t >= a.n_tokens) break;
+    const int pos = poss[i];
+    float x[8];
+    unpack(raws[i], x);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[e] += bv[e];
+    bool ok = true;
+    if (rot > 0) {
+      ok = !turns || (pos >= 0 && pos < a.table_rows);
+      if (!ok && li == 0) report(a.status, kStatusPositionOutOfRange, t, pos, a.table_rows);
+      const size_t at = (size_t)(turns && ok ? pos : 0) * half + (turns ? j : 0);
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {        // the tables stay in L2
+        const float4 c = *reinterpret_cast<const float4*>(a.cos_table + at + 4 * h), s = *reinterpret_cast<const float4*>(a.sin_table + at + 4 * h);
+        const float cv[4] = {c.x, c.y, c.z, c.w}, sv[4] = {s.x, s.y, s.z, s.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float other = __shfl_sync(0xffffffffu, x[4 * h + e], partner);
+          const float y = fmaf(sign * sv[e], other, x[4 * h + e] * cv[e]);
+          x[4 * h + e] = turns ? y : x[4 * h + e];
+        }
+      }
+    }
+    if (a.qk_unit) {
+      float ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
+      if (pow2) {
+        for (int o = lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      } else {
+        float total = 0.f;
+        for (int l = 0; l < lph; ++l) total += __shfl_sync(0xffffffffu, ss, (sub * lph + l) & 31);
+        ss = total;
+      }
+      const float inv = rsqrtf(ss / (float)D + a.eps);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] *= inv;
+    }
+    T* cache_row = cache_place(t, pos, pages[i]);
+    if (!active || !ok) continue;
+    const uint4 out = pack(x);
+    *reinterpret_cast<uint4*>((T*)a.qkv + (size_t)t * a.ld + row_off) = out;
     if (cache_row) *reinterpret_cast<uint4*>(cache_row) = out;
   }
 }
@@ -893,7 +926,7 @@ extern "C" int pe_qkv_rotate_append(int dtype, void* qkv, long long ld, int n_to
     const int qk_warps = (n_heads + n_kv_heads + qk_per_warp - 1) / qk_per_warp;
     const int all_warps = qk_warps + (n_kv_heads + v_per_warp - 1) / v_per_warp;
     if (n_tokens >= 256) {
-      constexpr int kTokensPerBlock = 4;
+      constexpr int kTokensPerBlock = 2;   // (2,048 tokens, 16 + 4 heads of 128: 2 tokens 21.6 us, 3 23.8, 4 28.7, 8 38.0)
       dim3 g((n_tokens + kTokensPerBlock - 1) / kTokensPerBlock, (all_warps + 7) / 8);
       if (g.y > 65535) return PE_ERR_UNSUPPORTED_SIZE;
       pe::launch(pe::qkv_rotate_append_halves_kernel<kTokensPerBlock>, g, 256, 0, stream, a, qk_warps);

@@ -95,6 +95,13 @@ __global__ void __launch_bounds__(S >= 4 ? 512 : 1024) streams_vec4_kernel(Strea
 #pragma unroll
     for (int t = 0; t < S; ++t) mix[i][t] = a.y ? a.mix[i * S + t] : 0.f;
   }
+  // nor do the norm's weight and the bias: on their way to L2 (a decode step has streamed gigabytes of other weights through
+  // it since the last one) while that kernel may still be running; one request a 128-byte line
+  if (a.n_rows < kSMs && (threadIdx.x & 7) == 0)
+    for (int c = threadIdx.x * 4; c < a.width; c += blockDim.x * 4) {
+      if (a.w) asm volatile("prefetch.global.L2 [%0];\n" ::"l"(a.w + c));
+      if (a.bias && a.y) asm volatile("prefetch.global.L2 [%0];\n" ::"l"(a.bias + c));
+    }
   pdl_wait_block();
   pdl_launch_dependents();
   const int r = blockIdx.x;

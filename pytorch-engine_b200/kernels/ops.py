@@ -529,18 +529,27 @@ def gemm_umma2_qkv_rope(x: torch.Tensor, weight: torch.Tensor, qkv: torch.Tensor
                         cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rotary_dim: int, token_seq: torch.Tensor,
                         token_pos: torch.Tensor, seq_slot: torch.Tensor, seq_qstart: torch.Tensor,
                         page_table: Optional[torch.Tensor], num_pages: int, k_pages: Optional[torch.Tensor],
-                        v_pages: Optional[torch.Tensor], write_cache: bool, status: torch.Tensor) -> None:
+                        v_pages: Optional[torch.Tensor], write_cache: bool, status: torch.Tensor, bias: Optional[torch.Tensor] = None,
+                        qk_unit: bool = False, v_mix: Optional[torch.Tensor] = None, v_lambda: float = 0.0,
+                        v_keep: Optional[torch.Tensor] = None) -> None:
     """``x @ weight^T`` (the fused q|k|v projection) with what ``qk_norm_rope_append`` does in the product's epilogue:
-    ``qkv[:, :n_heads * head_dim]`` gets the normalised, rotated queries; keys and values go to the cache only."""
+    ``qkv[:, :n_heads * head_dim]`` gets the normalised, rotated queries; keys and values go to the cache only.
+    ``bias``, ``qk_unit``, ``v_mix``, ``v_lambda``, ``v_keep``: as for ``qkv_rotate_append`` (the rotation must leave lengths as they
+    are); weight rows behind q|k|v give the output's columns behind them."""
     _need(gemm_umma2_qkv_rope_supported(x, weight, n_heads, n_kv_heads, head_dim, rotary_dim if cos is not None else 0),
           "gemm_umma2_qkv_rope: needs bfloat16, head size 128, whole-head rotation, K % 64 == 0")
     _need(qkv.dtype == torch.bfloat16 and qkv.stride(-1) == 1 and qkv.shape[0] == x.shape[0], "gemm_umma2_qkv_rope: qkv rows")
-    _need(weight.shape[0] == (n_heads + 2 * n_kv_heads) * head_dim, "gemm_umma2_qkv_rope: weight rows")
+    extra = weight.shape[0] - (n_heads + 2 * n_kv_heads) * head_dim
+    _need(extra >= 0 and qkv.shape[1] >= weight.shape[0], "gemm_umma2_qkv_rope: weight rows")
+    _need(bias is None or (bias.dtype == torch.float32 and bias.numel() == weight.shape[0] - extra), "gemm_umma2_qkv_rope: bias")
+    for t in (v_mix, v_keep):
+        _need(t is None or (t.dtype == torch.bfloat16 and t.is_contiguous() and t.numel() >= x.shape[0] * n_kv_heads * head_dim),
+              "gemm_umma2_qkv_rope: v_mix and v_keep are [n, n_kv_heads * head_dim]")
     m, k = x.shape
-    check(library().pe_gemm_umma2_qkv_rope(
-        _ptr(x), x.stride(0), _ptr(weight), _ptr(qkv), qkv.stride(0), m, k, n_heads, n_kv_heads, head_dim,
+    check(library().pe_gemm_umma2_qkv_rope_ex(
+        _ptr(x), x.stride(0), _ptr(weight), _ptr(qkv), qkv.stride(0), m, k, n_heads, n_kv_heads, head_dim, extra,
         _ptr(q_norm_w), _ptr(k_norm_w), float(eps), _ptr(cos), _ptr(sin), rotary_dim if cos is not None else 0,
-        0 if cos is None else cos.shape[0], _ptr(token_seq), _ptr(token_pos), _ptr(seq_slot), _ptr(seq_qstart),
+        0 if cos is None else cos.shape[0], _ptr(bias), 1 if qk_unit else 0, _ptr(v_mix), float(v_lambda), _ptr(v_keep), _ptr(token_seq), _ptr(token_pos), _ptr(seq_slot), _ptr(seq_qstart),
         _ptr(page_table), 0 if page_table is None else page_table.shape[1], num_pages, _ptr(k_pages), _ptr(v_pages),
         1 if write_cache else 0, sm_count(x.device), _ptr(status), _stream()), "gemm_umma2_qkv_rope")
     _count(1)

@@ -182,8 +182,18 @@ class GQAttention:
         where = (ctx.token_seq, ctx.token_pos, ctx.seq_slot, ctx.seq_qstart, view.page_table, view.num_pages,
                  view.k_pages, view.v_pages)
         if self.general:
-            rt.linear(x, self.qkv, out=qkv)
-            self.rotate_append_general(qkv, n, ctx, view, writes_cache)
+            if self.fuses_general_into_product(x, rt):
+                # many rows: biases, unit norm, rotation, value mixing and the append ride in the product's epilogue
+                cos = sin = None
+                rotary_dim = 0
+                if self.position is not None:
+                    cos, sin, rotary_dim = self.position.tables()
+                ops.gemm_umma2_qkv_rope(x, self.qkv, qkv, self.n_heads, self.n_kv_heads, self.head_dim, self.q_norm, self.k_norm,
+                                        self.eps, cos, sin, rotary_dim, *where, writes_cache, rt.status, self.bias,
+                                        **self.value_options(n, ctx))
+            else:
+                rt.linear(x, self.qkv, out=qkv)
+                self.rotate_append_general(qkv, n, ctx, view, writes_cache)
             out = ctx.buffer("attn.out", (n, self.n_heads * self.v_dim), rt.dtype)
             self.attend_general(qkv, out, ctx, view)
             if self.output_gate == "sigmoid" or (self.output_gate and not self.gate_in_kernel(ctx)):
@@ -231,15 +241,29 @@ class GQAttention:
         if self.value_position is not None:
             vcos, vsin, vrot = self.value_position.tables()
             vinter = bool(getattr(self.value_position, "interleaved", False))
-        kept = None
-        if self.value_mix:
-            kept = ctx.buffer("attn.kept_values", (n, self.n_kv_heads * self.v_dim), self.runtime.dtype)
         ops.qkv_rotate_append(qkv, n, self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim, self.q_norm, self.k_norm,
                               self.eps, cos, sin, rot, inter, self.v_norm == "unit", vcos, vsin, vrot, vinter,
                               ctx.token_seq, ctx.token_pos, ctx.seq_slot, ctx.seq_qstart, view.page_table, view.num_pages,
-                              view.k_pages, view.v_pages, writes_cache, self.runtime.status, self.bias, qk_unit=self.qk_unit,
-                              v_mix=kept if self.value_mix == "mix" else None, v_lambda=self.v_lambda,
-                              v_keep=kept if self.value_mix == "keep" else None)
+                              view.k_pages, view.v_pages, writes_cache, self.runtime.status, self.bias,
+                              **self.value_options(n, ctx))
+
+    def value_options(self, n: int, ctx) -> dict:
+        kept = None
+        if self.value_mix:
+            kept = ctx.buffer("attn.kept_values", (n, self.n_kv_heads * self.v_dim), self.runtime.dtype)
+        return dict(qk_unit=self.qk_unit, v_mix=kept if self.value_mix == "mix" else None, v_lambda=self.v_lambda,
+                    v_keep=kept if self.value_mix == "keep" else None)
+
+    def fuses_general_into_product(self, x: torch.Tensor, rt) -> bool:
+        """``fuses_rope_into_product`` for the general path: values as large as keys, neither normed nor turned; split-half pairs;
+        with unit q and k a rotation that leaves lengths as they are, and not a norm with a weight as well."""
+        if self.v_dim != self.head_dim or self.v_norm or self.value_position is not None:
+            return False
+        if self.position is not None and getattr(self.position, "interleaved", False):
+            return False
+        if self.qk_unit and (self.q_norm is not None or (self.position is not None and not getattr(self.position, "keeps_lengths", False))):
+            return False
+        return self.fuses_rope_into_product(x, rt)
 
     def gate_columns(self, qkv: torch.Tensor) -> torch.Tensor:
         width = self.n_heads if self.output_gate == "sigmoid_head" else self.n_heads * self.v_dim

@@ -56,6 +56,7 @@ class RotaryPosition:
         if self.rotary_dim <= 0 or self.rotary_dim % 2:
             raise ValueError(f"rotary_dim must be positive and even, got {self.rotary_dim}")
         scaling = params.get("scaling")
+        self.keeps_lengths = not (scaling and "original" in scaling)   # cos and sin carry no factor
         mult = 1.0
         linear = 1.0
         if scaling and "original" not in scaling:

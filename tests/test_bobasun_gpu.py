@@ -283,10 +283,58 @@ def test_bias_rotation_unit_norm_mixed_values_and_the_append(pe, dtype, nh, nkv,
         assert status.tolist()[0] == 0
 
 
+@pytest.mark.parametrize("nh,nkv,extra,rot", [(4, 2, 8, 128), (3, 1, 0, 0), (6, 3, 16, 128), (2, 2, 264, 128)])
+def test_the_products_epilogue_does_what_the_separate_kernel_does(pe, nh, nkv, extra, rot):
+    """q|k|v|extra product with biases, rotation, unit norm, kept or mixed values and the append in its epilogue, against the
+    plain equations and (for every page and every column) the separate kernel behind the same product."""
+    ops = pe.kernels.ops
+    bf, d, K = torch.bfloat16, 128, 192
+    g = torch.Generator().manual_seed(nh + extra)
+    rt = pe.parts.Runtime(torch.device(DEV), bf)
+    cos = sin = None
+    if rot:
+        cos, sin, _ = pe.parts.lookup("position", "rope")({"rotary_dim": rot, "theta": 300.0, "max_positions": 900, "style": "neox",
+                                                           "scaling": {"factor": 2.5}, "exact": True}, {}, rt).tables()
+    lens, pasts = [300, 1, 70], [3, 64, 65]
+    n, feats = sum(lens), (nh + 2 * nkv) * d
+    x = torch.randn(n, K, generator=g).to(bf).to(DEV)
+    w = (torch.randn(feats + extra, K, generator=g) * 0.2).to(bf).to(DEV)
+    bias = torch.randn(feats, generator=g).to(DEV)
+    first = torch.randn(n, nkv * d, generator=g).to(bf).to(DEV)
+    qstart = torch.tensor([0, 300, 301, n], dtype=torch.int32, device=DEV)
+    seq = torch.tensor([b for b in range(3) for _ in range(lens[b])], dtype=torch.int32, device=DEV)
+    pos = torch.tensor([p + i for p, q in zip(pasts, lens) for i in range(q)], dtype=torch.int32, device=DEV)
+    slots = torch.arange(3, dtype=torch.int32, device=DEV)
+    status = torch.zeros(4, dtype=torch.int32, device=DEV)
+    for mode in ("keep", "mix"):
+        results = []
+        for fused in (True, False):
+            pages = Pages([p + q for p, q in zip(pasts, lens)], nkv, d, d, seed=1, fill=7.0)
+            kp, vp = pages.k.to(DEV, bf), pages.v.to(DEV, bf)
+            qkv = torch.zeros(n, feats + extra, dtype=bf, device=DEV)
+            kept = torch.zeros(n, nkv * d, dtype=bf, device=DEV)
+            where = (seq, pos, slots, qstart, pages.table.to(DEV), pages.n_pages, kp, vp)
+            more = dict(qk_unit=True, v_mix=first if mode == "mix" else None, v_lambda=0.3, v_keep=kept if mode == "keep" else None)
+            if fused:
+                ops.gemm_umma2_qkv_rope(x, w, qkv, nh, nkv, d, None, None, 0.01, cos, sin, rot, *where, True, status, bias, **more)
+            else:
+                ops.gemm_umma2(x, w, qkv, status)
+                ops.qkv_rotate_append(qkv, n, nh, nkv, d, d, None, None, 0.01, cos, sin, rot, False, False, None, None, 0, False, *where, True,
+                                      status, bias, **more)
+            results.append([t.float().cpu() for t in (qkv[:, :nh * d], qkv[:, feats:], kp, vp, kept)])
+        for a, b in zip(*results):
+            assert (a - b).abs().max() <= 2e-2 * max(float(b.abs().max()), 1e-3) if b.numel() else True
+        y = (x.double() @ w.double().T).cpu()
+        q = plain.unit(plain.rotate((y[:, :nh * d] + bias[:nh * d].double().cpu()).view(n, nh, d), pos.cpu(),
+                                    {"base": 300.0, "dims": rot, "scaling": {"factor": 2.5}} if rot else None), 0.01)
+        assert (results[0][0].double().view(n, nh, d) - q).abs().max() < 2e-2 * float(q.abs().max())
+    assert status.tolist()[0] == 0
+
+
 ATT_KERNELS = {"float32 arithmetic": [(3, 1, 14, 10), (6, 2, 72, 40)],
                "mma": [(4, 2, 64, 64), (8, 2, 128, 128), (6, 2, 72, 40), (4, 1, 8, 8), (3, 3, 24, 128), (5, 1, 136, 64), (16, 1, 192, 120),
                        (2, 2, 256, 16), (4, 4, 104, 72), (2, 1, 200, 128)],
-               "umma": [(8, 2, 128, 128), (4, 1, 72, 40), (6, 2, 120, 128), (5, 5, 128, 64), (20, 1, 104, 72), (3, 1, 80, 8)]}
+               "umma": [(8, 2, 128, 128), (4, 2, 192, 128), (7, 1, 136, 40), (2, 2, 256, 128), (6, 3, 200, 8), (4, 1, 72, 40), (6, 2, 120, 128), (5, 5, 128, 64), (20, 1, 104, 72), (3, 1, 80, 8)]}
 
 
 @pytest.mark.parametrize("kernel,nh,nkv,d,dv", [(k, *s) for k, shapes in ATT_KERNELS.items() for s in shapes])
@@ -702,6 +750,9 @@ def test_a_model_of_real_layer_sizes_takes_the_many_row_products(pe, models, dty
     eng = models.engine(key, dtype, max_context_len=1152, max_cache_tokens=64 * 20)
     eng.runtime.large_gemm_min_fill = 0.0
     toks = _tokens(96, 1032, 12)
+    if dtype == "bfloat16":
+        x = torch.empty(1030, 256, dtype=torch.bfloat16, device=DEV)
+        assert all(parts["mixer"].fuses_general_into_product(x, eng.runtime) for parts in eng.model.block_parts)
     positions = list(range(0, 1030, 23)) + [1029]
     s = eng.alloc_slot()
     rows = [eng.step([_entry(pe, s, toks[:1030], positions)]).clone()]
