@@ -602,11 +602,13 @@ __global__ void __launch_bounds__(128) decode_split_kernel(Args a, const __grid_
 }
 
 // grid: (n_heads, n_seqs): merge the ranges of one (sequence, head) (pygguf_engine/kv_cache.py:273-282).
+// VD: the size of a value row, 0: a.vd.  GATE: outputs may carry a gate (a.gate).
+template <int VD, bool GATE>
 __global__ void decode_merge_kernel(Args a) {
   pdl_wait_block();
   pdl_launch_dependents();
   const int b = blockIdx.y, h = blockIdx.x;
-  const int vd = a.vd;
+  const int vd = VD > 0 ? VD : a.vd;
   const int tq = a.seq_qstart[b];
   const int len = a.seq_past[b] + 1;
   const int per_range = range_keys(a, len);
@@ -624,7 +626,7 @@ __global__ void decode_merge_kernel(Args a) {
   const int kept_ranges = min((keep + per_range - 1) / per_range, first);
   const size_t base = ((size_t)b * a.n_heads + h) * a.max_splits;
   __nv_bfloat16* o = a.out + (size_t)tq * a.out_ld + (size_t)h * vd;
-  const float gate = a.gate ? gate_of(a, tq, h) : 1.f;
+  const float gate = GATE && a.gate ? gate_of(a, tq, h) : 1.f;
   // Ranges are taken eight at a time: all their loads are issued before the first is used (this kernel
   // is short and a decode step waits for it once per layer), then they are folded into a running
   // maximum, denominator and sum, in range order.
@@ -656,7 +658,8 @@ __global__ void decode_merge_kernel(Args a) {
       }
       mx = m_new;
     }
-    v = v / fmaxf(denom, 1e-20f) * gate;
+    v = v / fmaxf(denom, 1e-20f);
+    if (GATE) v *= gate;
     if (a.out_cos) {
       // features c and c ^ 1 (adjacent lanes) are one interleaved pair; every lane of the warp is here (turned outputs: 64 or 128
       // features)
@@ -726,7 +729,7 @@ static int launch(const Args& a, bool decode, int n_seqs, int max_q, cudaStream_
   // 1 to 64.  Why its waiting blocks cost that much is not known; switching the early start off for any
   // other kernel of the step gained nothing or lost.
   dim3 mgrid(a.n_heads, n_seqs);
-  pe::launch_after(decode_merge_kernel, mgrid, a.vd > 64 ? 128 : 64, 0, stream, a);
+  pe::launch_after(a.gate ? decode_merge_kernel<0, true> : decode_merge_kernel<PAD ? 0 : VD, false>, mgrid, a.vd > 64 ? 128 : 64, 0, stream, a);
   PE_LAUNCH_CHECK();
   return PE_OK;
 }

@@ -19,6 +19,7 @@
 // pygguf_engine/quant_kernels.py:1467-1472 (silu(gate) * up in float32).
 #include "api.h"
 #include "common.cuh"
+#include <type_traits>
 
 namespace pe {
 namespace smallm {
@@ -61,13 +62,15 @@ template <typename T> __device__ __forceinline__ void store_out(T* p, float v);
 template <> __device__ __forceinline__ void store_out<float>(float* p, float v) { *p = v; }
 template <> __device__ __forceinline__ void store_out<__nv_bfloat16>(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
 
-// NT: 8-row groups of activations (1: M <= 8, 2: M <= 16).  PAIR: two weight-row blocks per warp
-// (gate and up), combined as silu(gate) * up.  WARPS: warps per block = K slices.  U: k blocks per batch
+// NT: 8-row groups of activations (1: M <= 8, 2: M <= 16).  GLU != 0: two weight-row blocks per warp
+// (gate and up), combined as silu(gate) * up (1) or as Args::glu says (2; an instantiation of its own, so that the
+// usual one carries nothing of it).  WARPS: warps per block = K slices.  U: k blocks per batch
 // of loads.
 // Registers are capped at 128 per thread for M <= 8 so that 16 warps fit on an SM: what limits this
 // kernel is how many bytes its SM has in flight.  For M <= 16 that cap would spill.
-template <int NT, bool PAIR, int WARPS, int U, typename OutT>
+template <int NT, int GLU, int WARPS, int U, typename OutT>
 __global__ void __launch_bounds__(WARPS * 32, NT == 1 ? 16 / WARPS : 1) gemm_smallm_kernel(Args a) {
+  constexpr bool PAIR = GLU != 0;
   __shared__ float red[WARPS][(PAIR ? 2 : 1) * NT][4][32];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, t = lane & 3;
@@ -192,21 +195,25 @@ __global__ void __launch_bounds__(WARPS * 32, NT == 1 ? 16 / WARPS : 1) gemm_sma
       float v = c[n][e];
       if (PAIR) {
         float up = c[NT + n][e];
-        if (a.glu.bias) {
-          v += a.glu.bias[col];
-          up += a.glu.bias[a.N + col];
+        if (GLU == 1) {
+          v = sizeof(OutT) == 2 ? silu_mul_fast(v, up) : v / (1.0f + expf(-v)) * up;   // exact for a float32 result
+        } else {
+          if (a.glu.bias) {
+            v += a.glu.bias[col];
+            up += a.glu.bias[a.N + col];
+          }
+          v = sizeof(OutT) == 2 ? glu_fast(a.glu, v, up) : glu_exact(a.glu.kind, v, up, a.glu.limit, a.glu.alpha);
         }
-        v = sizeof(OutT) == 2 ? glu_fast(a.glu, v, up) : glu_exact(a.glu.kind, v, up, a.glu.limit, a.glu.alpha);   // exact for a float32 result
       }
       store_out<OutT>(y + (size_t)m * a.ldy + col, v);
     }
 }
 
-template <int NT, bool PAIR, typename OutT>
+template <int NT, int GLU, typename OutT>
 static int launch(const Args& a, int n_sms, cudaStream_t stream) {
   const int blocks = (a.N + 15) / 16;
   const int kblocks = (a.K + 31) / 32;
-  constexpr int U = PAIR ? 2 : 4;
+  constexpr int U = GLU ? 2 : 4;
   // K slices per block of 16 weight rows: enough warps in flight over the whole GPU to cover the
   // memory latency, but at least two batches of k blocks per warp.  An SM holds 16 warps of the
   // M <= 8 kernels (128 registers) and 12 of the M <= 16 kernels (up to 168 registers) as long as their
@@ -220,10 +227,10 @@ static int launch(const Args& a, int n_sms, cudaStream_t stream) {
   // (6144 x 4096 at 8 rows: 11.5 us with 8 warps a block, 1.3 waves; 10.2 us with 4).
   if (warps > 1 && (long long)blocks * warps > slots && (long long)blocks * warps * 2 <= slots * 3) warps /= 2;
   switch (warps) {
-    case 1: pe::launch(gemm_smallm_kernel<NT, PAIR, 1, U, OutT>, blocks, 32, 0, stream, a); break;
-    case 2: pe::launch(gemm_smallm_kernel<NT, PAIR, 2, U, OutT>, blocks, 64, 0, stream, a); break;
-    case 4: pe::launch(gemm_smallm_kernel<NT, PAIR, 4, U, OutT>, blocks, 128, 0, stream, a); break;
-    default: pe::launch(gemm_smallm_kernel<NT, PAIR, 8, U, OutT>, blocks, 256, 0, stream, a); break;
+    case 1: pe::launch(gemm_smallm_kernel<NT, GLU, 1, U, OutT>, blocks, 32, 0, stream, a); break;
+    case 2: pe::launch(gemm_smallm_kernel<NT, GLU, 2, U, OutT>, blocks, 64, 0, stream, a); break;
+    case 4: pe::launch(gemm_smallm_kernel<NT, GLU, 4, U, OutT>, blocks, 128, 0, stream, a); break;
+    default: pe::launch(gemm_smallm_kernel<NT, GLU, 8, U, OutT>, blocks, 256, 0, stream, a); break;
   }
   PE_LAUNCH_CHECK();
   return PE_OK;
@@ -259,13 +266,14 @@ extern "C" int pe_gemm_smallm_glu(const void* x, long long ldx, const void* w, v
   a.group_rows = 0; a.x_group_stride = 0;
   using namespace pe::smallm;
   if (n_sms <= 0) n_sms = pe::kSMs;
-  const bool pair = pair_offset > 0;
-  if (M <= 8) {
-    if (pair) return out_f32 ? launch<1, true, float>(a, n_sms, stream) : launch<1, true, __nv_bfloat16>(a, n_sms, stream);
-    return out_f32 ? launch<1, false, float>(a, n_sms, stream) : launch<1, false, __nv_bfloat16>(a, n_sms, stream);
-  }
-  if (pair) return out_f32 ? launch<2, true, float>(a, n_sms, stream) : launch<2, true, __nv_bfloat16>(a, n_sms, stream);
-  return out_f32 ? launch<2, false, float>(a, n_sms, stream) : launch<2, false, __nv_bfloat16>(a, n_sms, stream);
+  const int mode = pair_offset <= 0 ? 0 : (kind == 1 && bias == nullptr ? 1 : 2);
+  auto go = [&](auto nt) -> int {
+    constexpr int NT = decltype(nt)::value;
+    if (mode == 0) return out_f32 ? launch<NT, 0, float>(a, n_sms, stream) : launch<NT, 0, __nv_bfloat16>(a, n_sms, stream);
+    if (mode == 1) return out_f32 ? launch<NT, 1, float>(a, n_sms, stream) : launch<NT, 1, __nv_bfloat16>(a, n_sms, stream);
+    return out_f32 ? launch<NT, 2, float>(a, n_sms, stream) : launch<NT, 2, __nv_bfloat16>(a, n_sms, stream);
+  };
+  return M <= 8 ? go(std::integral_constant<int, 1>()) : go(std::integral_constant<int, 2>());
 }
 
 // Several projections of several inputs in one launch: w holds `groups` matrices of `group_rows` rows stacked
@@ -286,6 +294,6 @@ extern "C" int pe_gemm_smallm_grouped(const void* x, long long ldx, long long x_
   a.group_rows = group_rows; a.x_group_stride = x_group_stride;
   using namespace pe::smallm;
   if (n_sms <= 0) n_sms = pe::kSMs;
-  if (M <= 8) return out_f32 ? launch<1, false, float>(a, n_sms, stream) : launch<1, false, __nv_bfloat16>(a, n_sms, stream);
-  return out_f32 ? launch<2, false, float>(a, n_sms, stream) : launch<2, false, __nv_bfloat16>(a, n_sms, stream);
+  if (M <= 8) return out_f32 ? launch<1, 0, float>(a, n_sms, stream) : launch<1, 0, __nv_bfloat16>(a, n_sms, stream);
+  return out_f32 ? launch<2, 0, float>(a, n_sms, stream) : launch<2, 0, __nv_bfloat16>(a, n_sms, stream);
 }
