@@ -33,7 +33,7 @@ def _layer(mixer, ff=None, limit=1.0):
 # B: sizes that the tensor-core attention kernels take whole (64 and 128, the latter on tcgen05 in prompts), a feed-forward
 # that the fused gate|up product takes, two streams, every layer mixes.  C: key and value sizes that run in padded tiles
 # (below and above 64, 128 and 192), one stream, groups of 8 and 1, scale one.  D: small sizes in steps of 8, four streams, no
-# mixing layer but one, nine streams' worth of nothing else.  E: nine streams (the kernel without a fixed number of them).
+# mixing layer but one.  E: nine streams (the kernel without a fixed number of them).
 CONFIGS = {
     "A": {"architecture": "Bobasun", "vocab": 131, "width": 54, "streams": 5, "norm": {"eps": 2e-5}, "embedding": {"scale": 3.0},
           "layers": [_layer(_att(3, 1, 14, 10, 0.4, 6, 100.0, 4.0), 37, 1.5), _layer(_att(4, 2, 10, 6, 0.5, mix=True)),
