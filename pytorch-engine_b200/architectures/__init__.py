@@ -1,5 +1,5 @@
 """Architectures known to the registry.  Each module turns a typed configuration into a plan of
 parts and registers itself under the name that ``config.json`` carries in ``architectures[0]``."""
-from . import bobasun, lunadra, qwen3, vabelorn, vemepel, zonevik  # noqa: F401
+from . import bobasun, burinex, lunadra, qwen3, vabelorn, vemepel, zonevik  # noqa: F401
 
-__all__ = ["bobasun", "lunadra", "qwen3", "vabelorn", "vemepel", "zonevik"]
+__all__ = ["bobasun", "burinex", "lunadra", "qwen3", "vabelorn", "vemepel", "zonevik"]

@@ -26,7 +26,7 @@ int pe_attention_generic_ex(int dtype, int decode, const void* q, long long q_ld
     cudaStream_t stream);
 int pe_attention_generic_masked(int dtype, int decode, const void* q, long long q_ld, void* out, long long out_ld,
     int n_seqs, int max_q, int n_heads, int n_kv_heads, int head_dim, int v_dim, float scale, int window, int chunk,
-    int keep_first, int v_ld, int v_heads, int out_f32, int sink, const float* out_cos, const float* out_sin, int out_rot, int out_rows, int out_inter,
+    int keep_first, int v_ld, int v_heads, int out_f32, int sink, const float* sinks, const float* out_cos, const float* out_sin, int out_rot, int out_rows, int out_inter,
     const int* seq_qstart, const int* seq_past, const int* seq_slot, const int* page_table, int table_stride,
     int num_pages, const void* k_pages, const void* v_pages, float* scratch, int split_keys, int max_splits, int* status,
     cudaStream_t stream);
@@ -67,7 +67,7 @@ int pe_attention_mma_gated(int decode, const void* q, long long q_ld, void* out,
 // attention_latent.cu
 int pe_attention_latent_supported(int row, int rank);
 int pe_attention_latent(int decode, const void* q, long long q_ld, void* out, long long out_ld, int n_seqs, int max_q,
-    int n_heads, int row, int rank, float scale, const int* seq_qstart, const int* seq_past, const int* seq_slot,
+    int n_heads, int row, int rank, float scale, int window, const float* sinks, const int* seq_qstart, const int* seq_past, const int* seq_slot,
     const int* page_table, int table_stride, int num_pages, const void* pages, float* scratch, int split_keys,
     int max_splits, int min_range_keys, int* status, cudaStream_t stream);
 
@@ -107,7 +107,7 @@ int pe_rows_to_pages(int dtype, const void* src, long long src_ld, int col0, int
 int pe_rows_to_pages_pair(int dtype, const void* src, long long src_ld, int col0, int heads, int dim, int col0_b, int heads_b,
     int dim_b, int n_tokens, const int* token_seq, const int* token_pos, const int* seq_slot, const int* page_table,
     int table_stride, int num_pages, void* pages, void* pages_b, int* status, cudaStream_t stream);
-int pe_latent_prepare(int dtype, const void* x, long long x_ld, int q_col0, int low_col0, int heads, int d, int dr,
+int pe_latent_prepare(int dtype, const void* q, long long q_ld, const void* low, long long low_ld, int heads, int d, int dr,
     int rank, const float* norm_w, float eps, const float* cos_t, const float* sin_t, int rot, int table_rows,
     int n_tokens, const int* token_seq, const int* token_pos, const int* seq_slot, const int* page_table,
     int table_stride, int num_pages, void* pages, void* qfull, const void* absorbed, int write_cache, int* status,
@@ -118,6 +118,7 @@ int pe_embed_gather(int dtype, const void* table, const int* ids, float* out, in
     int* status, cudaStream_t stream);
 int pe_embed_gather_scaled(int dtype, const void* table, const int* ids, float* out, int n_tokens, int hidden, int vocab,
     float scale, float* copy, int* status, cudaStream_t stream);
+int pe_softcap(float* x, long long n, float scale, float cap, cudaStream_t stream);
 
 // gemm_smallm.cu
 int pe_gemm_smallm_supported(int M, int N, int K);
@@ -162,6 +163,10 @@ int pe_rmsnorm_residual(int dtype, float* residual, const void* delta, const flo
     const int* rows, int n_rows, int dim, float eps, cudaStream_t stream);
 int pe_rmsnorm(int dtype, const void* x, const float* weight, void* out, int n_rows, int dim, float eps,
     cudaStream_t stream);
+int pe_rmsnorm_rows(int dtype, const void* x, long long x_ld, const float* weight, void* out, int n_rows, int dim, float eps,
+    cudaStream_t stream);
+int pe_rmsnorm_of_sum(int dtype, float* stream, const void* delta, float alpha, const float* scale, const float* weight,
+    void* cast, int n_rows, int dim, float eps, cudaStream_t stream_);
 int pe_rmsnorm_add(int dtype, float* stream, const void* delta, const float* weight, void* cast, int n_rows, int dim,
     float eps, cudaStream_t stream_);
 
@@ -180,6 +185,11 @@ int pe_qkv_rotate_append(int dtype, void* qkv, long long ld, int n_tokens, int n
     const int* seq_slot, const int* seq_qstart, const int* page_table, int table_stride, int num_pages, void* k_pages,
     void* v_pages, int write_cache, const float* bias, int qk_unit, const void* v_mix, float v_lambda, void* v_keep,
     int* status, cudaStream_t stream);
+int pe_qkv_row_norm_append(int dtype, void* qkv, long long ld, int n_tokens, int n_heads, int n_kv_heads, int head_dim,
+    int v_dim, const float* q_norm_w, const float* k_norm_w, float eps, float temp_coef, int temp_every,
+    const float* cos_table, const float* sin_table, int rotary_dim, int table_rows, int interleaved, const int* token_seq,
+    const int* token_pos, const int* seq_slot, const int* seq_qstart, const int* page_table, int table_stride, int num_pages,
+    void* k_pages, void* v_pages, int write_cache, int* status, cudaStream_t stream);
 
 // streams.cu
 int pe_stream_mix(int dtype, const float* single, float* x, const void* y, const float* bias, const float* mix,
@@ -246,16 +256,16 @@ int pe_moe_route_logits(const float* logits, const float* bias, int n_tokens, in
 int pe_moe_route_sigmoid_groups(const float* logits, int n_tokens, int n_all, int top, int n_groups, int keep, int* chosen,
     float* weight, int* dense_rows, int n_real, cudaStream_t stream);
 int pe_moe_group(const int* chosen, int n_tokens, int top, int n_real, int* offsets, int* row_token, int* pair_row,
-    cudaStream_t stream);
+    const float* weight, float* row_weight, cudaStream_t stream);
 int pe_moe_rows_gemm(int dtype, int out_dtype, const void* x, long long x_ld, const int* row_map, const int* offsets,
     int n_groups, int max_rows, const void* w, long long w_group_stride, void* out, long long out_ld, int n_out, int k_dim,
-    int glu, float limit, float alpha, cudaStream_t stream);
+    int glu, float limit, float alpha, const float* row_weight, cudaStream_t stream);
 int pe_moe_gather_rows(int dtype, const void* x, const int* row_token, const int* offsets, int n_groups, void* xs,
     int max_rows, int width, cudaStream_t stream);
 int pe_moe_combine(int dtype, const void* rows, const void* x, const void* shared, const int* pair_row,
     const float* weight, int top, void* out, int n_tokens, int width, cudaStream_t stream);
 int pe_glu_act(int dtype, const void* gate_up, void* out, int n_rows, int inter, int kind, float limit, float alpha,
-    const float* bias, cudaStream_t stream);
+    const float* bias, const float* row_weight, const int* chosen, const float* weight, int top, int n_real, cudaStream_t stream);
 
 // ssd.cu
 int pe_ssd_recurrence(int dtype, const void* xbc, long long xbc_ld, const void* dt, long long dt_ld, const float* dt_bias,
@@ -264,7 +274,10 @@ int pe_ssd_recurrence(int dtype, const void* xbc, long long xbc_ld, const void* 
     cudaStream_t stream);
 long long pe_ssd_scratch_floats(int n_seqs, int heads, int n, int dv, int max_chunks);
 int pe_gated_part_norm(int dtype, const float* y, const void* z, long long z_ld, const float* w, float eps, void* out,
-    int n_tokens, int width, int parts, cudaStream_t stream);
+    int n_tokens, int width, int parts, int gate_first, cudaStream_t stream);
+int pe_lightning_recurrence(int dtype, const void* qkv, long long ld, const float* decay, const float* log_decay, float* y,
+    float* S, const int* seq_slot, const int* seq_qstart, int n_seqs, int max_q, int heads, int n, int dv, int n_slots, int chunk,
+    int max_chunks, float* scratch, int* status, cudaStream_t stream);
 
 // dyt.cu
 int pe_dyt(int dtype, int in_f32, const void* x, const int* rows, const float* w, const float* b, float alpha, void* out,

@@ -53,7 +53,11 @@ struct AttnArgs {
                                       //   maps over one set of values)
   int out_f32;                        // != 0: `out` is float32 whatever the inputs' type (not with a turned output)
   int keep_first;                     // > 0: with a window, keys at positions < keep_first stay visible to every later query
+  const float* sinks;                 // [n_heads] with sink != 0: the score of each head's sink (null: 0); not scaled
 };
+
+// The score of head h's sink.
+__device__ __forceinline__ float sink_score(const AttnArgs& a, int h) { return a.sinks ? a.sinks[h] : 0.f; }
 
 // First visible key of a query at `qpos` under the window and chunk masks.
 __device__ __forceinline__ int first_visible(const AttnArgs& a, int qpos) {
@@ -219,8 +223,8 @@ __global__ void __launch_bounds__(256) attn_prefill_kernel(AttnArgs a) {
 #pragma unroll
   for (int h = 0; h < kGT; ++h) {
     if (h >= n_here) continue;
-    // the sink: a key of score 0 that every query sees and that carries no value
-    const float denom = l[h] + (a.sink ? expf(-m[h]) : 0.f);
+    // the sink: a key of a score of its own that every query sees and that carries no value
+    const float denom = l[h] + (a.sink ? expf(sink_score(a, h0 + h) - m[h]) : 0.f);
     const float inv = 1.f / fmaxf(denom, 1e-20f);
     T* o = (T*)a.out + (size_t)(q0 + my_row) * a.out_ld + (size_t)(h0 + h) * dv;
     if (a.out_cos) {
@@ -359,12 +363,13 @@ __global__ void attn_decode_combine_kernel(AttnArgs a) {
   const int keep = a.keep_first > 0 ? min(a.keep_first, win_lo) : 0;
   const int kept_ranges = min((keep + a.split_keys - 1) / a.split_keys, first);
   const size_t base = ((size_t)b * a.n_heads + h) * a.max_splits;
-  float mx = a.sink ? 0.f : -INFINITY;   // the sink is one more range whose log-sum is 0 and whose output is 0
+  const float sink = a.sink ? sink_score(a, h) : -INFINITY;
+  float mx = sink;                       // the sink is one more range whose log-sum is its score and whose output is 0
   for (int s = 0; s < n_splits; ++s) {
     if (s >= kept_ranges && s < first) continue;
     mx = fmaxf(mx, a.part_lse[base + s]);
   }
-  float denom = a.sink ? expf(-mx) : 0.f;
+  float denom = a.sink ? expf(sink - mx) : 0.f;
   for (int s = 0; s < n_splits; ++s) {
     if (s >= kept_ranges && s < first) continue;
     const float e = a.part_lse[base + s];
@@ -487,7 +492,7 @@ extern "C" int pe_attention_generic_ex(int dtype, int decode, const void* q, lon
                                        int num_pages, const void* k_pages, const void* v_pages, float* scratch,
                                        int split_keys, int max_splits, int* status, cudaStream_t stream) {
   return pe_attention_generic_masked(dtype, decode, q, q_ld, out, out_ld, n_seqs, max_q, n_heads, n_kv_heads, head_dim,
-                                     v_dim, scale, window, 0, 0, v_dim, n_kv_heads, 0, sink, out_cos, out_sin, out_rot, out_rows,
+                                     v_dim, scale, window, 0, 0, v_dim, n_kv_heads, 0, sink, nullptr, out_cos, out_sin, out_rot, out_rows,
                                      out_inter, seq_qstart, seq_past, seq_slot, page_table, table_stride, num_pages,
                                      k_pages, v_pages, scratch, split_keys, max_splits, status, stream);
 }
@@ -495,11 +500,12 @@ extern "C" int pe_attention_generic_ex(int dtype, int decode, const void* q, lon
 // The same with a chunk mask (`chunk` > 0: keys inside the query's own block of that many positions), kept first keys
 // (`keep_first` > 0 with a window: positions below it stay visible however far back they lie), value rows
 // `v_ld` elements apart (>= v_dim), `v_heads` value heads a page (kv head g reads value head g % v_heads), and
-// optionally a float32 output (`out_f32`: out_ld then counts floats).
+// optionally a float32 output (`out_f32`: out_ld then counts floats).  `sinks` [n_heads] (with `sink` != 0): the score of each
+// head's sink; null: 0.
 extern "C" int pe_attention_generic_masked(int dtype, int decode, const void* q, long long q_ld, void* out, long long out_ld,
                                            int n_seqs, int max_q, int n_heads, int n_kv_heads, int head_dim, int v_dim,
                                            float scale, int window, int chunk, int keep_first, int v_ld, int v_heads, int out_f32,
-                                           int sink,
+                                           int sink, const float* sinks,
                                            const float* out_cos, const float* out_sin, int out_rot, int out_rows,
                                            int out_inter, const int* seq_qstart, const int* seq_past, const int* seq_slot,
                                            const int* page_table, int table_stride, int num_pages, const void* k_pages,
@@ -513,6 +519,7 @@ extern "C" int pe_attention_generic_masked(int dtype, int decode, const void* q,
   pe::AttnArgs a;
   a.keep_first = window > 0 ? keep_first : 0;
   a.chunk = chunk; a.v_ld = v_ld; a.v_heads = v_heads; a.out_f32 = out_f32;
+  a.sinks = sink ? sinks : nullptr;
   a.v_dim = v_dim; a.sink = sink; a.out_cos = out_cos; a.out_sin = out_sin;
   a.out_rot = out_cos ? out_rot : 0; a.out_rows = out_rows; a.out_inter = out_inter;
   a.q = q; a.q_ld = q_ld; a.out = out; a.out_ld = out_ld;
@@ -588,7 +595,7 @@ extern "C" int pe_attention_decode_noalloc(int dtype, const void* q, long long q
   a.page_table = page_table; a.table_stride = table_stride; a.num_pages = num_pages;
   a.k_pages = k_pages; a.v_pages = v_pages; a.status = status;
   a.split_keys = split_keys; a.max_splits = max_splits;
-  a.chunk = 0; a.v_ld = head_dim; a.v_heads = n_kv_heads; a.out_f32 = 0; a.keep_first = 0;
+  a.chunk = 0; a.v_ld = head_dim; a.v_heads = n_kv_heads; a.out_f32 = 0; a.keep_first = 0; a.sinks = nullptr;
   a.v_dim = head_dim; a.sink = 0; a.out_cos = nullptr; a.out_sin = nullptr; a.out_rot = 0; a.out_rows = 0; a.out_inter = 0;
   a.part_acc = scratch;
   a.part_lse = scratch + (size_t)n_seqs * n_heads * max_splits * head_dim;

@@ -1,8 +1,11 @@
 // Causal attention of many query heads over ONE cached row per position whose leading features are also
 // the values (a latent cache: the row is [latent | rotated key part], the value is the latent), on the
-// tensor cores (mma.sync m16n8k16, bfloat16 operands, float32 accumulation).  Rows of up to 576 features
-// in steps of 64; values of 128, 256 or 512 features.  Other shapes and the float32 mode use
-// attention_generic.cu (same arguments: one kv head, v_ld = row).
+// tensor cores (mma.sync m16n8k16, bfloat16 operands, float32 accumulation).  Rows of up to 576 features and
+// values of up to 512, both in steps of 8; on chip a row is padded to a multiple of 64 and a value to 64, 128, 256 or 512
+// features (TMA fills what lies beyond a row with zeros; what lies beyond a value is computed and not stored).  Other
+// shapes and the float32 mode use attention_generic.cu (same arguments: one kv head, v_ld = row).  Optionally a sliding
+// window (a query sees itself and the window - 1 positions before it; pages in front of it are never loaded) and one sink
+// per head (a term exp(score) in the denominator that has no key and no value).
 //
 // Scores, the softmax state (m, l) and the output accumulator are float32.  The tensor cores take bfloat16
 // operands, so each probability enters the P.V product as the sum of two bfloat16 terms (its rounding and
@@ -34,8 +37,11 @@ constexpr int BN = 64;  // keys per tile = one cache page
 
 struct Args {
   const __nv_bfloat16* q; long long q_ld;   // token t, head h: q + t * q_ld + h * row
-  __nv_bfloat16* out;     long long out_ld; // token t, head h: out + t * out_ld + h * RANK
-  int n_heads, row;
+  __nv_bfloat16* out;     long long out_ld; // token t, head h: out + t * out_ld + h * rank
+  int n_heads, row, rank;
+  int row_pad;                              // features of a row on chip: a multiple of 64, at least the padded value size
+  int window;                               // <= 0: none
+  const float* sinks;                       // [n_heads] scores (natural units, not scaled), or null
   float scale_log2;                         // softmax scale * log2(e)
   const int* seq_qstart; const int* seq_past; const int* seq_slot;
   const int* page_table; int table_stride; int num_pages;
@@ -90,8 +96,8 @@ __device__ __forceinline__ void issue_page(const Args& a, const CUtensorMap* map
     report(a.status, kStatusPageOutOfRange, slot, page, k0);
     page = 0;
   }
-  tma::mbar_expect_tx(bar, BN * a.row * 2);
-  for (int sub = 0; sub < a.row / 64; ++sub) tma::load_2d(stage + sub * (BN * 128), map, sub * 64, page * BN, bar);
+  tma::mbar_expect_tx(bar, BN * a.row_pad * 2);
+  for (int sub = 0; sub < a.row_pad / 64; ++sub) tma::load_2d(stage + sub * (BN * 128), map, sub * 64, page * BN, bar);
 }
 
 // A wait ran out: record it, give copies still in flight a last bounded chance to land, and leave.
@@ -106,7 +112,10 @@ __device__ __forceinline__ char* align_1024(char* p) {
   return reinterpret_cast<char*>((reinterpret_cast<uintptr_t>(p) + 1023) & ~static_cast<uintptr_t>(1023));
 }
 
-// Keys per range of a sequence of `len` keys (decode): the fixed split_keys, or (split_keys == 0) the sequence's
+// First visible key of a query at `pos`.
+__device__ __forceinline__ int first_visible(const Args& a, int pos) { return a.window > 0 ? max(0, pos - a.window + 1) : 0; }
+
+// Keys per range of a sequence that sees `len` keys (decode): the fixed split_keys, or (split_keys == 0) the sequence's
 // own length shared out evenly over max_splits ranges, in whole pages, but no fewer than min_range_keys.
 __device__ __forceinline__ int range_keys(const Args& a, int len) {
   if (a.split_keys > 0) return a.split_keys;
@@ -115,7 +124,7 @@ __device__ __forceinline__ int range_keys(const Args& a, int len) {
 }
 
 template <int MB, int KS>
-constexpr size_t smem_bytes(int row) {
+constexpr size_t smem_bytes(int row) {   // row: padded
   // two stages, the queries, both terms of P, and the exchanged row maxima and denominators
   return (size_t)2 * BN * row * 2 + (size_t)MB * 16 * row * 2 + (size_t)2 * MB * 16 * 128 + (size_t)2 * KS * MB * 16 * 4 + 1024;
 }
@@ -134,7 +143,7 @@ __global__ void __launch_bounds__(MB * KS * 32, 1) latent_kernel(Args a, const _
   constexpr int NO = DW / 8;          // their n-tiles
   constexpr int THREADS = MB * KS * 32;
   static_assert(NT >= 2 && NT % 2 == 0 && NO % 2 == 0, "warps take pairs of n-tiles");
-  const int row = a.row;
+  const int row = a.row_pad;
   const int stage_bytes = BN * row * 2;
   char* smem = align_1024(smem_raw);
   char* q_s = smem + 2 * stage_bytes;                         // [M][row] swizzled
@@ -155,11 +164,13 @@ __global__ void __launch_bounds__(MB * KS * 32, 1) latent_kernel(Args a, const _
   int k_lo = 0, k_hi;
   if (DECODE) {
     const int len = past + 1;
-    const int per_range = range_keys(a, len);
-    k_lo = (int)blockIdx.x * per_range;
+    const int k_first = first_visible(a, past) / BN * BN;     // ranges start at the first page that is seen
+    const int per_range = range_keys(a, len - k_first);
+    k_lo = k_first + (int)blockIdx.x * per_range;
     k_hi = min(len, k_lo + per_range);
     if (k_lo >= len) return;
   } else {
+    k_lo = first_visible(a, past + row0 / nh) / BN * BN;
     k_hi = past + (min(n_rows, row0 + M) - 1) / nh + 1;       // the block's last row sees keys up to its own position
   }
   const int slot = a.seq_slot[b];
@@ -178,13 +189,15 @@ __global__ void __launch_bounds__(MB * KS * 32, 1) latent_kernel(Args a, const _
     const int r = i / cpr, chunk = i - r * cpr;
     const int rr = row0 + r;
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (rr < n_rows) v = *reinterpret_cast<const uint4*>(a.q + (size_t)(q0 + rr / nh) * a.q_ld + (size_t)(rr % nh) * row + chunk * 8);
+    if (rr < n_rows && chunk * 8 < a.row)
+      v = *reinterpret_cast<const uint4*>(a.q + (size_t)(q0 + rr / nh) * a.q_ld + (size_t)(rr % nh) * a.row + chunk * 8);
     *reinterpret_cast<uint4*>(q_s + tile_off(r, chunk, M)) = v;
   }
   __syncthreads();
   // this thread's two rows and their positions (rows beyond n_rows are never stored)
   const int r_lo = row0 + rb * 16 + g, r_hi = r_lo + 8;
-  const int pos_lo = past + r_lo / nh, pos_hi = past + r_hi / nh;
+  const int pos_lo = DECODE ? past : past + r_lo / nh, pos_hi = DECODE ? past : past + r_hi / nh;
+  const int from_lo = first_visible(a, pos_lo), from_hi = first_visible(a, pos_hi);
   float o[NO][4];
 #pragma unroll
   for (int n = 0; n < NO; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
@@ -227,7 +240,7 @@ __global__ void __launch_bounds__(MB * KS * 32, 1) latent_kernel(Args a, const _
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int kpos = k0 + ks * KW + n * 8 + 2 * t + (e & 1);
-        const bool vis = DECODE ? (kpos < k_hi) : (kpos <= ((e < 2) ? pos_lo : pos_hi));
+        const bool vis = (DECODE ? (kpos < k_hi) : (kpos <= ((e < 2) ? pos_lo : pos_hi))) && kpos >= ((e < 2) ? from_lo : from_hi);
         const float v = vis ? s[n][e] * a.scale_log2 : -INFINITY;
         s[n][e] = v;
         if (e < 2) mx_lo = fmaxf(mx_lo, v); else mx_hi = fmaxf(mx_hi, v);
@@ -318,35 +331,36 @@ __global__ void __launch_bounds__(MB * KS * 32, 1) latent_kernel(Args a, const _
     const int rr = half ? r_hi : r_lo;
     if (rr >= n_rows) continue;
     const int tok = rr / nh, head = rr % nh;
-    const float lt = half ? lt_hi : lt_lo, mm = half ? m_hi : m_lo;
+    float lt = half ? lt_hi : lt_lo;
+    const float mm = half ? m_hi : m_lo;
+    if (!DECODE && a.sinks) lt += fast_exp2(a.sinks[head] * 1.4426950408889634f - mm);   // (decode: the merge adds it)
     const float inv = (lt > 0.f) ? 1.f / lt : 0.f;
     if (DECODE) {
       const size_t pidx = ((size_t)b * nh + head) * a.max_splits + blockIdx.x;
-      float* dst = a.part_acc + pidx * RANK + ks * DW;
+      float* dst = a.part_acc + pidx * a.rank + ks * DW;
 #pragma unroll
       for (int n = 0; n < NO; ++n)
-        *reinterpret_cast<float2*>(dst + n * 8 + 2 * t) = make_float2(o[n][half * 2] * inv, o[n][half * 2 + 1] * inv);
+        if (ks * DW + n * 8 < a.rank) *reinterpret_cast<float2*>(dst + n * 8 + 2 * t) = make_float2(o[n][half * 2] * inv, o[n][half * 2 + 1] * inv);
       // log-sum-exp in natural units, as the merge expects: (m + log2 l) * ln 2
       if (ks == 0 && t == 0) a.part_lse[pidx] = (lt > 0.f) ? (mm + log2f(lt)) * 0.6931471805599453f : -INFINITY;
     } else {
-      __nv_bfloat16* dst = a.out + (size_t)(q0 + tok) * a.out_ld + (size_t)head * RANK + ks * DW;
+      __nv_bfloat16* dst = a.out + (size_t)(q0 + tok) * a.out_ld + (size_t)head * a.rank + ks * DW;
 #pragma unroll
       for (int n = 0; n < NO; ++n)
-        *reinterpret_cast<uint32_t*>(dst + n * 8 + 2 * t) = pack_bf16(o[n][half * 2] * inv, o[n][half * 2 + 1] * inv);
+        if (ks * DW + n * 8 < a.rank) *reinterpret_cast<uint32_t*>(dst + n * 8 + 2 * t) = pack_bf16(o[n][half * 2] * inv, o[n][half * 2 + 1] * inv);
     }
   }
 }
 
 // grid: (n_heads, n_seqs): merge the key ranges of one (sequence, head) by their log-sum-exp weights, in range order.
-template <int RANK>
 __global__ void latent_merge_kernel(Args a) {
   pdl_wait_block();
   pdl_launch_dependents();
   const int b = blockIdx.y, h = blockIdx.x;
   const int tq = a.seq_qstart[b];
-  const int len = a.seq_past[b] + 1;
-  const int per_range = range_keys(a, len);
-  int n_splits = (len + per_range - 1) / per_range;
+  const int len = a.seq_past[b] + 1, k_first = first_visible(a, len - 1) / BN * BN;
+  const int per_range = range_keys(a, len - k_first);
+  int n_splits = (len - k_first + per_range - 1) / per_range;
   if (n_splits > a.max_splits) {
     // only with a fixed split_keys: the sequence is longer than split_keys * max_splits keys, for which the split grid
     // has no blocks and the scratch no room; say so and merge what was computed
@@ -354,21 +368,23 @@ __global__ void latent_merge_kernel(Args a) {
     n_splits = a.max_splits;
   }
   const size_t base = ((size_t)b * a.n_heads + h) * a.max_splits;
-  __nv_bfloat16* o = a.out + (size_t)tq * a.out_ld + (size_t)h * RANK;
-  float mx = -INFINITY;
+  const int rank = a.rank;
+  __nv_bfloat16* o = a.out + (size_t)tq * a.out_ld + (size_t)h * rank;
+  const float sink = a.sinks ? a.sinks[h] : -INFINITY;   // one more range whose log-sum is its score and whose output is 0
+  float mx = sink;
   for (int s = 0; s < n_splits; ++s) mx = fmaxf(mx, a.part_lse[base + s]);
-  float denom = 0.f;
+  float denom = a.sinks ? expf(sink - mx) : 0.f;
   for (int s = 0; s < n_splits; ++s) {
     const float e = a.part_lse[base + s];
     denom += (e == -INFINITY) ? 0.f : expf(e - mx);
   }
   const float inv = 1.f / fmaxf(denom, 1e-20f);
-  for (int c = threadIdx.x; c < RANK; c += blockDim.x) {
+  for (int c = threadIdx.x; c < rank; c += blockDim.x) {
     float v = 0.f;
     for (int s = 0; s < n_splits; ++s) {
       const float e = a.part_lse[base + s];
       const float w = (e == -INFINITY) ? 0.f : expf(e - mx) * inv;
-      v = fmaf(w, a.part_acc[(base + s) * RANK + c], v);
+      v = fmaf(w, a.part_acc[(base + s) * rank + c], v);
     }
     o[c] = __float2bfloat16_rn(v);
   }
@@ -391,7 +407,7 @@ constexpr int kPrefillMB = 4, kPrefillMBSmall = 3, kPrefillKS = 2, kDecodeMB = 1
 template <int RANK, int MB>
 static int launch_prefill(const Args& a, const CUtensorMap& map, int n_seqs, int max_q, cudaStream_t stream) {
   auto k = latent_kernel<RANK, MB, kPrefillKS, false>;
-  const size_t smem = smem_bytes<MB, kPrefillKS>(a.row);
+  const size_t smem = smem_bytes<MB, kPrefillKS>(a.row_pad);
   int e = opt_in(k, smem);
   if (e) return e;
   const long long tiles = ((long long)max_q * a.n_heads + MB * 16 - 1) / (MB * 16);
@@ -407,20 +423,27 @@ static int launch(const Args& a, const void* pages, bool decode, int n_seqs, int
   const int me = tma::make_map_2d_bf16(&map, pages, a.row, (uint64_t)a.num_pages * BN, a.row, 64, BN);
   if (me != 0) return me < 0 ? me : PE_ERR_BAD_ARGUMENT;
   if (!decode) {
-    if (smem_bytes<kPrefillMB, kPrefillKS>(a.row) <= kSmemLimit) return launch_prefill<RANK, kPrefillMB>(a, map, n_seqs, max_q, stream);
+    if (smem_bytes<kPrefillMB, kPrefillKS>(a.row_pad) <= kSmemLimit) return launch_prefill<RANK, kPrefillMB>(a, map, n_seqs, max_q, stream);
     return launch_prefill<RANK, kPrefillMBSmall>(a, map, n_seqs, max_q, stream);
   }
   auto k = latent_kernel<RANK, kDecodeMB, kDecodeKS, true>;
-  const size_t smem = smem_bytes<kDecodeMB, kDecodeKS>(a.row);
+  const size_t smem = smem_bytes<kDecodeMB, kDecodeKS>(a.row_pad);
   int e = opt_in(k, smem);
   if (e) return e;
   const int head_blocks = (a.n_heads + 15) / 16;
   if (head_blocks > 65535 || n_seqs > 65535) return PE_ERR_UNSUPPORTED_SIZE;
   pe::launch(k, dim3(a.max_splits, head_blocks, n_seqs), kDecodeMB * kDecodeKS * 32, smem, stream, a, map);
   PE_LAUNCH_CHECK();
-  pe::launch_after(latent_merge_kernel<RANK>, dim3(a.n_heads, n_seqs), 128, 0, stream, a);
+  pe::launch_after(latent_merge_kernel, dim3(a.n_heads, n_seqs), 128, 0, stream, a);
   PE_LAUNCH_CHECK();
   return PE_OK;
+}
+
+// The padded value size (0: too large) and the padded row of a cached row.
+static int pad_rank(int rank) { return rank <= 64 ? 64 : (rank <= 128 ? 128 : (rank <= 256 ? 256 : (rank <= 512 ? 512 : 0))); }
+static int pad_row(int row, int rank) {
+  const int r = (row + 63) / 64 * 64, v = pad_rank(rank);
+  return r > v ? r : v;
 }
 
 }  // namespace la
@@ -428,18 +451,18 @@ static int launch(const Args& a, const void* pages, bool decode, int n_seqs, int
 
 // Whether these kernels take a cached row of `row` features whose leading `rank` are the values.
 extern "C" int pe_attention_latent_supported(int row, int rank) {
-  if (row <= 0 || row % 64 || rank > row) return 0;
-  if (rank != 128 && rank != 256 && rank != 512) return 0;
-  return pe::la::smem_bytes<pe::la::kPrefillMBSmall, pe::la::kPrefillKS>(row) <= pe::la::kSmemLimit ? 1 : 0;
+  if (row <= 0 || row % 8 || rank <= 0 || rank % 8 || rank > row || pe::la::pad_rank(rank) == 0) return 0;
+  return pe::la::smem_bytes<pe::la::kPrefillMBSmall, pe::la::kPrefillKS>(pe::la::pad_row(row, rank)) <= pe::la::kSmemLimit ? 1 : 0;
 }
 
 // q: [n_tokens, n_heads * row] (row stride q_ld); out: [n_tokens, n_heads * rank] (row stride out_ld); pages:
 // [num_pages, 64, row].  `decode` != 0: every sequence brings one token; scratch holds n_seqs * n_heads * max_splits *
 // (rank + 1) floats; with split_keys 0 a sequence's keys are shared out evenly over max_splits ranges of whole pages,
-// each of at least min_range_keys keys.
+// each of at least min_range_keys keys (with a window: the keys from the first visible page on).  window <= 0: none; sinks
+// [n_heads] float32 or null.
 extern "C" int pe_attention_latent(int decode, const void* q, long long q_ld, void* out, long long out_ld, int n_seqs, int max_q,
-                                   int n_heads, int row, int rank, float scale, const int* seq_qstart, const int* seq_past,
-                                   const int* seq_slot, const int* page_table, int table_stride, int num_pages,
+                                   int n_heads, int row, int rank, float scale, int window, const float* sinks, const int* seq_qstart,
+                                   const int* seq_past, const int* seq_slot, const int* page_table, int table_stride, int num_pages,
                                    const void* pages, float* scratch, int split_keys, int max_splits, int min_range_keys,
                                    int* status, cudaStream_t stream) {
   if (n_seqs <= 0) return PE_OK;
@@ -449,7 +472,8 @@ extern "C" int pe_attention_latent(int decode, const void* q, long long q_ld, vo
     return PE_ERR_BAD_ARGUMENT;
   pe::la::Args a;
   a.q = (const __nv_bfloat16*)q; a.q_ld = q_ld; a.out = (__nv_bfloat16*)out; a.out_ld = out_ld;
-  a.n_heads = n_heads; a.row = row; a.scale_log2 = scale * 1.4426950408889634f;
+  a.n_heads = n_heads; a.row = row; a.rank = rank; a.row_pad = pe::la::pad_row(row, rank); a.window = window; a.sinks = sinks;
+  a.scale_log2 = scale * 1.4426950408889634f;
   a.seq_qstart = seq_qstart; a.seq_past = seq_past; a.seq_slot = seq_slot;
   a.page_table = page_table; a.table_stride = table_stride; a.num_pages = num_pages; a.status = status;
   a.part_acc = nullptr; a.part_lse = nullptr; a.split_keys = 0; a.max_splits = 0; a.min_range_keys = 0;
@@ -460,7 +484,9 @@ extern "C" int pe_attention_latent(int decode, const void* q, long long q_ld, vo
     a.part_acc = scratch;
     a.part_lse = scratch + (size_t)n_seqs * n_heads * max_splits * rank;
   }
-  if (rank == 128) return pe::la::launch<128>(a, pages, decode != 0, n_seqs, max_q, stream);
-  if (rank == 256) return pe::la::launch<256>(a, pages, decode != 0, n_seqs, max_q, stream);
+  const int padded = pe::la::pad_rank(rank);
+  if (padded == 64) return pe::la::launch<64>(a, pages, decode != 0, n_seqs, max_q, stream);
+  if (padded == 128) return pe::la::launch<128>(a, pages, decode != 0, n_seqs, max_q, stream);
+  if (padded == 256) return pe::la::launch<256>(a, pages, decode != 0, n_seqs, max_q, stream);
   return pe::la::launch<512>(a, pages, decode != 0, n_seqs, max_q, stream);
 }

@@ -77,6 +77,15 @@ __global__ void embed_pair_kernel(const T* __restrict__ table, const T* __restri
   for (int c = threadIdx.x; c < hidden; c += blockDim.x) dst[c] = to_f32<T>(src[c]) + to_f32<T>(src2[c]);
 }
 
+// x <- cap * tanh(scale * x / cap), in place.
+__global__ void softcap_kernel(float* __restrict__ x, long long n, float scale, float cap) {
+  pdl_wait_block();
+  pdl_launch_dependents();
+  const float f = scale / cap;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x)
+    x[i] = cap * tanhf(x[i] * f);
+}
+
 }  // namespace pe
 
 extern "C" int pe_embed_gather(int dtype, const void* table, const int* ids, float* out, int n_tokens, int hidden,
@@ -117,6 +126,16 @@ extern "C" int pe_embed_pair_gather(int dtype, const void* table, const void* pa
                buckets, mul_prev, mul_cur, n_slots, status);
   else
     return PE_ERR_UNSUPPORTED_DTYPE;
+  PE_LAUNCH_CHECK();
+  return PE_OK;
+}
+
+extern "C" int pe_softcap(float* x, long long n, float scale, float cap, cudaStream_t stream) {
+  if (n <= 0) return PE_OK;
+  if (!(cap > 0.f)) return PE_ERR_BAD_ARGUMENT;
+  long long blocks = (n + 255) / 256;
+  if (blocks > pe::kSMs * 16) blocks = pe::kSMs * 16;
+  pe::launch(pe::softcap_kernel, (int)blocks, 256, 0, stream, x, n, scale, cap);
   PE_LAUNCH_CHECK();
   return PE_OK;
 }

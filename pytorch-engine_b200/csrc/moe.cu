@@ -10,6 +10,9 @@
 //             choice is an identity expert, which returns its input)
 //   product   out[r] = W[e(r)] x[row_token[r]]  (optionally act(gate rows, up rows) of a [gate | up] matrix)
 //   combine   y[t] = sum_j weight[t, j] * (out[pair_row[t, j]] or x[t]) (+ shared[t])
+//   A weight may stand on an expert's input instead of its output, out = E(weight x): both sums of a row of the [gate | up]
+//   product are multiplied by the row's weight before the activation (the product is linear in x), and the combination adds
+//   with weight one.
 //
 // Which row a pair gets inside its expert's range depends on the order in which blocks arrive; the values do not:
 // every row is computed by itself, and a token's sum runs over its choices in their own order.
@@ -175,7 +178,8 @@ __global__ void moe_route_sigmoid_groups_kernel(const float* logits, int n_token
 
 // One block: counts, offsets, then places.  `offsets` has n_real + 1 entries.
 __global__ void moe_group_kernel(const int* chosen, int n_pairs, int top, int n_real, int* __restrict__ offsets,
-                                 int* __restrict__ row_token, int* __restrict__ pair_row) {
+                                 int* __restrict__ row_token, int* __restrict__ pair_row, const float* weight,
+                                 float* __restrict__ row_weight) {
   extern __shared__ int cnt[];   // n_real counters, then n_real + 1 offsets
   int* off = cnt + n_real;
   pdl_wait_block();
@@ -205,6 +209,7 @@ __global__ void moe_group_kernel(const int* chosen, int n_pairs, int top, int n_
       const int r = off[e] + atomicAdd(&cnt[e], 1);
       row_token[r] = p / top;
       pair_row[p] = r;
+      if (row_weight) row_weight[r] = weight[p];
     } else {
       pair_row[p] = -1;
     }
@@ -243,7 +248,8 @@ template <typename T, typename TOut>
 __global__ void __launch_bounds__(256) moe_rows_gemm_kernel(const T* x, long long x_ld, const int* row_map, const int* offsets,
                                                             int n_groups, const T* __restrict__ w, long long w_group_stride,
                                                             TOut* __restrict__ out, long long out_ld, int n_out, int k_dim,
-                                                            int glu, float limit, float alpha, int vec_ok) {
+                                                            int glu, float limit, float alpha, int vec_ok,
+                                                            const float* row_weight) {
   extern __shared__ float xs[];   // [kMoeRows][k_dim]
   __shared__ int tile_info[3];    // group, first row, rows
   pdl_wait_block();
@@ -322,7 +328,12 @@ __global__ void __launch_bounds__(256) moe_rows_gemm_kernel(const T* x, long lon
         float y = acc[r];
         if (glu) {
           // the two products are rounded as a kernel that writes them would round them
-          const float g = to_f32<T>(from_f32<T>(acc[r])), u = to_f32<T>(from_f32<T>(acc2[r]));
+          float g = to_f32<T>(from_f32<T>(acc[r])), u = to_f32<T>(from_f32<T>(acc2[r]));
+          if (row_weight) {
+            const float f = row_weight[first + r];
+            g *= f;
+            u *= f;
+          }
           y = glu_exact(glu, g, u, limit, alpha);
         }
         out[(size_t)(first + r) * out_ld + n] = from_f32<TOut>(y);
@@ -350,7 +361,7 @@ __global__ void moe_gather_kernel(const T* x, const int* row_token, const int* o
   }
 }
 
-// y[t][c] = sum_j weight[t][j] * (rows[pair_row[t][j]][c] or x[t][c]) (+ shared[t][c])
+// y[t][c] = sum_j weight[t][j] * (rows[pair_row[t][j]][c] or x[t][c]) (+ shared[t][c]); weight null: all of them 1
 template <typename T>
 __global__ void moe_combine_kernel(const T* rows, const T* x, const T* shared, const int* pair_row, const float* weight,
                                    int top, T* __restrict__ out, int n_tokens, int width) {
@@ -363,14 +374,14 @@ __global__ void moe_combine_kernel(const T* rows, const T* x, const T* shared, c
   if (t >= n_tokens) return;
   if (threadIdx.x < top && threadIdx.x < kKeep) {
     s_row[threadIdx.x] = pair_row[(size_t)t * top + threadIdx.x];
-    s_w[threadIdx.x] = weight[(size_t)t * top + threadIdx.x];
+    s_w[threadIdx.x] = weight ? weight[(size_t)t * top + threadIdx.x] : 1.f;
   }
   __syncthreads();
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
     float acc = 0.f;
     for (int j = 0; j < top; ++j) {
       const int r = j < kKeep ? s_row[j] : pair_row[(size_t)t * top + j];
-      const float wj = j < kKeep ? s_w[j] : weight[(size_t)t * top + j];
+      const float wj = j < kKeep ? s_w[j] : (weight ? weight[(size_t)t * top + j] : 1.f);
       const float v = r >= 0 ? to_f32<T>(rows[(size_t)r * width + c]) : to_f32<T>(x[(size_t)t * width + c]);
       acc = fmaf(wj, v, acc);
     }
@@ -405,7 +416,7 @@ __global__ void moe_combine_vec8_kernel(const __nv_bfloat16* rows, const __nv_bf
     };
     for (int j = 0; j < top; ++j) {
       const int r = pair_row[(size_t)t * top + j];
-      add(r >= 0 ? rows + (size_t)r * width + c : x + (size_t)t * width + c, weight[(size_t)t * top + j]);
+      add(r >= 0 ? rows + (size_t)r * width + c : x + (size_t)t * width + c, weight ? weight[(size_t)t * top + j] : 1.f);
     }
     if (shared) add(shared + (size_t)t * width + c, 1.f);
     uint4 o;
@@ -416,10 +427,25 @@ __global__ void moe_combine_vec8_kernel(const __nv_bfloat16* rows, const __nv_bf
   }
 }
 
+// What multiplies both sums of a row before the activation: row_weight[r]; or, where every expert ran on every token (row
+// t * n_real + e), the weight of the token's choice that is e (0: not chosen, nobody reads the row); or nothing.
+struct RowFactor {
+  const float* row_weight;
+  const int* chosen; const float* weight; int top, n_real;
+};
+__device__ __forceinline__ float row_factor(const RowFactor& f, size_t r) {
+  if (f.row_weight) return f.row_weight[r];
+  const size_t t = r / f.n_real;
+  const int e = (int)(r - t * f.n_real);
+  for (int j = 0; j < f.top; ++j)
+    if (f.chosen[t * f.top + j] == e) return f.weight[t * f.top + j];
+  return 0.f;
+}
+
 // act(gate, up) over the two halves of a row of a [gate | up] product (kinds as above); bias: [2 * inter] added first, or null
-template <typename T>
+template <typename T, bool SCALED>
 __global__ void glu_act_kernel(const T* gate_up, T* __restrict__ out, int n_rows, int inter, int kind, float limit, float alpha,
-                               const float* __restrict__ bias) {
+                               const float* __restrict__ bias, RowFactor rf) {
   pdl_wait_block();
   pdl_launch_dependents();
   const size_t total = (size_t)n_rows * inter;
@@ -431,13 +457,19 @@ __global__ void glu_act_kernel(const T* gate_up, T* __restrict__ out, int n_rows
       g += bias[c];
       u += bias[inter + c];
     }
+    if (SCALED) {
+      const float f = row_factor(rf, r);
+      g *= f;
+      u *= f;
+    }
     out[i] = from_f32<T>(glu_exact(kind, g, u, limit, alpha));
   }
 }
 
 // The same for bfloat16 with 16-byte accesses (inter a multiple of 8, everything 16-byte aligned).
+template <bool SCALED>
 __global__ void __launch_bounds__(256) glu_act_vec8_kernel(const __nv_bfloat16* gate_up, __nv_bfloat16* __restrict__ out, int n_rows,
-                                                           int inter, GluEpilogue e) {
+                                                           int inter, GluEpilogue e, RowFactor rf) {
   pdl_wait_block();
   pdl_launch_dependents();
   const int per_row = inter / 8;
@@ -450,6 +482,7 @@ __global__ void __launch_bounds__(256) glu_act_vec8_kernel(const __nv_bfloat16* 
     const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&graw);
     const __nv_bfloat162* u2 = reinterpret_cast<const __nv_bfloat162*>(&uraw);
     uint32_t o[4];
+    const float f = SCALED ? row_factor(rf, r) : 1.f;
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
       float2 g = __bfloat1622float2(g2[k]), u = __bfloat1622float2(u2[k]);
@@ -457,6 +490,7 @@ __global__ void __launch_bounds__(256) glu_act_vec8_kernel(const __nv_bfloat16* 
         const float2 bg = __ldg(reinterpret_cast<const float2*>(e.bias + c) + k), bu = __ldg(reinterpret_cast<const float2*>(e.bias + inter + c) + k);
         g.x += bg.x; g.y += bg.y; u.x += bu.x; u.y += bu.y;
       }
+      if (SCALED) { g.x *= f; g.y *= f; u.x *= f; u.y *= f; }
       o[k] = glu_fast_pair(e, g.x, g.y, u.x, u.y);
     }
     *reinterpret_cast<uint4*>(out + r * inter + c) = make_uint4(o[0], o[1], o[2], o[3]);
@@ -504,22 +538,23 @@ extern "C" int pe_moe_route_sigmoid_groups(const float* logits, int n_tokens, in
 }
 
 extern "C" int pe_moe_group(const int* chosen, int n_tokens, int top, int n_real, int* offsets, int* row_token, int* pair_row,
-                            cudaStream_t stream) {
+                            const float* weight, float* row_weight, cudaStream_t stream) {
   if (n_tokens <= 0) return PE_OK;
-  if (top <= 0 || n_real < 0 || n_real > 4096) return PE_ERR_BAD_ARGUMENT;
+  if (top <= 0 || n_real < 0 || n_real > 4096 || (row_weight && !weight)) return PE_ERR_BAD_ARGUMENT;
   const int n_pairs = n_tokens * top;
   const int threads = n_pairs >= 1024 ? 1024 : (n_pairs + 31) / 32 * 32;
   pe::launch(pe::moe_group_kernel, 1, threads, (size_t)(2 * n_real + 1) * sizeof(int), stream, chosen, n_pairs, top, n_real,
-             offsets, row_token, pair_row);
+             offsets, row_token, pair_row, weight, row_weight);
   PE_LAUNCH_CHECK();
   return PE_OK;
 }
 
 extern "C" int pe_moe_rows_gemm(int dtype, int out_dtype, const void* x, long long x_ld, const int* row_map, const int* offsets,
                                 int n_groups, int max_rows, const void* w, long long w_group_stride, void* out, long long out_ld,
-                                int n_out, int k_dim, int glu, float limit, float alpha, cudaStream_t stream) {
+                                int n_out, int k_dim, int glu, float limit, float alpha, const float* row_weight,
+                                cudaStream_t stream) {
   if (max_rows <= 0 || n_groups <= 0) return PE_OK;
-  if (n_out <= 0 || k_dim <= 0 || glu < 0 || glu > 3) return PE_ERR_BAD_ARGUMENT;
+  if (n_out <= 0 || k_dim <= 0 || glu < 0 || glu > 3 || (row_weight && !glu)) return PE_ERR_BAD_ARGUMENT;
   const size_t smem = (size_t)pe::kMoeRows * k_dim * sizeof(float);
   if (smem > 200 * 1024) return PE_ERR_UNSUPPORTED_SIZE;
   const int elem = dtype == PE_F32 ? 4 : 2;
@@ -536,7 +571,7 @@ extern "C" int pe_moe_rows_gemm(int dtype, int out_dtype, const void* x, long lo
       if (e != cudaSuccess) return (int)e;                                                                              \
     }                                                                                                                   \
     pe::launch(kernel, grid, dim3(256), smem, stream, (const T*)x, x_ld, row_map, offsets, n_groups, (const T*)w,       \
-               w_group_stride, (TOut*)out, out_ld, n_out, k_dim, glu, limit, alpha, vec_ok);                            \
+               w_group_stride, (TOut*)out, out_ld, n_out, k_dim, glu, limit, alpha, vec_ok, row_weight);                \
   } while (0)
   if (dtype == PE_F32 && out_dtype == PE_F32) PE_MOE_LAUNCH(float, float);
   else if (dtype == PE_BF16 && out_dtype == PE_BF16) PE_MOE_LAUNCH(__nv_bfloat16, __nv_bfloat16);
@@ -590,10 +625,17 @@ extern "C" int pe_moe_combine(int dtype, const void* rows, const void* x, const 
   return PE_OK;
 }
 
+// row_weight [n_rows], or chosen / weight [n_rows / n_real, top] (rows token * n_real + expert), or neither: what multiplies
+// both halves of a row before the activation.
 extern "C" int pe_glu_act(int dtype, const void* gate_up, void* out, int n_rows, int inter, int kind, float limit, float alpha,
-                          const float* bias, cudaStream_t stream) {
+                          const float* bias, const float* row_weight, const int* chosen, const float* weight, int top, int n_real,
+                          cudaStream_t stream) {
   if (n_rows <= 0) return PE_OK;
   if (inter <= 0 || kind < 1 || kind > 3) return PE_ERR_BAD_ARGUMENT;
+  if (chosen && (!weight || top <= 0 || n_real <= 0 || n_rows % n_real)) return PE_ERR_BAD_ARGUMENT;
+  if (dtype != PE_F32 && dtype != PE_BF16) return PE_ERR_UNSUPPORTED_DTYPE;
+  const pe::RowFactor rf = {row_weight, chosen, weight, top, n_real};
+  const bool scaled = row_weight || chosen;
   const size_t total = (size_t)n_rows * inter;
   const int threads = 256;
   size_t blocks = (total + threads - 1) / threads;
@@ -602,17 +644,19 @@ extern "C" int pe_glu_act(int dtype, const void* gate_up, void* out, int n_rows,
     pe::GluEpilogue e = {kind, limit, alpha, bias};
     blocks = (total / 8 + threads - 1) / threads;
     if (blocks > pe::kSMs * 16) blocks = pe::kSMs * 16;
-    pe::launch(pe::glu_act_vec8_kernel, (int)blocks, threads, 0, stream, (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, n_rows, inter, e);
+    auto k = scaled ? pe::glu_act_vec8_kernel<true> : pe::glu_act_vec8_kernel<false>;
+    pe::launch(k, (int)blocks, threads, 0, stream, (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, n_rows, inter, e, rf);
     PE_LAUNCH_CHECK();
     return PE_OK;
   }
-  if (dtype == PE_F32)
-    pe::launch(pe::glu_act_kernel<float>, (int)blocks, threads, 0, stream, (const float*)gate_up, (float*)out, n_rows, inter, kind, limit, alpha, bias);
-  else if (dtype == PE_BF16)
-    pe::launch(pe::glu_act_kernel<__nv_bfloat16>, (int)blocks, threads, 0, stream, (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out,
-               n_rows, inter, kind, limit, alpha, bias);
-  else
-    return PE_ERR_UNSUPPORTED_DTYPE;
+  if (dtype == PE_F32) {
+    auto k = scaled ? pe::glu_act_kernel<float, true> : pe::glu_act_kernel<float, false>;
+    pe::launch(k, (int)blocks, threads, 0, stream, (const float*)gate_up, (float*)out, n_rows, inter, kind, limit, alpha, bias, rf);
+  } else {
+    auto k = scaled ? pe::glu_act_kernel<__nv_bfloat16, true> : pe::glu_act_kernel<__nv_bfloat16, false>;
+    pe::launch(k, (int)blocks, threads, 0, stream, (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, n_rows, inter, kind, limit,
+               alpha, bias, rf);
+  }
   PE_LAUNCH_CHECK();
   return PE_OK;
 }

@@ -109,7 +109,7 @@ __global__ void __launch_bounds__(1024) rmsnorm_vec4_kernel(float* __restrict__ 
 // Plain RMSNorm of a tensor in the run dtype (rows of any width), used by parts that normalise
 // something other than the residual stream.
 template <typename T>
-__global__ void rmsnorm_plain_kernel(const T* x, const float* __restrict__ weight, T* __restrict__ out,
+__global__ void rmsnorm_plain_kernel(const T* x, long long x_ld, const float* __restrict__ weight, T* __restrict__ out,
                                      int n_rows, int dim, float eps) {
   extern __shared__ float row_buf[];
   __shared__ float red[32];
@@ -119,13 +119,40 @@ __global__ void rmsnorm_plain_kernel(const T* x, const float* __restrict__ weigh
   if (r >= n_rows) return;
   float ss = 0.f;
   for (int c = threadIdx.x; c < dim; c += blockDim.x) {
-    const float h = to_f32<T>(x[(size_t)r * dim + c]);
+    const float h = to_f32<T>(x[(size_t)r * x_ld + c]);
     row_buf[c] = h;
     ss += h * h;
   }
   const float inv = rsqrtf(block_sum(ss, red) / (float)dim + eps);
   for (int c = threadIdx.x; c < dim; c += blockDim.x)
     out[(size_t)r * dim + c] = from_f32<T>(row_buf[c] * inv * weight[c]);
+}
+
+// The same for rows in 4-element pieces that a block holds in registers (up to VPT pieces a thread).
+template <typename T, int VPT>
+__global__ void __launch_bounds__(1024) rmsnorm_plain_vec4_kernel(const T* x, long long x_ld, const float* __restrict__ weight,
+                                                                   T* __restrict__ out, int dim, float eps) {
+  __shared__ float red[32];
+  pdl_wait_block();
+  pdl_launch_dependents();
+  const T* row = x + (size_t)blockIdx.x * x_ld;
+  float4 h[VPT];
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * 4;
+    h[k] = c < dim ? Vec4<T>::load(row + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) ss += h[k].x * h[k].x + h[k].y * h[k].y + h[k].z * h[k].z + h[k].w * h[k].w;
+  const float inv = rsqrtf(block_sum(ss, red) / (float)dim + eps);
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * 4;
+    if (c >= dim) break;
+    const float4 w = Vec4<float>::load(weight + c);
+    Vec4<T>::store(out + (size_t)blockIdx.x * dim + c, make_float4(h[k].x * inv * w.x, h[k].y * inv * w.y, h[k].z * inv * w.z, h[k].w * inv * w.w));
+  }
 }
 
 // Norm on a sublayer's output, then the residual add (a block that norms what it adds, not what it reads):
@@ -270,6 +297,86 @@ __global__ void __launch_bounds__(1024) rmsnorm_sum_vec4_kernel(float* __restric
   }
 }
 
+// Norm behind the sum (the stream itself is what the norm returns):
+//   h = alpha * stream[row] + scale * delta[row] ;  stream[row] = h * rsqrt(mean(h^2) + eps) * w          float32
+// with one factor `scale` per feature (null: 1), and, when `cast` is given, cast[row] = stream[row] in the run dtype: the
+// next sublayer's input.
+template <typename T>
+__global__ void rmsnorm_of_sum_kernel(float* __restrict__ stream, const T* delta, float alpha, const float* __restrict__ scale,
+                                      const float* __restrict__ weight, T* __restrict__ cast, int n_rows, int dim, float eps) {
+  extern __shared__ float row_buf[];  // dim floats
+  __shared__ float red[32];
+  pdl_wait_block();
+  pdl_launch_dependents();
+  const int r = blockIdx.x;
+  if (r >= n_rows) return;
+  float* s_row = stream + (size_t)r * dim;
+  const T* d_row = delta + (size_t)r * dim;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < dim; c += blockDim.x) {
+    const float y = to_f32<T>(d_row[c]) * (scale ? scale[c] : 1.f);
+    const float h = fmaf(alpha, s_row[c], y);
+    row_buf[c] = h;
+    ss += h * h;
+  }
+  const float inv = rsqrtf(block_sum(ss, red) / (float)dim + eps);
+  for (int c = threadIdx.x; c < dim; c += blockDim.x) {
+    const float h = row_buf[c] * inv * weight[c];
+    s_row[c] = h;
+    if (cast) cast[(size_t)r * dim + c] = from_f32<T>(h);
+  }
+}
+
+// The same with 4-element accesses, for widths that are a multiple of 4 and 16-byte aligned rows; a thread keeps up to VPT
+// pieces of the row in registers.
+template <typename T, int VPT>
+__global__ void __launch_bounds__(1024) rmsnorm_of_sum_vec4_kernel(float* __restrict__ stream, const T* delta, float alpha,
+                                                                    const float* __restrict__ scale,
+                                                                    const float* __restrict__ weight, T* __restrict__ cast,
+                                                                    int n_rows, int dim, float eps) {
+  __shared__ float red[32];
+  const int c0 = threadIdx.x * 4, step = blockDim.x * 4;
+  // neither the weight nor the factors come from the kernel before this one
+  float4 f[VPT];
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    f[k] = make_float4(1.f, 1.f, 1.f, 1.f);
+    if (scale && c0 + k * step < dim) f[k] = Vec4<float>::load(scale + c0 + k * step);
+  }
+  float4 w0 = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (c0 < dim) w0 = Vec4<float>::load(weight + c0);
+  pdl_wait_block();
+  pdl_launch_dependents();
+  const int r = blockIdx.x;
+  if (r >= n_rows) return;
+  float* s_row = stream + (size_t)r * dim;
+  const T* d_row = delta + (size_t)r * dim;
+  float4 h[VPT];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int c = c0 + k * step;
+    h[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < dim) {
+      const float4 x = Vec4<float>::load(s_row + c), y = Vec4<T>::load(d_row + c);
+      h[k] = make_float4(fmaf(alpha, x.x, f[k].x * y.x), fmaf(alpha, x.y, f[k].y * y.y), fmaf(alpha, x.z, f[k].z * y.z),
+                         fmaf(alpha, x.w, f[k].w * y.w));
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) ss += h[k].x * h[k].x + h[k].y * h[k].y + h[k].z * h[k].z + h[k].w * h[k].w;
+  const float inv = rsqrtf(block_sum(ss, red) / (float)dim + eps);
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int c = c0 + k * step;
+    if (c >= dim) break;
+    const float4 w = k == 0 ? w0 : Vec4<float>::load(weight + c);
+    const float4 o = make_float4(h[k].x * inv * w.x, h[k].y * inv * w.y, h[k].z * inv * w.z, h[k].w * inv * w.w);
+    Vec4<float>::store(s_row + c, o);
+    if (cast) Vec4<T>::store(cast + (size_t)r * dim + c, o);
+  }
+}
+
 template <typename K>
 static int set_smem(K kernel, size_t bytes) {
   if (bytes > 48 * 1024) {
@@ -310,27 +417,54 @@ extern "C" int pe_rmsnorm_residual(int dtype, float* residual, const void* delta
   return PE_OK;
 }
 
-extern "C" int pe_rmsnorm(int dtype, const void* x, const float* weight, void* out, int n_rows, int dim, float eps,
-                          cudaStream_t stream) {
+// Rows of x lie x_ld elements apart; rows of out are packed.
+extern "C" int pe_rmsnorm_rows(int dtype, const void* x, long long x_ld, const float* weight, void* out, int n_rows, int dim,
+                               float eps, cudaStream_t stream) {
   if (n_rows <= 0) return PE_OK;
-  if (dim <= 0) return PE_ERR_BAD_ARGUMENT;
+  if (dim <= 0 || x_ld < dim) return PE_ERR_BAD_ARGUMENT;
+  if (dtype != PE_F32 && dtype != PE_BF16) return PE_ERR_UNSUPPORTED_DTYPE;
   const size_t smem = (size_t)dim * sizeof(float);
   if (smem > 200 * 1024) return PE_ERR_UNSUPPORTED_SIZE;
+  const bool vec = dim % 4 == 0 && x_ld % 4 == 0 && dim <= 16384 && ((uintptr_t)x % 16 == 0) && ((uintptr_t)weight % 16 == 0) &&
+                   ((uintptr_t)out % 16 == 0);
+  if (vec) {
+    int threads = (dim / 4 + 31) / 32 * 32;
+    if (n_rows > 2 * pe::kSMs && threads > 256) threads = 256;
+    if (threads > 1024) threads = 1024;
+    while (threads < 1024 && dim > threads * 16) threads *= 2;
+    const int vpt = (dim + threads * 4 - 1) / (threads * 4);
+#define PE_ROWS(T, V) pe::launch(pe::rmsnorm_plain_vec4_kernel<T, V>, n_rows, threads, 0, stream, (const T*)x, x_ld, weight, (T*)out, dim, eps)
+#define PE_ROWS_T(T)               \
+  do {                             \
+    if (vpt <= 1) PE_ROWS(T, 1);   \
+    else if (vpt <= 2) PE_ROWS(T, 2); \
+    else PE_ROWS(T, 4);            \
+  } while (0)
+    if (dtype == PE_F32) PE_ROWS_T(float);
+    else PE_ROWS_T(__nv_bfloat16);
+#undef PE_ROWS_T
+#undef PE_ROWS
+    PE_LAUNCH_CHECK();
+    return PE_OK;
+  }
   const int threads = dim >= 2048 ? 512 : (dim >= 512 ? 256 : 128);
   int e;
   if (dtype == PE_F32) {
     auto k = pe::rmsnorm_plain_kernel<float>;
     if ((e = pe::set_smem(k, smem))) return e;
-    pe::launch(k, n_rows, threads, smem, stream, (const float*)x, weight, (float*)out, n_rows, dim, eps);
-  } else if (dtype == PE_BF16) {
+    pe::launch(k, n_rows, threads, smem, stream, (const float*)x, x_ld, weight, (float*)out, n_rows, dim, eps);
+  } else {
     auto k = pe::rmsnorm_plain_kernel<__nv_bfloat16>;
     if ((e = pe::set_smem(k, smem))) return e;
-    pe::launch(k, n_rows, threads, smem, stream, (const __nv_bfloat16*)x, weight, (__nv_bfloat16*)out, n_rows, dim, eps);
-  } else {
-    return PE_ERR_UNSUPPORTED_DTYPE;
+    pe::launch(k, n_rows, threads, smem, stream, (const __nv_bfloat16*)x, x_ld, weight, (__nv_bfloat16*)out, n_rows, dim, eps);
   }
   PE_LAUNCH_CHECK();
   return PE_OK;
+}
+
+extern "C" int pe_rmsnorm(int dtype, const void* x, const float* weight, void* out, int n_rows, int dim, float eps,
+                          cudaStream_t stream) {
+  return pe_rmsnorm_rows(dtype, x, dim, weight, out, n_rows, dim, eps, stream);
 }
 
 extern "C" int pe_rmsnorm_add(int dtype, float* stream, const void* delta, const float* weight, void* cast, int n_rows,
@@ -387,6 +521,48 @@ extern "C" int pe_rmsnorm_residual_sum(int dtype, float* residual, const void* c
     pe::launch(k, n_rows, threads, smem, stream, residual, list, weight, (__nv_bfloat16*)out, rows, n_rows, dim, eps);
   } else {
     return PE_ERR_UNSUPPORTED_DTYPE;
+  }
+  PE_LAUNCH_CHECK();
+  return PE_OK;
+}
+
+extern "C" int pe_rmsnorm_of_sum(int dtype, float* stream, const void* delta, float alpha, const float* scale, const float* weight,
+                                 void* cast, int n_rows, int dim, float eps, cudaStream_t stream_) {
+  if (n_rows <= 0) return PE_OK;
+  if (dim <= 0 || !stream || !delta || !weight) return PE_ERR_BAD_ARGUMENT;
+  if (dtype != PE_F32 && dtype != PE_BF16) return PE_ERR_UNSUPPORTED_DTYPE;
+  const size_t smem = (size_t)dim * sizeof(float);
+  if (smem > 200 * 1024) return PE_ERR_UNSUPPORTED_SIZE;
+  int threads = dim >= 2048 ? 512 : (dim >= 512 ? 256 : 128);
+  const bool vec = (dim % 4 == 0) && dim <= 16384 && ((uintptr_t)stream % 16 == 0) && ((uintptr_t)weight % 16 == 0) &&
+                   ((uintptr_t)scale % 16 == 0) && ((uintptr_t)cast % 16 == 0) && ((uintptr_t)delta % 16 == 0);
+  if (vec && n_rows <= 64 && dim > 2048) threads = 1024;   // a handful of rows: latency counts (see pe_rmsnorm_residual)
+  if (vec) {
+    while (threads < 1024 && dim > threads * 16) threads *= 2;
+    const int vpt = (dim + threads * 4 - 1) / (threads * 4);
+#define PE_OF_SUM(T, V)                                                                                                        \
+  pe::launch(pe::rmsnorm_of_sum_vec4_kernel<T, V>, n_rows, threads, 0, stream_, stream, (const T*)delta, alpha, scale, weight, \
+             (T*)cast, n_rows, dim, eps)
+#define PE_OF_SUM_T(T)               \
+  do {                               \
+    if (vpt <= 1) PE_OF_SUM(T, 1);   \
+    else if (vpt <= 2) PE_OF_SUM(T, 2); \
+    else PE_OF_SUM(T, 4);            \
+  } while (0)
+    if (dtype == PE_F32) PE_OF_SUM_T(float);
+    else PE_OF_SUM_T(__nv_bfloat16);
+#undef PE_OF_SUM_T
+#undef PE_OF_SUM
+  } else if (dtype == PE_F32) {
+    int e;
+    if ((e = pe::set_smem(pe::rmsnorm_of_sum_kernel<float>, smem))) return e;
+    pe::launch(pe::rmsnorm_of_sum_kernel<float>, n_rows, threads, smem, stream_, stream, (const float*)delta, alpha, scale, weight,
+               (float*)cast, n_rows, dim, eps);
+  } else {
+    int e;
+    if ((e = pe::set_smem(pe::rmsnorm_of_sum_kernel<__nv_bfloat16>, smem))) return e;
+    pe::launch(pe::rmsnorm_of_sum_kernel<__nv_bfloat16>, n_rows, threads, smem, stream_, stream, (const __nv_bfloat16*)delta, alpha,
+               scale, weight, (__nv_bfloat16*)cast, n_rows, dim, eps);
   }
   PE_LAUNCH_CHECK();
   return PE_OK;

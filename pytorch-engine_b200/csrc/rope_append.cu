@@ -825,6 +825,217 @@ __global__ void __launch_bounds__(256, 4) qkv_rotate_append_vec8_kernel(QkvRotat
   }
 }
 
+// ---- one norm over all heads ------------------------------------------------------------------------------------
+// The form in which q and k are each divided by the root mean square of the whole projection (all heads together) and
+// multiplied by a weight of that length; queries may carry a temperature that grows with their position:
+//   q <- unit(q_row) * w_q * (1 + coef * ln(floor((p + 1) / every) + 1)) ;  k <- unit(k_row) * w_k
+// then the rotation (either layout of pairs, or none) and the append as above; values go to the cache as they are.  Without
+// weights nothing is divided.  One block per token; the row's two sums meet in shared memory before anything is written.
+struct QkvRowArgs {
+  QkvRotateArgs r;
+  float temp_coef; int temp_every;   // temp_every <= 0: no temperature
+};
+
+__device__ __forceinline__ float query_temperature(const QkvRowArgs& a, int pos) {
+  if (a.temp_every <= 0) return 1.f;
+  return fmaf(a.temp_coef, logf((float)((pos + 1) / a.temp_every) + 1.f), 1.f);
+}
+
+// The page that holds position `pos` of token t's sequence; -1 (with a report by the first thread) if there is none.
+__device__ __forceinline__ int row_page(const QkvRotateArgs& a, int t, int pos) {
+  if (pos < 0 || pos / kPageTokens >= a.table_stride) {
+    if (threadIdx.x == 0) report(a.status, kStatusPositionOutOfRange, t, pos, a.table_stride * kPageTokens);
+    return -1;
+  }
+  const int page = a.page_table[(size_t)a.seq_slot[a.token_seq[t]] * a.table_stride + pos / kPageTokens];
+  if (page < 0 || page >= a.num_pages) {
+    if (threadIdx.x == 0) report(a.status, kStatusPageOutOfRange, t, page, a.num_pages);
+    return -1;
+  }
+  return page;
+}
+
+// Whether token t clears the rows of its page behind its own (see the first kernel for when and why).
+__device__ __forceinline__ bool clears_page(const QkvRotateArgs& a, int t, int off) {
+  const int b = a.token_seq[t], q_begin = a.seq_qstart[b], q_end = a.seq_qstart[b + 1];
+  return t + 1 == q_end && off + 1 < kPageTokens && (off == 0 || q_end - q_begin > 1);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) qkv_row_norm_append_kernel(QkvRowArgs x) {
+  __shared__ float red[32];
+  const QkvRotateArgs& a = x.r;
+  const int t = blockIdx.x;
+  // the batch description and the page table do not come from the kernel before this one
+  const int pos = a.token_pos[t];
+  const int page = a.write_cache ? row_page(a, t, pos) : -1;
+  const int off = pos % kPageTokens;
+  const bool clears = page >= 0 && clears_page(a, t, off);
+  pdl_wait_block();
+  pdl_launch_dependents();
+  const int d = a.head_dim, dv = a.v_dim, H = a.n_heads, G = a.n_kv_heads;
+  T* row = (T*)a.qkv + (size_t)t * a.ld;
+  const int q_cols = H * d, k_cols = G * d;
+  float inv_q = 1.f, inv_k = 1.f;
+  if (a.q_norm_w) {
+    float sq = 0.f, sk = 0.f;
+    for (int c = threadIdx.x; c < q_cols; c += blockDim.x) {
+      const float v = to_f32<T>(row[c]);
+      sq = fmaf(v, v, sq);
+    }
+    for (int c = threadIdx.x; c < k_cols; c += blockDim.x) {
+      const float v = to_f32<T>(row[q_cols + c]);
+      sk = fmaf(v, v, sk);
+    }
+    inv_q = rsqrtf(block_sum(sq, red) / (float)q_cols + a.eps);
+    inv_k = rsqrtf(block_sum(sk, red) / (float)k_cols + a.eps);
+  }
+  const int rot = a.cos_table ? a.rotary_dim : 0, half = rot / 2;
+  if (rot > 0 && (pos < 0 || pos >= a.table_rows)) {
+    if (threadIdx.x == 0) report(a.status, kStatusPositionOutOfRange, t, pos, a.table_rows);
+    return;
+  }
+  inv_q *= query_temperature(x, pos);
+  auto value = [&](int head, int c) -> float {
+    const bool is_q = head < H;
+    const int col = head * d + c;
+    float v = to_f32<T>(row[col]) * (is_q ? inv_q : inv_k);
+    if (a.q_norm_w) v *= is_q ? a.q_norm_w[col] : a.k_norm_w[col - q_cols];
+    return v;
+  };
+  auto put = [&](int head, int c, float v) {
+    const T o = from_f32<T>(v);
+    if (head < H) row[head * d + c] = o;
+    else if (page >= 0) ((T*)a.k_pages)[(((size_t)page * G + (head - H)) * kPageTokens + off) * d + c] = o;
+  };
+  const int units = half + (d - rot);      // pairs, then single features
+  for (int i = threadIdx.x; i < (H + G) * units; i += blockDim.x) {
+    const int head = i / units, u = i - head * units;
+    if (u < half) {
+      const int i0 = a.interleaved ? 2 * u : u, i1 = a.interleaved ? 2 * u + 1 : u + half;
+      const float x0 = value(head, i0), x1 = value(head, i1);
+      const float c = a.cos_table[(size_t)pos * half + u], s = a.sin_table[(size_t)pos * half + u];
+      put(head, i0, x0 * c - x1 * s);
+      put(head, i1, x1 * c + x0 * s);
+    } else {
+      const int c = rot + (u - half);
+      put(head, c, value(head, c));
+    }
+  }
+  if (page < 0) return;
+  const T* v_row = row + q_cols + k_cols;
+  for (int i = threadIdx.x; i < G * dv; i += blockDim.x) {
+    const int g = i / dv, c = i - g * dv;
+    ((T*)a.v_pages)[(((size_t)page * G + g) * kPageTokens + off) * dv + c] = v_row[i];
+  }
+  if (clears) {
+    const int rest = kPageTokens - 1 - off;
+    for (int g = 0; g < G; ++g) {
+      const size_t first = ((size_t)page * G + g) * kPageTokens + off + 1;
+      for (int i = threadIdx.x; i < rest * d; i += blockDim.x) ((T*)a.k_pages)[first * d + i] = from_f32<T>(0.f);
+      for (int i = threadIdx.x; i < rest * dv; i += blockDim.x) ((T*)a.v_pages)[first * dv + i] = from_f32<T>(0.f);
+    }
+  }
+}
+
+// The same for bfloat16 rows without a rotation, 16 bytes an access (head sizes multiples of 8, everything 16-byte aligned): a
+// thread holds up to VPT pieces of the row in registers, all in flight before the first use.
+template <int VPT>
+__global__ void __launch_bounds__(1024) qkv_row_norm_append_vec8_kernel(QkvRowArgs x) {
+  typedef __nv_bfloat16 T;
+  __shared__ float red_q[32], red_k[32];
+  const QkvRotateArgs& a = x.r;
+  const int t = blockIdx.x;
+  const int pos = a.token_pos[t];
+  const int page = a.write_cache ? row_page(a, t, pos) : -1;
+  const int off = pos % kPageTokens;
+  const bool clears = page >= 0 && clears_page(a, t, off);
+  const int d8 = a.head_dim / 8, dv8 = a.v_dim / 8, G = a.n_kv_heads;
+  const int q8 = a.n_heads * d8, k8 = q8 + G * d8, all8 = k8 + G * dv8;
+  const float temp = query_temperature(x, pos);
+  pdl_wait_block();
+  pdl_launch_dependents();
+  uint4* row = reinterpret_cast<uint4*>((T*)a.qkv + (size_t)t * a.ld);
+  uint4 raw[VPT];
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    raw[k] = i < all8 ? row[i] : make_uint4(0, 0, 0, 0);
+  }
+  float inv_q = 1.f, inv_k = 1.f;
+  if (a.q_norm_w) {
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = threadIdx.x + k * blockDim.x;
+      const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw[k]);
+      float s = 0.f;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 f = __bfloat1622float2(h2[e]);
+        s = fmaf(f.x, f.x, fmaf(f.y, f.y, s));
+      }
+      if (i < q8) sq += s;
+      else if (i < k8) sk += s;
+    }
+    // both sums at one barrier
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = (blockDim.x + 31) >> 5;
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0) { red_q[warp] = sq; red_k[warp] = sk; }
+    __syncthreads();
+    sq = warp_sum(lane < n_warps ? red_q[lane] : 0.f);
+    sk = warp_sum(lane < n_warps ? red_k[lane] : 0.f);
+    inv_q = rsqrtf(sq / (float)(q8 * 8) + a.eps);
+    inv_k = rsqrtf(sk / (float)((k8 - q8) * 8) + a.eps);
+  }
+  inv_q *= temp;
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    if (i >= all8) break;
+    if (i >= k8) {                         // a value: to its page as it is
+      if (page < 0) continue;
+      const int j = i - k8, g = j / dv8, c = j - g * dv8;
+      reinterpret_cast<uint4*>(a.v_pages)[(((size_t)page * G + g) * kPageTokens + off) * dv8 + c] = raw[k];
+      continue;
+    }
+    const bool is_q = i < q8;
+    const float inv = is_q ? inv_q : inv_k;
+    float f[8];
+    const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw[k]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 v = __bfloat1622float2(h2[e]);
+      f[2 * e] = v.x * inv;
+      f[2 * e + 1] = v.y * inv;
+    }
+    if (a.q_norm_w) {
+      const float4* w = reinterpret_cast<const float4*>(is_q ? a.q_norm_w + 8 * i : a.k_norm_w + 8 * (i - q8));
+      const float4 w0 = w[0], w1 = w[1];
+      f[0] *= w0.x; f[1] *= w0.y; f[2] *= w0.z; f[3] *= w0.w; f[4] *= w1.x; f[5] *= w1.y; f[6] *= w1.z; f[7] *= w1.w;
+    }
+    uint4 out;
+    __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&out);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o2[e] = __floats2bfloat162_rn(f[2 * e], f[2 * e + 1]);
+    if (is_q) {
+      row[i] = out;
+    } else if (page >= 0) {
+      const int j = i - q8, g = j / d8, c = j - g * d8;
+      reinterpret_cast<uint4*>(a.k_pages)[(((size_t)page * G + g) * kPageTokens + off) * d8 + c] = out;
+    }
+  }
+  if (clears) {
+    const int rest = kPageTokens - 1 - off;
+    for (int g = 0; g < G; ++g) {
+      const size_t first = ((size_t)page * G + g) * kPageTokens + off + 1;
+      for (int i = threadIdx.x; i < rest * d8; i += blockDim.x) reinterpret_cast<uint4*>(a.k_pages)[first * d8 + i] = make_uint4(0, 0, 0, 0);
+      for (int i = threadIdx.x; i < rest * dv8; i += blockDim.x) reinterpret_cast<uint4*>(a.v_pages)[first * dv8 + i] = make_uint4(0, 0, 0, 0);
+    }
+  }
+}
+
 }  // namespace pe
 
 extern "C" int pe_batch_expand(const int* seq_qstart, const int* seq_past, int n_seqs, int* token_seq, int* token_pos,
@@ -955,6 +1166,52 @@ extern "C" int pe_qkv_rotate_append(int dtype, void* qkv, long long ld, int n_to
   if (dtype == PE_F32) pe::launch(pe::qkv_rotate_append_kernel<float>, grid, warps * 32, 0, stream, a);
   else if (dtype == PE_BF16) pe::launch(pe::qkv_rotate_append_kernel<__nv_bfloat16>, grid, warps * 32, 0, stream, a);
   else return PE_ERR_UNSUPPORTED_DTYPE;
+  PE_LAUNCH_CHECK();
+  return PE_OK;
+}
+
+// q_norm_w [n_heads * head_dim] and k_norm_w [n_kv_heads * head_dim]: both or neither.  temp_every <= 0: no temperature.
+extern "C" int pe_qkv_row_norm_append(int dtype, void* qkv, long long ld, int n_tokens, int n_heads, int n_kv_heads, int head_dim,
+                                      int v_dim, const float* q_norm_w, const float* k_norm_w, float eps, float temp_coef,
+                                      int temp_every, const float* cos_table, const float* sin_table, int rotary_dim,
+                                      int table_rows, int interleaved, const int* token_seq, const int* token_pos,
+                                      const int* seq_slot, const int* seq_qstart, const int* page_table, int table_stride,
+                                      int num_pages, void* k_pages, void* v_pages, int write_cache, int* status,
+                                      cudaStream_t stream) {
+  if (n_tokens <= 0) return PE_OK;
+  if (dtype != PE_F32 && dtype != PE_BF16) return PE_ERR_UNSUPPORTED_DTYPE;
+  if (head_dim <= 0 || v_dim <= 0 || n_heads <= 0 || n_kv_heads <= 0) return PE_ERR_BAD_ARGUMENT;
+  if ((q_norm_w == nullptr) != (k_norm_w == nullptr) || (cos_table == nullptr) != (sin_table == nullptr)) return PE_ERR_BAD_ARGUMENT;
+  if (rotary_dim < 0 || rotary_dim > head_dim || (rotary_dim & 1)) return PE_ERR_UNSUPPORTED_SIZE;
+  if (ld < (long long)(n_heads + n_kv_heads) * head_dim + (long long)n_kv_heads * v_dim) return PE_ERR_BAD_ARGUMENT;
+  pe::QkvRowArgs x = {};
+  pe::QkvRotateArgs& a = x.r;
+  a.qkv = qkv; a.ld = ld; a.n_tokens = n_tokens; a.n_heads = n_heads; a.n_kv_heads = n_kv_heads; a.head_dim = head_dim;
+  a.v_dim = v_dim; a.q_norm_w = q_norm_w; a.k_norm_w = k_norm_w; a.eps = eps;
+  a.cos_table = cos_table; a.sin_table = sin_table; a.rotary_dim = cos_table ? rotary_dim : 0; a.table_rows = table_rows;
+  a.interleaved = interleaved;
+  a.token_seq = token_seq; a.token_pos = token_pos; a.seq_slot = seq_slot; a.seq_qstart = seq_qstart;
+  a.page_table = page_table; a.table_stride = table_stride; a.num_pages = num_pages;
+  a.k_pages = k_pages; a.v_pages = v_pages; a.write_cache = write_cache; a.status = status;
+  x.temp_coef = temp_coef; x.temp_every = temp_every;
+  auto al16 = [](const void* p) { return (uintptr_t)p % 16 == 0; };
+  const long long all8 = ((long long)(n_heads + n_kv_heads) * head_dim + (long long)n_kv_heads * v_dim) / 8;
+  const bool vec8 = dtype == PE_BF16 && a.rotary_dim == 0 && head_dim % 8 == 0 && v_dim % 8 == 0 && ld % 8 == 0 && al16(qkv) &&
+                    al16(k_pages) && al16(v_pages) && al16(q_norm_w) && al16(k_norm_w) && all8 <= 4096;
+  if (vec8) {
+    // a few tokens (decode): one piece a thread, the shortest chain; many: two pieces a thread in flight
+    int threads = (int)((n_tokens < 256 ? all8 : (all8 + 1) / 2) + 31) / 32 * 32;
+    if (threads > 1024) threads = 1024;
+    if (threads < 32) threads = 32;
+    const int vpt = (int)((all8 + threads - 1) / threads);
+    if (vpt <= 1) pe::launch(pe::qkv_row_norm_append_vec8_kernel<1>, n_tokens, threads, 0, stream, x);
+    else if (vpt <= 2) pe::launch(pe::qkv_row_norm_append_vec8_kernel<2>, n_tokens, threads, 0, stream, x);
+    else pe::launch(pe::qkv_row_norm_append_vec8_kernel<4>, n_tokens, threads, 0, stream, x);
+  } else if (dtype == PE_F32) {
+    pe::launch(pe::qkv_row_norm_append_kernel<float>, n_tokens, 256, 0, stream, x);
+  } else {
+    pe::launch(pe::qkv_row_norm_append_kernel<__nv_bfloat16>, n_tokens, 256, 0, stream, x);
+  }
   PE_LAUNCH_CHECK();
   return PE_OK;
 }

@@ -331,15 +331,15 @@ __global__ void rows_to_pages_kernel(const T* src, long long src_ld, int col0, i
   }
 }
 
-// A latent-attention layer's step, per token (grid: tokens).  x row: [.. q: heads x (d + dr) at q_col0 ..
-// low: rank + dr at low_col0 ..].
+// A latent-attention layer's step, per token (grid: tokens).  q row: heads x (d + dr); low row: rank + dr (two column ranges
+// of one product, or rows of two).
 //   cached row  = [ low[:rank] / rms(low[:rank]) * norm_w | turn(low[rank:]) ]        -> pages [num_pages, 1, 64, rank + dr]
 //   qfull[t, h] = [ absorbed[h, t] (a product over heads left it as [heads, n, rank]; null: left as it is) | turn(q[h, d:]) ]
 // turn: adjacent pairs (2i, 2i+1) of the first `rot` features by the angle tables' row of the token's position.
 template <typename T>
-__global__ void __launch_bounds__(256) latent_prepare_kernel(const T* x, long long x_ld, int q_col0, int low_col0, int heads,
-                                                             int d, int dr, int rank, const float* __restrict__ norm_w,
-                                                             float eps, const float* __restrict__ cos_t,
+__global__ void __launch_bounds__(256) latent_prepare_kernel(const T* q_rows, long long q_ld, const T* low_rows,
+                                                             long long low_ld, int heads, int d, int dr, int rank,
+                                                             const float* __restrict__ norm_w, float eps, const float* __restrict__ cos_t,
                                                              const float* __restrict__ sin_t, int rot, int table_rows,
                                                              const int* token_seq, const int* token_pos, const int* seq_slot,
                                                              const int* page_table, int table_stride, int num_pages,
@@ -350,7 +350,7 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const T* x, long lo
   pdl_launch_dependents();
   const int t = blockIdx.x;
   const int pos = token_pos[t];
-  const T* row = x + (size_t)t * x_ld;
+  const T* row = q_rows + (size_t)t * q_ld;
   const int half = rot / 2;
   if (rot > 0 && (pos < 0 || pos >= table_rows)) {
     if (threadIdx.x == 0) report(status, kStatusPositionOutOfRange, t, pos, table_rows);
@@ -362,7 +362,7 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const T* x, long lo
   const int wide = rank + dr;
   for (int i = threadIdx.x; i < heads * dr; i += blockDim.x) {
     const int h = i / dr, c = i - h * dr;
-    const T* q = row + q_col0 + (size_t)h * (d + dr) + d;
+    const T* q = row + (size_t)h * (d + dr) + d;
     float v = to_f32<T>(q[c]);
     if (c < rot) {
       const int m = c >> 1;
@@ -378,7 +378,7 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const T* x, long lo
     }
   }
   if (!write_cache) return;
-  const T* low = row + low_col0;
+  const T* low = low_rows + (size_t)t * low_ld;
   float ss = 0.f;
   for (int c = threadIdx.x; c < rank; c += blockDim.x) {
     const float v = to_f32<T>(low[c]);
@@ -516,15 +516,15 @@ extern "C" int pe_rows_to_pages_pair(int dtype, const void* src, long long src_l
   return PE_OK;
 }
 
-extern "C" int pe_latent_prepare(int dtype, const void* x, long long x_ld, int q_col0, int low_col0, int heads, int d, int dr,
-                                 int rank, const float* norm_w, float eps, const float* cos_t, const float* sin_t, int rot,
+extern "C" int pe_latent_prepare(int dtype, const void* q, long long q_ld, const void* low, long long low_ld, int heads, int d,
+                                 int dr, int rank, const float* norm_w, float eps, const float* cos_t, const float* sin_t, int rot,
                                  int table_rows, int n_tokens, const int* token_seq, const int* token_pos,
                                  const int* seq_slot, const int* page_table, int table_stride, int num_pages, void* pages,
                                  void* qfull, const void* absorbed, int write_cache, int* status, cudaStream_t stream) {
   if (n_tokens <= 0) return PE_OK;
   if (heads <= 0 || d <= 0 || dr < 0 || rank <= 0 || rot < 0 || rot > dr || (rot & 1)) return PE_ERR_BAD_ARGUMENT;
   if (rot > 0 && (!cos_t || !sin_t)) return PE_ERR_BAD_ARGUMENT;
-  PE_BY_DTYPE(dtype, pe::launch(pe::latent_prepare_kernel<T>, n_tokens, 256, 0, stream, (const T*)x, x_ld, q_col0, low_col0,
+  PE_BY_DTYPE(dtype, pe::launch(pe::latent_prepare_kernel<T>, n_tokens, 256, 0, stream, (const T*)q, q_ld, (const T*)low, low_ld,
                                 heads, d, dr, rank, norm_w, eps, cos_t, sin_t, rot, table_rows, token_seq, token_pos, seq_slot,
                                 page_table, table_stride, num_pages, (T*)pages, (T*)qfull, (const T*)absorbed, n_tokens,
                                 write_cache, status));

@@ -77,7 +77,7 @@ _SIGNATURES = {
     "pe_attention_mma_masked": [I, P, L, P, L, I, I, I, I, I, F, I, I, I, I, I, I, I, P, P, I, P, P, P, P, I, I, P, P, P, I, I, I,
                                 P, P],
     "pe_attention_latent_supported": [I, I],
-    "pe_attention_latent": [I, P, L, P, L, I, I, I, I, I, F, P, P, P, P, I, I, P, P, I, I, I, P, P],
+    "pe_attention_latent": [I, P, L, P, L, I, I, I, I, I, F, I, P, P, P, P, P, I, I, P, P, I, I, I, P, P],
     "pe_attention_umma_prefill_ex": [P, L, L, P, L, I, I, I, I, I, F, I, I, P, P, I, P, P, P, P, I, I, P, P, I, P, P, P],
     "pe_attention_decode_noalloc": [I, P, L, P, L, I, I, I, I, F, I, P, P, P, P, I, I, P, P, I, I, P, P],
     "pe_embed_pair_gather": [I, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P, P],
@@ -86,11 +86,11 @@ _SIGNATURES = {
     "pe_short_conv_silu": [I, P, L, I, P, P, I, P, P, P, P, P, I, I, I, I, P, P],
     "pe_delta_rule_recurrence": [I, P, P, P, P, P, P, L, P, F, F, P, P, P, P, I, I, I, I, I, I, I, I, I, P, I, I, L, L, P, P],
     "pe_moe_route": [P, P, I, I, I, P, P, P, I, P],
-    "pe_moe_group": [P, I, I, I, P, P, P, P],
-    "pe_moe_rows_gemm": [I, I, P, L, P, P, I, I, P, L, P, L, I, I, I, F, F, P],
+    "pe_moe_group": [P, I, I, I, P, P, P, P, P, P],
+    "pe_moe_rows_gemm": [I, I, P, L, P, P, I, I, P, L, P, L, I, I, I, F, F, P, P],
     "pe_moe_gather_rows": [I, P, P, P, I, P, I, I, P],
     "pe_moe_combine": [I, P, P, P, P, P, I, P, I, I, P],
-    "pe_glu_act": [I, P, P, I, I, I, F, F, P, P],
+    "pe_glu_act": [I, P, P, I, I, I, F, F, P, P, P, P, I, I, P],
     "pe_gemm_smallm_glu": [P, L, P, P, L, I, I, I, I, I, I, F, F, P, I, P],
     "pe_gemm_umma_glu": [P, L, P, P, L, I, I, I, I, I, I, F, F, P, I, P, P],
     "pe_gemm_umma2_glu": [P, L, P, P, L, I, I, I, I, I, I, F, F, P, I, P, P],
@@ -102,12 +102,17 @@ _SIGNATURES = {
     "pe_attention_umma_dims_supported": [I, I, I, I],
     "pe_attention_umma_prefill_gated": [P, L, L, P, L, I, I, I, I, I, I, F, I, I, P, P, I, P, L, P, P, P, P, I, I, P, P, I, P, P, P],
     "pe_moe_route_logits": [P, P, I, I, I, P, P, P, I, P],
-    "pe_attention_generic_masked": [I, I, P, L, P, L, I, I, I, I, I, I, F, I, I, I, I, I, I, I, P, P, I, I, I, P, P, P, P, I, I,
+    "pe_attention_generic_masked": [I, I, P, L, P, L, I, I, I, I, I, I, F, I, I, I, I, I, I, I, P, P, P, I, I, I, P, P, P, P, I, I,
                                     P, P, P, I, I, P, P],
     "pe_embed_gather_scaled": [I, P, P, P, I, I, I, F, P, P, P],
     "pe_moe_route_sigmoid_groups": [P, I, I, I, I, I, P, P, P, I, P],
     "pe_ssd_recurrence": [I, P, L, P, L, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P, P, P],
-    "pe_gated_part_norm": [I, P, P, L, P, F, P, I, I, I, P],
+    "pe_gated_part_norm": [I, P, P, L, P, F, P, I, I, I, I, P],
+    "pe_lightning_recurrence": [I, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, P, P],
+    "pe_softcap": [P, L, F, F, P],
+    "pe_rmsnorm_rows": [I, P, L, P, P, I, I, F, P],
+    "pe_rmsnorm_of_sum": [I, P, P, F, P, P, P, I, I, F, P],
+    "pe_qkv_row_norm_append": [I, P, L, I, I, I, I, I, P, P, F, F, I, P, P, I, I, I, P, P, P, P, P, I, I, P, P, I, P, P],
     "pe_dyt": [I, I, P, P, P, P, F, P, I, I, P],
     "pe_dyt_add": [I, P, P, P, P, F, P, P, F, P, I, I, P],
     "pe_rmsnorm_pair_mix": [I, P, P, P, P, F, F, F, P, I, I, P],
@@ -120,7 +125,7 @@ _SIGNATURES = {
     "pe_diff_combine": [I, P, P, I, I, I, F, F, F, P],
     "pe_rows_to_pages": [I, P, L, I, I, I, I, P, P, P, P, I, I, P, P, P],
     "pe_rows_to_pages_pair": [I, P, L, I, I, I, I, I, I, I, P, P, P, P, I, I, P, P, P, P],
-    "pe_latent_prepare": [I, P, L, I, I, I, I, I, I, P, F, P, P, I, I, I, P, P, P, P, I, I, P, P, P, I, P, P],
+    "pe_latent_prepare": [I, P, L, P, L, I, I, I, I, P, F, P, P, I, I, I, P, P, P, P, I, I, P, P, P, I, P, P],
 }
 _RESTYPES = {"pe_wait_limit_polls": (L, []),
              "pe_attention_generic_scratch_floats": (L, [I, I, I, I]),

@@ -90,10 +90,34 @@ def rmsnorm_residual(residual: torch.Tensor, delta: Optional[torch.Tensor], weig
 
 
 def rmsnorm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float) -> None:
-    _need(x.is_contiguous() and out.is_contiguous() and weight.dtype == torch.float32, "rmsnorm: contiguous, weight f32")
+    """``out = x / rms(x) * weight`` over the last dimension; ``x`` may be a matrix whose rows lie further apart."""
+    rows = x.dim() == 2 and x.stride(1) == 1
+    _need((x.is_contiguous() or rows) and out.is_contiguous() and out.shape == x.shape and out.dtype == x.dtype
+          and weight.dtype == torch.float32, "rmsnorm: contiguous rows, weight f32")
     dim = x.shape[-1]
-    check(library().pe_rmsnorm(dtype_tag(x.dtype), _ptr(x), _ptr(weight), _ptr(out), x.numel() // dim, dim, float(eps),
-                               _stream()), "rmsnorm")
+    check(library().pe_rmsnorm_rows(dtype_tag(x.dtype), _ptr(x), x.stride(0) if rows and x.shape[0] > 1 else dim, _ptr(weight),
+                                    _ptr(out), x.numel() // dim, dim, float(eps), _stream()), "rmsnorm")
+    _count(1)
+
+
+def rmsnorm_of_sum(stream: torch.Tensor, delta: torch.Tensor, alpha: float, scale: Optional[torch.Tensor], weight: torch.Tensor,
+                   eps: float, cast: Optional[torch.Tensor] = None) -> None:
+    """``h = alpha * stream + scale * delta`` (``scale``: float32, one factor a feature, or None); ``stream = h / rms(h) * weight``
+    (float32, in place); ``cast``, if given, gets the new rows in the run dtype (csrc/rmsnorm.cu)."""
+    n, dim = stream.shape
+    _need(stream.dtype == torch.float32 and weight.dtype == torch.float32 and weight.numel() == dim, "rmsnorm_of_sum: stream and weight float32")
+    _need(scale is None or (scale.dtype == torch.float32 and scale.is_contiguous() and scale.numel() == dim), "rmsnorm_of_sum: scale")
+    _need(stream.is_contiguous() and delta.is_contiguous() and delta.shape == stream.shape, "rmsnorm_of_sum: shapes")
+    _need(cast is None or (cast.dtype == delta.dtype and cast.is_contiguous() and cast.shape == stream.shape), "rmsnorm_of_sum: cast rows")
+    check(library().pe_rmsnorm_of_sum(dtype_tag(delta.dtype), _ptr(stream), _ptr(delta), float(alpha), _ptr(scale), _ptr(weight),
+                                      _ptr(cast), n, dim, float(eps), _stream()), "rmsnorm_of_sum")
+    _count(1)
+
+
+def softcap_(x: torch.Tensor, cap: float, scale: float = 1.0) -> None:
+    """``x <- cap * tanh(scale * x / cap)``, float32, in place."""
+    _need(x.dtype == torch.float32 and x.is_contiguous(), "softcap: contiguous float32")
+    check(library().pe_softcap(_ptr(x), x.numel(), float(scale), float(cap), _stream()), "softcap")
     _count(1)
 
 
@@ -206,6 +230,30 @@ def qkv_rotate_append(qkv: torch.Tensor, n_tokens: int, n_heads: int, n_kv_heads
         0 if page_table is None else page_table.shape[1], num_pages, _ptr(k_pages), _ptr(v_pages),
         1 if write_cache else 0, _ptr(bias), 1 if qk_unit else 0, _ptr(v_mix), float(v_lambda), _ptr(v_keep), _ptr(status),
         _stream()), "qkv_rotate_append")
+    _count(1)
+
+
+def qkv_row_norm_append(qkv: torch.Tensor, n_tokens: int, n_heads: int, n_kv_heads: int, head_dim: int, v_dim: int,
+                        q_norm_w: Optional[torch.Tensor], k_norm_w: Optional[torch.Tensor], eps: float, temperature,
+                        cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rotary_dim: int, interleaved: bool,
+                        token_seq: torch.Tensor, token_pos: torch.Tensor, seq_slot: torch.Tensor, seq_qstart: torch.Tensor,
+                        page_table: Optional[torch.Tensor], num_pages: int, k_pages: Optional[torch.Tensor],
+                        v_pages: Optional[torch.Tensor], write_cache: bool, status: torch.Tensor) -> None:
+    """``qkv_rotate_append`` with q and k each divided by the root mean square of all their heads together, times
+    ``q_norm_w [n_heads * head_dim]`` and ``k_norm_w [n_kv_heads * head_dim]`` (both None: no norm).  ``temperature`` = (coef,
+    every) multiplies q at position p by ``1 + coef * ln(floor((p + 1) / every) + 1)``; None: 1 (csrc/rope_append.cu)."""
+    _need(qkv.stride(-1) == 1, "qkv_row_norm_append: rows of qkv must be contiguous")
+    for t, size in ((q_norm_w, n_heads * head_dim), (k_norm_w, n_kv_heads * head_dim)):
+        _need(t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == size), "qkv_row_norm_append: norm weights")
+    for t in (cos, sin):
+        _need(t is None or (t.dtype == torch.float32 and t.is_contiguous()), "qkv_row_norm_append: float32 tables")
+    coef, every = temperature if temperature is not None else (0.0, 0)
+    check(library().pe_qkv_row_norm_append(
+        dtype_tag(qkv.dtype), _ptr(qkv), qkv.stride(0), n_tokens, n_heads, n_kv_heads, head_dim, v_dim, _ptr(q_norm_w),
+        _ptr(k_norm_w), float(eps), float(coef), int(every), _ptr(cos), _ptr(sin), rotary_dim if cos is not None else 0,
+        0 if cos is None else cos.shape[0], 1 if interleaved else 0, _ptr(token_seq), _ptr(token_pos), _ptr(seq_slot),
+        _ptr(seq_qstart), _ptr(page_table), 0 if page_table is None else page_table.shape[1], num_pages, _ptr(k_pages),
+        _ptr(v_pages), 1 if write_cache else 0, _ptr(status), _stream()), "qkv_row_norm_append")
     _count(1)
 
 
@@ -374,7 +422,7 @@ def attention_mma_masked(decode: bool, q: torch.Tensor, out: torch.Tensor, n_seq
 
 def attention_latent_supported(dtype: torch.dtype, row: int, rank: int) -> bool:
     """Whether the tensor-core kernels of csrc/attention_latent.cu take cached rows of ``row`` features whose leading
-    ``rank`` are the values (bfloat16; rows in steps of 64 up to 576; values of 128, 256 or 512 features)."""
+    ``rank`` are the values (bfloat16; rows up to 576 and values up to 512 features, in steps of 8)."""
     return dtype == torch.bfloat16 and bool(library().pe_attention_latent_supported(int(row), int(rank)))
 
 
@@ -386,17 +434,21 @@ def attention_latent_decode_ranges(device: torch.device, n_seqs: int, n_heads: i
 def attention_latent(decode: bool, q: torch.Tensor, out: torch.Tensor, n_seqs: int, max_q: int, n_heads: int, row: int,
                      rank: int, scale: float, seq_qstart: torch.Tensor, seq_past: torch.Tensor, seq_slot: torch.Tensor,
                      page_table: torch.Tensor, num_pages: int, pages: torch.Tensor, scratch: Optional[torch.Tensor],
-                     split_keys: int, max_splits: int, status: torch.Tensor, min_range_keys: int = 0) -> None:
+                     split_keys: int, max_splits: int, status: torch.Tensor, min_range_keys: int = 0, window: int = 0,
+                     sinks: Optional[torch.Tensor] = None) -> None:
     """Causal attention of ``q [n, n_heads * row]`` over the cached rows ``pages [pages, 1, 64, row]`` taken as one kv head
     whose values are the rows' leading ``rank`` features; ``out [n, n_heads * rank]``.  bfloat16, on the tensor cores.
     Decode: ``scratch`` of ``attention_generic_scratch_floats(n_seqs, n_heads, rank, max_splits)`` floats; with
-    ``split_keys`` 0 a sequence's keys are shared out evenly over ``max_splits`` ranges of at least ``min_range_keys``."""
+    ``split_keys`` 0 a sequence's keys are shared out evenly over ``max_splits`` ranges of at least ``min_range_keys``.
+    ``window`` > 0: a query sees itself and the ``window - 1`` positions before it.  ``sinks [n_heads]`` float32: the
+    denominator of head h also holds ``exp(sinks[h])``."""
+    _need(sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == n_heads), "attention_latent: a float32 sink a head")
     _need(q.stride(-1) == 1 and out.stride(-1) == 1 and pages.is_contiguous(), "attention: rows must be contiguous")
     _need(q.dtype == out.dtype == pages.dtype == torch.bfloat16, "attention_latent: bfloat16 tensors only")
     _need(pages.shape[-1] == row and pages.shape[-2] == 64, "attention_latent: pages of 64 rows of `row` features")
     check(library().pe_attention_latent(
         1 if decode else 0, _ptr(q), q.stride(0), _ptr(out), out.stride(0), n_seqs, max_q, n_heads, row, rank, float(scale),
-        _ptr(seq_qstart), _ptr(seq_past), _ptr(seq_slot), _ptr(page_table), page_table.shape[1], num_pages, _ptr(pages),
+        int(window), _ptr(sinks), _ptr(seq_qstart), _ptr(seq_past), _ptr(seq_slot), _ptr(page_table), page_table.shape[1], num_pages, _ptr(pages),
         _ptr(scratch), split_keys, max_splits, int(min_range_keys), _ptr(status), _stream()), "attention_latent")
     _count(2 if decode else 1)
 
@@ -797,23 +849,26 @@ def moe_route(logits: torch.Tensor, correction: torch.Tensor, top: int, chosen: 
 
 
 def moe_group(chosen: torch.Tensor, n_tokens: int, top: int, n_real: int, offsets: torch.Tensor, row_token: torch.Tensor,
-              pair_row: torch.Tensor) -> None:
+              pair_row: torch.Tensor, weight: Optional[torch.Tensor] = None, row_weight: Optional[torch.Tensor] = None) -> None:
+    """``row_weight`` (float32, as long as ``row_token``), if given, gets every row's ``weight``."""
     _need(offsets.numel() == n_real + 1 and row_token.numel() >= n_tokens * top and pair_row.numel() == n_tokens * top, "moe_group: sizes")
     check(library().pe_moe_group(_ptr(chosen), n_tokens, int(top), int(n_real), _ptr(offsets), _ptr(row_token), _ptr(pair_row),
-                                 _stream()), "moe_group")
+                                 _ptr(weight), _ptr(row_weight), _stream()), "moe_group")
     _count(1)
 
 
 def moe_rows_gemm(x: torch.Tensor, row_map: Optional[torch.Tensor], offsets: torch.Tensor, n_groups: int, max_rows: int,
-                  w: torch.Tensor, out: torch.Tensor, glu: int = 0, limit: float = 0.0, alpha: float = 1.0) -> None:
+                  w: torch.Tensor, out: torch.Tensor, glu: int = 0, limit: float = 0.0, alpha: float = 1.0,
+                  row_weight: Optional[torch.Tensor] = None) -> None:
     """``out[r] = w[group of r] @ x[row_map[r]]`` for the rows ``offsets[g] .. offsets[g + 1]`` of every group; ``w [groups,
-    n_out (twice with glu), k]``; with ``glu`` the output is act(gate rows, up rows) (csrc/moe.cu)."""
+    n_out (twice with glu), k]``; with ``glu`` the output is act(gate rows, up rows), both sums times ``row_weight[r]`` first if
+    that is given (csrc/moe.cu)."""
     _need(w.dim() == 3 and w.is_contiguous() and w.dtype == x.dtype and x.stride(1) == 1 and out.stride(1) == 1, "moe_rows_gemm: layouts")
     n_out = w.shape[1] // 2 if glu else w.shape[1]
     _need(out.shape[1] == n_out and x.shape[1] == w.shape[2], "moe_rows_gemm: shapes")
     check(library().pe_moe_rows_gemm(dtype_tag(x.dtype), dtype_tag(out.dtype), _ptr(x), x.stride(0), _ptr(row_map), _ptr(offsets),
                                      int(n_groups), int(max_rows), _ptr(w), w.stride(0), _ptr(out), out.stride(0), n_out, w.shape[2],
-                                     int(glu), float(limit), float(alpha), _stream()), "moe_rows_gemm")
+                                     int(glu), float(limit), float(alpha), _ptr(row_weight), _stream()), "moe_rows_gemm")
     _count(1)
 
 
@@ -825,8 +880,9 @@ def moe_gather_rows(x: torch.Tensor, row_token: torch.Tensor, offsets: torch.Ten
     _count(1)
 
 
-def moe_combine(rows: torch.Tensor, x: torch.Tensor, shared: Optional[torch.Tensor], pair_row: torch.Tensor, weight: torch.Tensor,
+def moe_combine(rows: torch.Tensor, x: torch.Tensor, shared: Optional[torch.Tensor], pair_row: torch.Tensor, weight: Optional[torch.Tensor],
                 top: int, out: torch.Tensor) -> None:
+    """The chosen rows' sum, weighted with ``weight`` (None: all weights one)."""
     _need(x.is_contiguous() and out.is_contiguous() and rows.is_contiguous() and rows.shape[1] == x.shape[1], "moe_combine: layouts")
     _need(shared is None or (shared.is_contiguous() and shared.shape == x.shape), "moe_combine: shared like x")
     check(library().pe_moe_combine(dtype_tag(x.dtype), _ptr(rows), _ptr(x), _ptr(shared), _ptr(pair_row), _ptr(weight), int(top),
@@ -835,13 +891,23 @@ def moe_combine(rows: torch.Tensor, x: torch.Tensor, shared: Optional[torch.Tens
 
 
 def glu_act(gate_up: torch.Tensor, out: torch.Tensor, kind: str, limit: float = 0.0, alpha: float = 1.0,
-            bias: Optional[torch.Tensor] = None) -> None:
+            bias: Optional[torch.Tensor] = None, row_weight: Optional[torch.Tensor] = None, chosen: Optional[torch.Tensor] = None,
+            weight: Optional[torch.Tensor] = None) -> None:
     """``out = act(gate, up)`` over the halves of ``gate_up [N, 2 * I]``: "silu", "relu", or "clamped_swish"
-    (``g' sigmoid(alpha g') (u' + 1)`` with ``g' = min(g, limit)``, ``u' = clamp(u, -limit, limit)``); ``bias`` (float32 ``[2 * I]``) is added first."""
+    (``g' sigmoid(alpha g') (u' + 1)`` with ``g' = min(g, limit)``, ``u' = clamp(u, -limit, limit)``); ``bias`` (float32 ``[2 * I]``) is added first.
+    Both halves of row r are multiplied before the activation by ``row_weight[r]``; or, with ``chosen`` and ``weight`` ``[tokens,
+    top]``, where row ``t * experts + e`` is expert e's of token t, by the weight of the token's choice e (0: not chosen)."""
+    for t in (row_weight, weight):
+        _need(t is None or (t.dtype == torch.float32 and t.is_contiguous()), "glu_act: float32 weights")
+    _need((chosen is None) == (weight is None) and (chosen is None or (chosen.dtype == torch.int32 and chosen.shape == weight.shape
+          and out.shape[0] % chosen.shape[0] == 0)), "glu_act: chosen and weight [tokens, top]")
+    _need(row_weight is None or row_weight.numel() >= out.shape[0], "glu_act: a weight a row")
     _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == gate_up.shape[1]), "glu_act: bias")
     _need(gate_up.is_contiguous() and out.is_contiguous() and gate_up.shape[1] == 2 * out.shape[1], "glu_act: shapes")
     check(library().pe_glu_act(dtype_tag(gate_up.dtype), _ptr(gate_up), _ptr(out), out.shape[0], out.shape[1], GLU_KINDS[kind],
-                               float(limit), float(alpha), _ptr(bias), _stream()), "glu_act")
+                               float(limit), float(alpha), _ptr(bias), _ptr(row_weight), _ptr(chosen), _ptr(weight),
+                               0 if chosen is None else chosen.shape[1],
+                               0 if chosen is None else out.shape[0] // chosen.shape[0], _stream()), "glu_act")
     _count(1)
 
 
@@ -865,11 +931,14 @@ def attention_generic_masked(decode: bool, q: torch.Tensor, out: torch.Tensor, n
                              seq_past: torch.Tensor, seq_slot: torch.Tensor, page_table: torch.Tensor, num_pages: int,
                              k_pages: torch.Tensor, v_pages: torch.Tensor, scratch: Optional[torch.Tensor], split_keys: int,
                              max_splits: int, status: torch.Tensor, *, window: int = 0, chunk: int = 0,
-                             v_ld: Optional[int] = None, v_heads: Optional[int] = None, keep_first: int = 0) -> None:
+                             v_ld: Optional[int] = None, v_heads: Optional[int] = None, keep_first: int = 0,
+                             sinks: Optional[torch.Tensor] = None) -> None:
     """``attention_generic_ex`` with a chunk mask (``chunk`` > 0: a query sees the keys of its own block of that many
     positions, blocks counted from the sequence's start), kept first keys (``keep_first`` > 0 with a ``window``: positions
     below it stay visible to every later query), value rows ``v_ld`` elements apart (values that are the leading
-    ``v_dim`` features of wider rows) and ``v_heads`` value heads a page (kv head g reads value head ``g % v_heads``)."""
+    ``v_dim`` features of wider rows), ``v_heads`` value heads a page (kv head g reads value head ``g % v_heads``) and ``sinks
+    [n_heads]`` (float32: head h's denominator also holds ``exp(sinks[h])``)."""
+    _need(sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == n_heads), "attention: a float32 sink a head")
     _need(q.stride(-1) == 1 and out.stride(-1) == 1, "attention: rows must be contiguous")
     _need(q.dtype == k_pages.dtype == v_pages.dtype and out.dtype in (q.dtype, torch.float32),
           "attention: q and the cache must share a dtype; out has it too, or is float32")
@@ -878,7 +947,8 @@ def attention_generic_masked(decode: bool, q: torch.Tensor, out: torch.Tensor, n
     check(library().pe_attention_generic_masked(
         dtype_tag(q.dtype), 1 if decode else 0, _ptr(q), q.stride(0), _ptr(out), out.stride(0), n_seqs, max_q, n_heads,
         n_kv_heads, head_dim, v_dim, float(scale), int(window), int(chunk), int(keep_first), v_ld, v_heads,
-        1 if (out.dtype == torch.float32 and q.dtype != torch.float32) else 0, 0, None, None, 0, 0, 0,
+        1 if (out.dtype == torch.float32 and q.dtype != torch.float32) else 0, 0 if sinks is None else 1,
+        _ptr(sinks), None, None, 0, 0, 0,
         _ptr(seq_qstart), _ptr(seq_past), _ptr(seq_slot), _ptr(page_table), page_table.shape[1], num_pages, _ptr(k_pages),
         _ptr(v_pages), _ptr(scratch), split_keys, max_splits, _ptr(status), _stream()), "attention_generic_masked")
     _count(2 if decode else 1)
@@ -976,10 +1046,14 @@ def latent_prepare(x: torch.Tensor, q_col0: int, low_col0: int, heads: int, d: i
                    eps: float, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rot: int, token_seq: torch.Tensor,
                    token_pos: torch.Tensor, seq_slot: torch.Tensor, page_table: torch.Tensor, num_pages: int,
                    pages: torch.Tensor, qfull: torch.Tensor, write_cache: bool, status: torch.Tensor,
-                   absorbed: Optional[torch.Tensor] = None) -> None:
+                   absorbed: Optional[torch.Tensor] = None, q: Optional[torch.Tensor] = None) -> None:
     """A latent-attention layer's cached rows ``[normed low-rank row | turned shared key part]`` into their pages, and the
     turned part of every head's query into ``qfull [n, heads, rank + dr]``; ``absorbed [heads, n, rank]``, if given, fills
-    the leading features of ``qfull``'s rows (csrc/stream_parts.cu)."""
+    the leading features of ``qfull``'s rows.  The queries are columns of ``x`` from ``q_col0`` on, or of ``q`` if that is
+    given; the low-rank row and the key part are columns of ``x`` from ``low_col0`` on (csrc/stream_parts.cu)."""
+    qs = x if q is None else q
+    _need(qs.stride(-1) == 1 and qs.dtype == x.dtype and qs.shape[0] == x.shape[0] and q_col0 + heads * (d + dr) <= qs.shape[1]
+          and low_col0 + rank + dr <= x.shape[1], "latent_prepare: query and low-rank columns")
     _need(absorbed is None or (absorbed.is_contiguous() and absorbed.dtype == x.dtype
                                and tuple(absorbed.shape) == (heads, x.shape[0], rank)), "latent_prepare: absorbed [heads, n, rank]")
     _need(x.stride(-1) == 1 and pages.is_contiguous() and qfull.is_contiguous() and x.dtype == pages.dtype == qfull.dtype
@@ -987,7 +1061,8 @@ def latent_prepare(x: torch.Tensor, q_col0: int, low_col0: int, heads: int, d: i
     if rot:
         _need(cos is not None and cos.dtype == torch.float32 and cos.is_contiguous() and cos.shape == sin.shape
               and cos.shape[1] * 2 == rot, "latent_prepare: angle tables float32 [rows, rot / 2]")
-    check(library().pe_latent_prepare(dtype_tag(x.dtype), _ptr(x), x.stride(0), int(q_col0), int(low_col0), heads, d, dr, rank,
+    check(library().pe_latent_prepare(dtype_tag(x.dtype), _ptr(qs[:, q_col0:]), qs.stride(0), _ptr(x[:, low_col0:]), x.stride(0),
+                                      heads, d, dr, rank,
                                       _ptr(norm_w), float(eps), _ptr(cos) if rot else None, _ptr(sin) if rot else None, int(rot),
                                       cos.shape[0] if rot else 0, x.shape[0], _ptr(token_seq), _ptr(token_pos), _ptr(seq_slot),
                                       _ptr(page_table), page_table.shape[1], num_pages, _ptr(pages), _ptr(qfull), _ptr(absorbed),
@@ -1033,15 +1108,34 @@ def ssd_recurrence(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, A
     _count(3 if chunk > 0 else 1)
 
 
-def gated_part_norm(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor, parts: int) -> None:
+def lightning_recurrence(qkv: torch.Tensor, decay: torch.Tensor, log_decay: torch.Tensor, y: torch.Tensor, S: torch.Tensor,
+                         seq_slot: torch.Tensor, seq_qstart: torch.Tensor, n_seqs: int, max_q: int, heads: int, n: int, dv: int,
+                         status: torch.Tensor, chunk: int = 0, max_chunks: int = 1, scratch: Optional[torch.Tensor] = None) -> None:
+    """``S <- decay S + silu(k) silu(v)^T``, ``y = S^T silu(q)`` with one constant decay per head (csrc/ssd.cu).  ``qkv [N, heads
+    * (2 * n + dv)]`` (q | k | v before their silu, any row stride), ``y [N, heads * dv]`` float32, ``S [slots, heads, n, dv]``
+    float32; ``chunk`` > 0: prompts cut into chunks that run side by side (``scratch``: ``ssd_scratch_floats``)."""
+    _need(qkv.stride(1) == 1 and qkv.shape[1] == heads * (2 * n + dv), "lightning: q|k|v layout")
+    _need(y.dtype == torch.float32 and y.is_contiguous() and S.dtype == torch.float32 and S.is_contiguous()
+          and tuple(S.shape[1:]) == (heads, n, dv), "lightning: y, S f32")
+    for t in (decay, log_decay):
+        _need(t.dtype == torch.float32 and t.numel() == heads, "lightning: float32 decays, one per head")
+    check(library().pe_lightning_recurrence(dtype_tag(qkv.dtype), _ptr(qkv), qkv.stride(0), _ptr(decay), _ptr(log_decay), _ptr(y),
+                                            _ptr(S), _ptr(seq_slot), _ptr(seq_qstart), n_seqs, int(max_q), heads, n, dv, S.shape[0],
+                                            int(chunk), int(max_chunks), _ptr(scratch), _ptr(status), _stream()), "lightning_recurrence")
+    _count(3 if chunk > 0 else 1)
+
+
+def gated_part_norm(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor, parts: int,
+                    gate_first: bool = True) -> None:
     """``v = y * silu(z)``; each of ``parts`` equal parts of a row divided by its root mean square, times ``w`` (csrc/ssd.cu).
+    Without ``gate_first`` the parts of ``y`` itself are normed and weighted and the result is multiplied by ``sigmoid(z)``.
     ``y`` float32, ``z`` and ``out`` in the run dtype (``z`` with any row stride)."""
     n, width = y.shape
     _need(y.dtype == torch.float32 and y.is_contiguous() and out.is_contiguous() and z.stride(1) == 1 and z.dtype == out.dtype
           and tuple(out.shape) == (n, width) and tuple(z.shape) == (n, width), "gated_part_norm: shapes and dtypes")
     _need(w.dtype == torch.float32 and w.numel() == width and width % parts == 0, "gated_part_norm: weight, parts")
     check(library().pe_gated_part_norm(dtype_tag(out.dtype), _ptr(y), _ptr(z), z.stride(0), _ptr(w), float(eps), _ptr(out), n,
-                                       width, int(parts), _stream()), "gated_part_norm")
+                                       width, int(parts), 1 if gate_first else 0, _stream()), "gated_part_norm")
     _count(1)
 
 

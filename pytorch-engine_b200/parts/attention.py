@@ -39,6 +39,9 @@ class GQAttention:
     added in float32 before anything else), ``keep_first`` (with a ``window``: the first that many positions of a sequence stay
     visible to every later query, at their own positions), ``output_gate`` ("sigmoid": the joined heads are multiplied feature
     by feature with ``sigmoid(g_proj x)`` before the output projection; the gate's product rides in the q|k|v product).
+    ``qk_norm`` may also be "row": q and k are each divided by the root mean square of all their heads together, with weights as
+    long as the projections.  ``query_temperature`` ({"coef", "every"}): q at position p is multiplied by ``1 + coef *
+    ln(floor((p + 1) / every) + 1)`` behind its norm (with ``qk_norm`` "row" or none).
     With any of these the mixer runs on the general kernels (``qkv_rotate_append``, ``attention_generic_ex``) unless a
     tensor-core kernel takes the case."""
 
@@ -55,8 +58,9 @@ class GQAttention:
             "o_proj": WeightDecl((h, nh * dv)),
         }
         if params.get("qk_norm", False):
-            decls["q_norm"] = WeightDecl((d,), "norm")
-            decls["k_norm"] = WeightDecl((d,), "norm")
+            row = params["qk_norm"] == "row"
+            decls["q_norm"] = WeightDecl((nh * d if row else d,), "norm")
+            decls["k_norm"] = WeightDecl((nkv * d if row else d,), "norm")
         if params.get("bias", False):
             decls.update({"q_bias": WeightDecl((nh * d,)), "k_bias": WeightDecl((nkv * d,)), "v_bias": WeightDecl((nkv * dv,))})
         if params.get("output_gate"):
@@ -137,6 +141,17 @@ class GQAttention:
             self.fused_position = bool(getattr(self.position, "fusable_rotary", False))
             if not self.fused_position and not hasattr(self.position, "apply"):
                 raise ValueError(f"position encoding {name!r} offers neither tables() nor apply(q, k, positions)")
+        # one norm over all heads, a temperature on the queries: the append is the kernel that takes a token's whole row
+        qk_norm = params.get("qk_norm", False)
+        qt = params.get("query_temperature")
+        self.temperature = None if not qt else (float(qt["coef"]), int(qt["every"]))
+        if self.temperature is not None and self.temperature[1] <= 0:
+            raise ValueError(f"query_temperature: 'every' must be positive, got {self.temperature[1]}")
+        self.row_norm = qk_norm == "row" or self.temperature is not None
+        if self.row_norm and ((qk_norm and qk_norm != "row") or self.bias is not None or self.qk_unit or self.value_mix
+                              or self.v_norm or params.get("value_position") is not None):
+            raise ValueError("a norm over all heads or a query temperature is not built together with a norm per head, biases, unit "
+                             "queries, or normed, mixed or turned values")
         self.value_position = None
         vname = params.get("value_position")
         if vname is not None:
@@ -149,7 +164,7 @@ class GQAttention:
         # what the kernels of the plain softmax attention do not do
         self.general = bool(self.sink or self.v_norm or self.value_position is not None or self.v_dim != self.head_dim
                             or interleaved or self.bias is not None or self.keep_first or self.output_gate or self.qk_unit
-                            or self.value_mix or self.out_bias is not None)
+                            or self.value_mix or self.out_bias is not None or self.row_norm)
         if self.general and self.position is not None and not self.fused_position:
             raise ValueError("the general attention path takes a rotary position encoding with tables(), or none")
         self.qkv_dim = (self.n_heads + self.n_kv_heads) * self.head_dim + self.n_kv_heads * self.v_dim
@@ -241,6 +256,12 @@ class GQAttention:
         if self.value_position is not None:
             vcos, vsin, vrot = self.value_position.tables()
             vinter = bool(getattr(self.value_position, "interleaved", False))
+        if self.row_norm:
+            ops.qkv_row_norm_append(qkv, n, self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim, self.q_norm, self.k_norm,
+                                    self.eps, self.temperature, cos, sin, rot, inter, ctx.token_seq, ctx.token_pos, ctx.seq_slot,
+                                    ctx.seq_qstart, view.page_table, view.num_pages, view.k_pages, view.v_pages, writes_cache,
+                                    self.runtime.status)
+            return
         ops.qkv_rotate_append(qkv, n, self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim, self.q_norm, self.k_norm,
                               self.eps, cos, sin, rot, inter, self.v_norm == "unit", vcos, vsin, vrot, vinter,
                               ctx.token_seq, ctx.token_pos, ctx.seq_slot, ctx.seq_qstart, view.page_table, view.num_pages,
@@ -257,7 +278,7 @@ class GQAttention:
     def fuses_general_into_product(self, x: torch.Tensor, rt) -> bool:
         """``fuses_rope_into_product`` for the general path: values as large as keys, neither normed nor turned; split-half pairs;
         with unit q and k a rotation that leaves lengths as they are, and not a norm with a weight as well."""
-        if self.v_dim != self.head_dim or self.v_norm or self.value_position is not None:
+        if self.v_dim != self.head_dim or self.v_norm or self.value_position is not None or self.row_norm:
             return False
         if self.position is not None and getattr(self.position, "interleaved", False):
             return False

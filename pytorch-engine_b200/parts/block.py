@@ -157,6 +157,50 @@ class PostNormBlock:
         return None
 
 
+@register("arrangement", "norm_of_sum")
+class NormOfSumBlock:
+    """The norm behind the sum: ``x = mixer_norm(alpha x + mixer_scale * mixer(x))``; ``x = ffn_norm(alpha x + ffn_scale *
+    ffn(x))`` if the block has a feed-forward.  Parts by name: ``mixer, mixer_norm`` and optionally ``mixer_scale`` (kind
+    ``feature_scale``), ``ffn, ffn_norm, ffn_scale``.  ``BlockSpec.params``: ``alpha`` (default 1).  The sublayers read the
+    stream itself: in a float32 run directly, otherwise through a copy in the run dtype that every norm leaves behind."""
+
+    graph_safe = True  # launches only; nothing in forward() waits for the device
+
+    def __init__(self, spec, parts, runtime) -> None:
+        self.runtime = runtime
+        self.name = spec.name
+        self.alpha = float(spec.params.get("alpha", 1.0))
+        self.steps = []
+        for name in ("mixer", "ffn"):
+            if name in parts:
+                scale = parts.get(f"{name}_scale")
+                self.steps.append((parts[name], parts[f"{name}_norm"], None if scale is None else scale.weight, name == "mixer"))
+
+    def forward(self, stream: torch.Tensor, pending, ctx, view, writes_cache: bool = True):
+        rt = self.runtime
+        if pending is not None:       # a block before this one left its last delta to be added
+            settle_pending(stream, pending)
+            ctx.stream_copy = None
+        same = rt.dtype == torch.float32
+        x = stream
+        if not same:
+            x = getattr(ctx, "stream_copy", None)
+            if x is None:
+                x = ctx.buffer("block.x", tuple(stream.shape), rt.dtype)
+                x.copy_(stream)
+        cast = None if same else ctx.buffer("block.x", tuple(stream.shape), rt.dtype)
+        for part, norm, scale, is_mixer in self.steps:
+            if is_mixer:
+                mview = view["mixer"] if isinstance(view, dict) else view
+                delta = part.forward(x, ctx, mview) if writes_cache else part.forward(x, ctx, mview, writes_cache=False)
+            else:
+                delta = part.forward(x, ctx)
+            norm.of_sum(stream, delta, self.alpha, scale, cast)
+            x = stream if same else cast
+        ctx.stream_copy = None if same else cast
+        return None
+
+
 @register("arrangement", "parallel")
 class ParallelBlock:
     """One norm feeds every sublayer, and their outputs are added together: ``h = norm(x)``;

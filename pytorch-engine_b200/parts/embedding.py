@@ -75,7 +75,8 @@ class TokenPairEmbedding:
 class LinearHead:
     """params: ``vocab``, ``hidden``.  weights: ``weight [vocab, hidden]``; a tied head names the
     embedding's tensor and shares its storage (pygguf_engine/model.py:1678-1683, 2206-2214).
-    ``scale`` (optional): a factor on the logits.  Output: float32 logits."""
+    ``scale`` (optional): a factor on the logits; ``softcap`` (optional): the logits become ``softcap * tanh(logits / softcap)``
+    behind it.  Output: float32 logits."""
 
     graph_safe = True  # launches only; nothing in forward() waits for the device
 
@@ -88,9 +89,12 @@ class LinearHead:
         self.vocab = int(params["vocab"])
         self.weight = runtime.adopt(weights["weight"])
         self.scale = float(params.get("scale", 1.0) or 1.0)
+        self.softcap = float(params.get("softcap") or 0.0)
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         logits = self.runtime.linear(x, self.weight, out_dtype=torch.float32)
-        if self.scale != 1.0:
+        if self.softcap:
+            ops.softcap_(logits, self.softcap, self.scale)
+        elif self.scale != 1.0:
             logits.mul_(self.scale)
         return logits

@@ -10,7 +10,9 @@ With ``choice = "top_logits"`` the router instead takes the ``top`` largest of `
 over the chosen ones alone (no correction).  With ``choice = "sigmoid_groups"`` the scores are ``s = sigmoid(z)``; the
 experts form ``groups`` equal groups of neighbours, a group scores the sum of its two largest ``s``, and only experts of the
 ``keep_groups`` best groups can be chosen: the ``top`` largest ``s`` among them, weighted with ``s`` itself (no weights beside
-the router's matrix).
+the router's matrix).  With ``weight_on = "input"`` a chosen expert's weight multiplies what the expert reads instead of what
+it returns, ``y = sum_chosen expert_e(s_e h)``; since both products of an expert are linear in what it reads, the weight goes
+onto their sums before the activation.
 
 The (token, choice) pairs are grouped by expert on the device and every expert's rows go through its matrices in one
 launch per product, so nothing is read back to the host and a decode step stays recordable.  A handful of pairs (a
@@ -40,7 +42,8 @@ class RoutedExperts:
     """params: ``hidden``, ``n_experts``, ``n_identity`` (router outputs beyond the real experts), ``top``, ``intermediate``,
     ``activation`` / ``limit`` / ``alpha`` (of every expert), ``shared`` (None, or the params of a ``swiglu`` part).
     ``choice`` ("softmax_all", the default: softmax over every output, the choice moved by ``correction``, weights not
-    renormalised; "top_logits": the largest of ``z + router_bias``, softmax over the chosen).
+    renormalised; "top_logits": the largest of ``z + router_bias``, softmax over the chosen; "sigmoid_groups" with ``groups`` and
+    ``keep_groups``, both 1 by default), ``weight_on`` ("output", the default, or "input"; not with identity experts).
     weights: ``router [n_experts + n_identity, hidden]``, ``correction [n_experts + n_identity]`` (softmax_all) or
     ``router_bias [n_experts + n_identity]`` (top_logits), ``e<i>.gate, e<i>.up
     [I, H]``, ``e<i>.down [H, I]``, and ``shared.gate, shared.up, shared.down`` with a shared expert."""
@@ -80,6 +83,12 @@ class RoutedExperts:
         self.choice = str(params.get("choice") or "softmax_all")
         if self.choice not in ("softmax_all", "top_logits", "sigmoid_groups"):
             raise ValueError(f"router choice {self.choice!r} is not built ('softmax_all', 'top_logits' and 'sigmoid_groups' are)")
+        self.weight_on = str(params.get("weight_on") or "output")
+        if self.weight_on not in ("output", "input"):
+            raise ValueError(f"weight_on {self.weight_on!r} is not built ('output' and 'input' are)")
+        self.on_input = self.weight_on == "input"
+        if self.on_input and self.n_identity:
+            raise ValueError("weight_on 'input' is not built together with identity experts")
         self.correction = self.router_bias = None
         self.groups = int(params.get("groups") or 1)
         self.keep_groups = int(params.get("keep_groups") or self.groups)
@@ -133,12 +142,13 @@ class RoutedExperts:
         gu = ctx.buffer("moe.every_gu", (n, E * 2 * ff), rt.dtype)
         ops.gemm_smallm(x, self.gate_up.view(E * 2 * ff, self.hidden), gu)
         act = ctx.buffer("moe.every_act", (n * E, ff), rt.dtype)
-        ops.glu_act(gu.view(n * E, 2 * ff), act, self.activation, self.limit, self.alpha)
+        ops.glu_act(gu.view(n * E, 2 * ff), act, self.activation, self.limit, self.alpha,
+                    **(dict(chosen=chosen, weight=weight) if self.on_input else {}))
         rows = ctx.buffer("moe.every_rows", (n, E * self.hidden), rt.dtype)
         ops.gemm_smallm_grouped(act.view(n, E, ff).transpose(0, 1), self.down.view(E * self.hidden, ff), rows, self.hidden)
         shared = self.shared.forward(x, ctx) if self.shared is not None else None
         delta = ctx.buffer("moe.delta", (n, self.hidden), rt.dtype)
-        ops.moe_combine(rows.view(n * E, self.hidden), x, shared, pair_row, weight, self.top, delta)
+        ops.moe_combine(rows.view(n * E, self.hidden), x, shared, pair_row, None if self.on_input else weight, self.top, delta)
         return delta
 
     def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
@@ -157,7 +167,8 @@ class RoutedExperts:
         offsets = ctx.buffer("moe.offsets", (self.n_experts + 1,), torch.int32)
         row_token = ctx.buffer("moe.row_token", (n * top,), torch.int32)
         pair_row = ctx.buffer("moe.pair_row", (n, top), torch.int32)
-        ops.moe_group(chosen, n, top, self.n_experts, offsets, row_token, pair_row)
+        row_weight = ctx.buffer("moe.row_weight", (n * top,), torch.float32) if self.on_input else None
+        ops.moe_group(chosen, n, top, self.n_experts, offsets, row_token, pair_row, weight, row_weight)
         rows = ctx.buffer("moe.rows", (n * top, self.hidden), rt.dtype)
         if self.n_experts and self.library_product and n * top > LIBRARY_ROWS and rt.gemm_backend is None:
             # many rows: the rows in expert order, then the library's product over row groups (bfloat16, float32 sums)
@@ -166,13 +177,14 @@ class RoutedExperts:
             ends = offsets[1:]
             gu = torch._grouped_mm(xs, self.gate_up.transpose(1, 2), offs=ends, out_dtype=rt.dtype)
             act = ctx.buffer("moe.act", (n * top, self.intermediate), rt.dtype)
-            ops.glu_act(gu, act, self.activation, self.limit, self.alpha)
+            ops.glu_act(gu, act, self.activation, self.limit, self.alpha, row_weight=row_weight)
             rows = torch._grouped_mm(act, self.down.transpose(1, 2), offs=ends, out_dtype=rt.dtype)
         elif self.n_experts:
             act = ctx.buffer("moe.act", (n * top, self.intermediate), rt.dtype)
-            ops.moe_rows_gemm(x, row_token, offsets, self.n_experts, n * top, self.gate_up, act, self.glu, self.limit, self.alpha)
+            ops.moe_rows_gemm(x, row_token, offsets, self.n_experts, n * top, self.gate_up, act, self.glu, self.limit, self.alpha,
+                              row_weight)
             ops.moe_rows_gemm(act, None, offsets, self.n_experts, n * top, self.down, rows)
         shared = self.shared.forward(x, ctx) if self.shared is not None else None
         delta = ctx.buffer("moe.delta", (n, self.hidden), rt.dtype)
-        ops.moe_combine(rows, x, shared, pair_row, weight, top, delta)
+        ops.moe_combine(rows, x, shared, pair_row, None if self.on_input else weight, top, delta)
         return delta

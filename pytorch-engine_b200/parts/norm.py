@@ -54,6 +54,11 @@ class RMSNorm:
         """The norm on what is added: ``stream += rmsnorm(delta) * w``; ``cast`` gets the new rows in the run dtype."""
         ops.rmsnorm_add(stream, delta, self.weight, self.eps, cast)
 
+    def of_sum(self, stream: torch.Tensor, delta: torch.Tensor, alpha: float, scale: Optional[torch.Tensor],
+               cast: Optional[torch.Tensor] = None) -> None:
+        """The norm behind the sum: ``stream = rmsnorm(alpha * stream + scale * delta) * w``; ``cast`` as above."""
+        ops.rmsnorm_of_sum(stream, delta, alpha, scale, self.weight, self.eps, cast)
+
 
 @register("norm", "layer_norm")
 class LayerNorm:

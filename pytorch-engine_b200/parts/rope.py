@@ -13,7 +13,7 @@ YaRN (``scaling`` = factor, original, fast, slow): with ``turn(t) = rotary_dim *
 the pair index at which a pair makes ``t`` turns over ``original`` positions, ``lo = max(floor(turn(fast)), 0)``,
 ``hi = min(ceil(turn(slow)), rotary_dim - 1)`` and ``ramp_j = clamp((j - lo) / max(hi - lo, 0.001), 0, 1)``, pair j
 turns with ``f_j / factor * ramp_j + f_j * (1 - ramp_j)``, and cos and sin carry the factor ``0.1 ln(factor) + 1``.
-The scaled frequencies are computed in float64 on the host and rounded once to float32.
+The scaled frequencies are computed in float64 on the host (and rounded once to float32 unless the tables are ``exact``).
 """
 from __future__ import annotations
 
@@ -61,12 +61,15 @@ class RotaryPosition:
         linear = 1.0
         if scaling and "original" not in scaling:
             linear, scaling = float(scaling["factor"]), None
-        if params.get("exact") and not scaling:
+        if params.get("exact"):
             # frequencies, angles, cos and sin in float64 on the host, each table entry rounded once to float32
-            idx = torch.arange(0, self.rotary_dim, 2, dtype=torch.float64)
-            ang = torch.outer(torch.arange(0, self.max_positions, dtype=torch.float64), self.theta ** (-idx / self.rotary_dim) / linear)
-            self.cos = torch.cos(ang).to(torch.float32).to(runtime.device).contiguous()
-            self.sin = torch.sin(ang).to(torch.float32).to(runtime.device).contiguous()
+            if scaling:
+                freq, mult = yarn_frequencies(self.rotary_dim, self.theta, scaling, torch.float64)
+            else:
+                freq = self.theta ** (-torch.arange(0, self.rotary_dim, 2, dtype=torch.float64) / self.rotary_dim) / linear
+            ang = torch.outer(torch.arange(0, self.max_positions, dtype=torch.float64), freq)
+            self.cos = (torch.cos(ang) * mult).to(torch.float32).to(runtime.device).contiguous()
+            self.sin = (torch.sin(ang) * mult).to(torch.float32).to(runtime.device).contiguous()
             return
         if not scaling:
             idx = torch.arange(0, self.rotary_dim, 2, dtype=torch.float32)
@@ -88,8 +91,8 @@ class RotaryPosition:
         return self.cos, self.sin, self.rotary_dim
 
 
-def yarn_frequencies(rotary_dim: int, theta: float, scaling):
-    """(float32 frequencies ``[rotary_dim / 2]``, factor on cos and sin) of a YaRN-scaled encoding."""
+def yarn_frequencies(rotary_dim: int, theta: float, scaling, dtype: torch.dtype = torch.float32):
+    """(frequencies ``[rotary_dim / 2]``, factor on cos and sin) of a YaRN-scaled encoding."""
     factor, original = float(scaling["factor"]), float(scaling["original"])
     j = torch.arange(rotary_dim // 2, dtype=torch.float64)
     f = float(theta) ** (-2.0 * j / rotary_dim)
@@ -101,4 +104,4 @@ def yarn_frequencies(rotary_dim: int, theta: float, scaling):
     hi = min(math.ceil(turn(float(scaling["slow"]))), rotary_dim - 1)
     ramp = ((j - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
     f = f / factor * ramp + f * (1.0 - ramp)
-    return f.to(torch.float32), 0.1 * math.log(factor) + 1.0
+    return f.to(dtype), 0.1 * math.log(factor) + 1.0

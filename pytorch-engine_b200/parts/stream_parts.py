@@ -20,6 +20,9 @@ runs several times over takes the model's input in again in front of every pass)
 ``stream_bundle``: how a sublayer reads several residual streams and writes its output back into them (learned numbers per
 stream and per pair of streams; the ``streams`` arrangement of ``parts/block.py`` runs it fused with the norms).
 
+``feature_scale``: one learned factor per feature on a sublayer's output before it is added (a layer scale; the arrangement runs
+it fused with the add and the norm).
+
 ``normed_mean``: two sublayer outputs side by side become one, ``(unit(a) * w_a + unit(b) * w_b) / 2``, each divided by its own
 root mean square over the row first.
 """
@@ -174,3 +177,17 @@ class StreamBundle:
         self.read = runtime.adopt(weights["read"], torch.float32)
         self.mix = runtime.adopt(weights["mix"], torch.float32)
         self.write = runtime.adopt(weights["write"], torch.float32)
+
+
+@register("stream", "feature_scale")
+class FeatureScale:
+    """params: ``dim``.  weights: ``weight [dim]`` (kept in float32)."""
+
+    graph_safe = True  # nothing runs here: the arrangement reads the factors
+
+    @classmethod
+    def weight_decls(cls, params) -> Dict[str, WeightDecl]:
+        return {"weight": WeightDecl((int(params["dim"]),), "norm")}
+
+    def __init__(self, params, weights, runtime) -> None:
+        self.weight = runtime.adopt(weights["weight"], torch.float32)
