@@ -140,3 +140,28 @@ def test_cli_greedy_zonevik(pe, tmp_path, capsys):
         for j, tok in enumerate(r["token_ids"]):
             row = ref[len(p) - 1 + j]
             assert float(row.max() - row[tok]) <= 1e-4 * float(ref.abs().max())
+
+
+def test_cli_greedy_burinex(pe, tmp_path, capsys):
+    """The seventh architecture through the same command line: a folder written from the preset (lightning, latent attention under
+    a window, attention with one norm over all heads, experts weighted on their input), greedy tokens in float32 against the plain
+    implementation's best token at every step."""
+    import plain_burinex
+    from safetensors.torch import load_file
+
+    folder = str(tmp_path / "x")
+    pe.write_random_model(folder, pe.preset("burinex_tiny"), 7)
+    with open(folder + "/config.json") as fh:
+        cfg = json.load(fh)
+    w = {k: v.float() for k, v in load_file(folder + "/model.safetensors").items()}
+    prompts = _prompts(cfg["vocab"], (3, 11, 150), 3)
+    argv = ["--model", folder, "--dtype", "fp32", "--ctx", "256", "--max-tokens", "6", "--temperature", "0", "--json"]
+    for p in prompts:
+        argv += ["--prompt-ids", ",".join(map(str, p))]
+    out = _run_cli(capsys, argv)
+    for r, p in zip(out, prompts):
+        assert r["completion_tokens"] == 6
+        ref = plain_burinex.forward(cfg, w, p + r["token_ids"])
+        for j, tok in enumerate(r["token_ids"]):
+            row = ref[len(p) - 1 + j]
+            assert float(row.max() - row[tok]) <= 1e-4 * float(ref.abs().max())
