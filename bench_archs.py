@@ -1,6 +1,7 @@
-"""``python bench.py --archs``: the Vabelorn, Lunadra, Vemepel, Zonevik and Bobasun architectures beside the Qwen3 dense decoder
+"""``python bench.py --archs``: the Vabelorn, Lunadra, Vemepel, Zonevik, Bobasun and Burinex architectures beside the Qwen3 dense decoder
 at equal layer sizes (``--arch-names`` picks among them; Lunadra's own kernels stand beside the like kernels of the Vabelorn
-path, Zonevik's beside those of the Lunadra path, Vemepel's and Bobasun's beside those of the Qwen3 path).
+path, Zonevik's beside those of the Lunadra path, Vemepel's and Bobasun's beside those of the Qwen3 path, Burinex's beside
+those of Vemepel, Zonevik and Bobasun).
 
 Random weights, bfloat16, one B200.  For each size: tokens/s of a 2,048-token prompt and of decode steps at batch 8
 (context 2,048) through ``ModelRunner.step``, for both architectures; then the kernels that only the new
@@ -880,6 +881,178 @@ def bobasun_kernel_pairs(pe, torch, s, peaks, prompt, batch, context):
     return out
 
 
+def burinex_config(pe, s):
+    """Burinex at the same width, attention heads and vocabulary: latent attention (rows of 512 + 64 features, a window of 1,024
+    positions), attention with one norm over all heads, lightning attention with heads of 128 x 128; routed experts (8, two chosen)
+    whose chosen experts and shared expert together are as wide as the dense feed-forward."""
+    d, H = s["dim"], s["heads"]
+    moe = {"kind": "moe", "router": {"experts": 8, "top": 2}, "expert": {"ff": s["ff"] // 4}, "shared": {"ff": s["ff"] // 2}}
+    lat = {"type": "latent_attention", "mlp": moe,
+           "mixer": {"heads": H, "dim": d, "rot_dim": d // 2, "vdim": d, "kv_rank": 4 * d, "q_rank": 3 * s["width"] // 8, "scale": (1.5 * d) ** -0.5,
+                     "mask": {"size": 1024}, "rot": {"base": 1e6, "dims": d // 2, "scaling": YARN}}}
+    att = {"type": "attention", "mlp": moe,
+           "mixer": {"heads": H, "kv_heads": s["kv_heads"], "dim": d, "vdim": d, "scale": d ** -0.5, "q_temp": {"coef": 0.1, "every": 1024}}}
+    lig = {"type": "lightning", "mlp": moe,
+           "mixer": {"heads": H, "dim": d, "vdim": d, "decay": [1.0 - 2.0 ** -(1.0 + 9.0 * i / H) for i in range(H)]}}
+    pattern = [lat, att, lig, att]
+    return pe.BurinexConfig.from_dict({"architecture": "Burinex", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
+                                       "postln_alpha": 2.0, "logit_softcap": 30.0, "layers": [pattern[i % 4] for i in range(s["layers"])]})
+
+
+def burinex_kernel_pairs(pe, torch, s, peaks, prompt, batch, context):
+    """The kernels that only Burinex has, each beside the like kernel of the closest model that has one: Vemepel's latent attention,
+    Bobasun's attention and append, Zonevik's state-space recurrence and gated norm, the experts' activation and sum of all of
+    them, the usual add and norm.  Rooflines as in ``zonevik_kernel_pairs`` (recurrences: float32 operations over the CUDA cores'
+    rate) and ``vemepel_kernel_pairs`` (attention: tensor operations over the products' rate)."""
+    ops = pe.kernels.ops
+    dev = torch.device("cuda:0")
+    bf = torch.bfloat16
+    H, G, d, width, ff = s["heads"], s["kv_heads"], s["dim"], s["width"], s["ff"]
+    hbm_gbs, tflops = peaks["hbm_gbs"], peaks.get("bf16_tflops") or 1590.0
+    flush = torch.zeros(96 * 2 ** 20, device=dev)
+    status = torch.zeros(4, dtype=torch.int32, device=dev)
+    out, held = {}, {}
+
+    def buffer(name, shape, dtype):
+        key = (name, tuple(shape), dtype)
+        if key not in held:
+            held[key] = torch.empty(shape, dtype=dtype, device=dev)
+        return held[key]
+
+    def us_of(fn):
+        return 1e3 * timed(torch, fn, 20, 5, flush, graph=True)
+
+    def roof_us(nbytes, flops=0.0, rate=tflops):
+        return max(nbytes / (hbm_gbs * 1e9), flops / (rate * 1e12)) * 1e6
+
+    def entry(name, us_new, roof_new, like, us_like, roof_like):
+        out[name] = {"us": round(us_new, 2), "roofline_us": round(roof_new, 2), "of_roofline": round(roof_new / us_new, 3),
+                     "like_kernel": like, "like_us": round(us_like, 2), "like_of_roofline": round(roof_like / us_like, 3),
+                     "times_as_far_from_roofline": round((us_new / roof_new) / (us_like / roof_like), 2)}
+
+    rn = lambda *shape: torch.randn(*shape, device=dev)
+    for what, n_seqs, q_len, past in (("prompt", 1, prompt, 0), ("decode", batch, 1, context - 1)):
+        n, decode, length = n_seqs * q_len, q_len == 1, past + q_len
+        pages_per = -(-length // 64)
+        n_pages = n_seqs * pages_per
+        table = torch.arange(n_pages, dtype=torch.int32, device=dev).view(n_seqs, pages_per).contiguous()
+        qstart = torch.arange(0, n + 1, q_len, dtype=torch.int32, device=dev)
+        pasts = torch.full((n_seqs,), past, dtype=torch.int32, device=dev)
+        slots = torch.arange(n_seqs, dtype=torch.int32, device=dev)
+        token_seq = slots.repeat_interleave(q_len).contiguous()
+        token_pos = (torch.arange(q_len, dtype=torch.int32, device=dev)[None] + past).repeat(n_seqs, 1).view(-1).contiguous()
+        where = (qstart, pasts, slots, table, n_pages)
+        # ---- the norm behind the sum
+        stream, delta = rn(n, width), rn(n, width).to(bf)
+        w, normed = torch.ones(width, device=dev), torch.empty(n, width, dtype=bf, device=dev)
+        us_add = us_of(lambda: ops.rmsnorm_residual(stream, delta, w, normed, 1e-6))
+        us = us_of(lambda: ops.rmsnorm_of_sum(stream, delta, 2.0, w, w, 1e-6, normed))
+        entry(f"{what}: layer scale, weighted add, norm of the sum", us, roof_us(n * width * 12), "rmsnorm_residual", us_add, roof_us(n * width * 12))
+        # ---- latent attention under a window with sinks
+        rank, dr, window = 4 * d, d // 2, 1024
+        row = rank + dr
+        lp = rn(n_pages, 1, 64, row).to(bf)
+        qf, mixed = (0.3 * rn(n, H * row)).to(bf), torch.empty(n, H * rank, dtype=bf, device=dev)
+        lat = pe.parts.latent_attention.attend_rows
+        run = lambda **kw: lat(ops, decode, qf, mixed, n_seqs, q_len, H, row, rank, 0.07, *where, lp, status, context + 64, buffer, **kw)
+        sinks = torch.zeros(H, device=dev)
+
+        def latent_roof(seen):
+            pairs = n_seqs * sum(min(past + i + 1, seen) for i in range(q_len))
+            return roof_us(n * H * (row + rank) * 2 + n_seqs * (min(length, seen) if decode else length) * row * 2, pairs * H * (row + rank) * 2.0)
+        us_lat = us_of(run)
+        us = us_of(lambda: run(sinks=sinks))
+        entry(f"{what}: latent attention ({rank} + {dr} features), sinks", us, latent_roof(length), "the same without sinks", us_lat, latent_roof(length))
+        us = us_of(lambda: run(window=window, sinks=sinks))
+        entry(f"{what}: latent attention ({rank} + {dr} features), a window of {window}, sinks", us, latent_roof(window),
+              "latent attention over all keys", us_lat, latent_roof(length))
+        # ---- the latent rows: the query latent's norm; the cached row and the turned queries
+        q_rank = 3 * width // 8
+        low = rn(n, q_rank + row).to(bf)
+        qn, cq = torch.ones(q_rank, device=dev), torch.empty(n, q_rank, dtype=bf, device=dev)
+        us = us_of(lambda: ops.rmsnorm(low[:, :q_rank], qn, cq, 1e-6))
+        entry(f"{what}: norm of the query latent", us, roof_us(n * q_rank * 4), "rmsnorm_residual", us_add, roof_us(n * width * 12))
+        rt = pe.parts.Runtime(dev, bf)
+        ci, si, ri = pe.parts.lookup("position", "rope")({"rotary_dim": dr, "theta": 1e6, "max_positions": context + 64, "style": "interleaved",
+                                                          "scaling": YARN, "exact": True}, {}, rt).tables()
+        qh, qfull, nw = rn(n, H * (d + dr)).to(bf), torch.empty(n, H, row, dtype=bf, device=dev), torch.ones(rank, device=dev)
+        absorbed = rn(H, n, rank).to(bf)
+        prep = lambda **kw: ops.latent_prepare(low, 0, q_rank, H, d, dr, rank, nw, 1e-6, ci, si, ri, token_seq, token_pos, slots, table,
+                                               n_pages, lp, qfull, True, status, q=qh, **kw)
+        base = n * (H * dr + row) * 4
+        us_like = us_of(lambda: prep(absorbed=absorbed))
+        entry(f"{what}: latent row's norm, rotation, append, turned queries", us_of(prep), roof_us(base),
+              "latent_prepare that also copies the folded queries", us_like, roof_us(base + n * H * rank * 4))
+        # ---- q|k|v rows: one norm over all heads, temperature, append
+        kp, vp = rn(n_pages, G, 64, d).to(bf), rn(n_pages, G, 64, d).to(bf)
+        rows = rn(n, (H + 2 * G) * d + 8).to(bf)
+        qw, kw = torch.ones(H * d, device=dev), torch.ones(G * d, device=dev)
+        at = (token_seq, token_pos, slots, qstart, table, n_pages, kp, vp, True, status)
+        nbytes = n * (H + 2 * G) * d * 2 + n * (H + G) * d * 2 + n * G * d * 2
+        us_like = us_of(lambda: ops.qkv_rotate_append(rows, n, H, G, d, d, None, None, 1e-6, None, None, 0, False, False, None, None, 0, False,
+                                                      *at, qk_unit=True))
+        us = us_of(lambda: ops.qkv_row_norm_append(rows, n, H, G, d, d, qw, kw, 1e-6, (0.1, 1024), None, None, 0, False, *at))
+        entry(f"{what}: one norm over all heads, query temperature, append", us, roof_us(nbytes), "qkv_rotate_append (unit norm a head)", us_like,
+              roof_us(nbytes))
+
+        # ---- attention with a sink and a gate per head
+        def attention(hd, vd, gated):
+            q = (0.5 * rn(n, H * hd + H)).to(bf)
+            k, v = (0.5 * rn(n_pages, G, 64, hd)).to(bf), (0.5 * rn(n_pages, G, 64, vd)).to(bf)
+            o = torch.empty(n, H * vd, dtype=bf, device=dev)
+            kw = dict(sink=gated, gate=q[:, H * hd:] if gated else None)
+            if not decode and ops.attention_umma_dims_supported(bf, hd, vd, H, G):
+                us = us_of(lambda: ops.attention_umma_prefill(q, o, n_seqs, q_len, H, G, hd, hd ** -0.5, 0, *where, k, v, status, v_dim=vd, **kw))
+            else:
+                sk, ms, fl = ops.attention_mma_decode_ranges(dev, hd, n_seqs, G, context + 64, 512, v_dim=vd) if decode else (512, 0, 0)
+                scr = torch.empty(ops.attention_generic_scratch_floats(n_seqs, H, vd, max(ms, 1)), device=dev)
+                us = us_of(lambda: ops.attention_mma_gated(decode, q, o, n_seqs, q_len, H, G, hd, vd, hd ** -0.5, 0, *where, k, v, scr, sk, ms, status,
+                                                           min_range_keys=fl, **kw))
+            flops = 2.0 * n * H * (hd + vd) * (length if decode else length / 2)
+            return us, roof_us(n * H * (hd + vd) * 2 + n_seqs * length * G * (hd + vd) * 2, flops)
+
+        for hd, vd in ((d, d), (d // 2, 5 * d // 8)):
+            us_like, roof_like = attention(hd, hd, False)
+            us, roof = attention(hd, vd, True)
+            entry(f"{what}: attention with sink and gates, keys of {hd}, values of {vd}", us, roof, f"attention, {hd} and {hd}", us_like, roof_like)
+        # ---- the recurrence with constant decays beside the state-space recurrence of the same state and row sizes
+        chunked = q_len > 128
+        qkv, dec = rn(n, 3 * H * d).to(bf), torch.full((H,), 0.99, device=dev)
+        y, S = torch.empty(n, H * d, device=dev), torch.zeros(n_seqs, H, d, d, device=dev)
+        smax = -(-q_len // 64) if chunked else 1
+        scratch = torch.empty(ops.ssd_scratch_floats(n_seqs, H, d, d, smax), device=dev) if chunked else None
+        ck = (64 if chunked else 0, smax, scratch)
+        zero, one = torch.zeros(H, device=dev), torch.ones(H, device=dev)
+        dt = rn(n, H).to(bf)
+        us_like = us_of(lambda: ops.ssd_recurrence(qkv, dt, zero, zero, one, y, S, slots, qstart, n_seqs, q_len, H, H, d, d, status, *ck))
+        roof = roof_us(n * H * d * (6 + 4) + n_seqs * H * d * d * 8, n * H * d * d * 4.0, FP32_TFLOPS)
+        us = us_of(lambda: ops.lightning_recurrence(qkv, dec, torch.log(dec), y, S, slots, qstart, n_seqs, q_len, H, d, d, status, *ck))
+        entry(f"{what}: lightning recurrence", us, roof, "ssd_recurrence", us_like, roof)
+        z, nw2, yo = rn(n, H * d).to(bf), torch.ones(H * d, device=dev), torch.empty(n, H * d, dtype=bf, device=dev)
+        us_like = us_of(lambda: ops.gated_part_norm(y, z, nw2, 1e-6, yo, 8))
+        us = us_of(lambda: ops.gated_part_norm(y, z, nw2, 1e-6, yo, 1, gate_first=False))
+        entry(f"{what}: norm over all heads, sigmoid gate", us, roof_us(n * H * d * 8), "gated_part_norm (8 parts)", us_like, roof_us(n * H * d * 8))
+        # ---- experts weighted on their input
+        E, top, eff = 8, 2, ff // 4
+        pairs = n * E if decode else n * top
+        gu, act = rn(pairs, 2 * eff).to(bf), torch.empty(pairs, eff, dtype=bf, device=dev)
+        chosen = torch.randint(0, E, (n, top), dtype=torch.int32, device=dev)
+        weight, row_w = torch.rand(n, top, device=dev), torch.rand(pairs, device=dev)
+        us_like = us_of(lambda: ops.glu_act(gu, act, "silu"))
+        us = us_of(lambda: ops.glu_act(gu, act, "silu", **(dict(chosen=chosen, weight=weight) if decode else dict(row_weight=row_w))))
+        entry(f"{what}: experts' activation with the weights on their inputs", us, roof_us(pairs * eff * 6), "glu_act", us_like, roof_us(pairs * eff * 6))
+        expert_rows, x, y2 = rn(pairs, width).to(bf), rn(n, width).to(bf), torch.empty(n, width, dtype=bf, device=dev)
+        pair_row = torch.arange(n * top, dtype=torch.int32, device=dev).view(n, top).contiguous()
+        us_like = us_of(lambda: ops.moe_combine(expert_rows, x, x, pair_row, weight, top, y2))
+        us = us_of(lambda: ops.moe_combine(expert_rows, x, x, pair_row, None, top, y2))
+        roof = roof_us(n * width * 2 * (top + 2))
+        entry(f"{what}: sum of the chosen experts and the shared one", us, roof, "moe_combine (weighted)", us_like, roof)
+    logits = rn(batch, s["vocab"])
+    us_like = us_of(lambda: logits.mul_(1.0))
+    entry("decode: logits capped", us_of(lambda: ops.softcap_(logits, 30.0)), roof_us(logits.numel() * 8), "logits times a number", us_like,
+          roof_us(logits.numel() * 8))
+    return out
+
 def main(args):
     import torch
 
@@ -896,9 +1069,9 @@ def main(args):
     for name in names:
         s = SIZES[name]
         row = {"shape": s}
-        wanted = [a for a in (args.arch_names or "vabelorn,qwen3,lunadra,vemepel,zonevik,bobasun").split(",") if a]
+        wanted = [a for a in (args.arch_names or "vabelorn,qwen3,lunadra,vemepel,zonevik,bobasun,burinex").split(",") if a]
         for arch, make in (("vabelorn", vabelorn_config), ("qwen3", qwen3_config), ("lunadra", lunadra_config),
-                           ("vemepel", vemepel_config), ("zonevik", zonevik_config), ("bobasun", bobasun_config)):
+                           ("vemepel", vemepel_config), ("zonevik", zonevik_config), ("bobasun", bobasun_config), ("burinex", burinex_config)):
             if arch not in wanted:
                 continue
             row[arch] = model_speeds(pe, torch, make(pe, s), prompt, batch, context, args.steps, max(args.warmup, 3))
@@ -922,6 +1095,10 @@ def main(args):
         if "bobasun" in wanted:
             row["bobasun_kernels"] = bobasun_kernel_pairs(pe, torch, s, peaks, prompt, batch, context)
             for k, v in row["bobasun_kernels"].items():
+                print(f"[{name}] {k}: {v}", file=sys.stderr, flush=True)
+        if "burinex" in wanted:
+            row["burinex_kernels"] = burinex_kernel_pairs(pe, torch, s, peaks, prompt, batch, context)
+            for k, v in row["burinex_kernels"].items():
                 print(f"[{name}] {k}: {v}", file=sys.stderr, flush=True)
         result["sizes"][name] = row
     result["gpu_launches"] = pe.kernels.ops.launch_count()

@@ -401,6 +401,87 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const T* q_rows, lo
   }
 }
 
+// The same without folded queries to copy, two features an access (even sizes and strides, rows aligned to two elements): the
+// position, the page and the norm's weights are fetched before the wait, a row's pairs are held in registers between its sum
+// and its store (up to VPT pairs a thread).
+template <typename T> struct Pair;
+template <> struct Pair<float> {
+  typedef float2 Raw;
+  __device__ static float2 get(Raw v) { return v; }
+  __device__ static Raw put(float2 v) { return v; }
+};
+template <> struct Pair<__nv_bfloat16> {
+  typedef __nv_bfloat162 Raw;
+  __device__ static float2 get(Raw v) { return __bfloat1622float2(v); }
+  __device__ static Raw put(float2 v) { return __floats2bfloat162_rn(v.x, v.y); }
+};
+template <typename T, int VPT>
+__global__ void __launch_bounds__(256) latent_prepare_pairs_kernel(const T* q_rows, long long q_ld, const T* low_rows,
+                                                                   long long low_ld, int heads, int d, int dr, int rank,
+                                                                   const float* __restrict__ norm_w, float eps,
+                                                                   const float* __restrict__ cos_t,
+                                                                   const float* __restrict__ sin_t, int rot, int table_rows,
+                                                                   const int* token_seq, const int* token_pos,
+                                                                   const int* seq_slot, const int* page_table,
+                                                                   int table_stride, int num_pages, T* __restrict__ pages,
+                                                                   T* __restrict__ qfull, int write_cache, int* status) {
+  typedef typename Pair<T>::Raw Raw;
+  __shared__ float red[32];
+  const int t = blockIdx.x;
+  const int pos = token_pos[t];
+  const int half = rot / 2, low2 = rank / 2, dr2 = dr / 2, wide = rank + dr;
+  const bool in_table = rot == 0 || (pos >= 0 && pos < table_rows);
+  const long long pr = write_cache ? page_row(t, token_seq, token_pos, seq_slot, page_table, table_stride, num_pages, status) : -1;
+  float2 w[VPT];
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int c = threadIdx.x + k * blockDim.x;
+    w[k] = c < low2 ? reinterpret_cast<const float2*>(norm_w)[c] : make_float2(0.f, 0.f);
+  }
+  pdl_wait_block();
+  pdl_launch_dependents();
+  if (!in_table) {
+    if (threadIdx.x == 0) report(status, kStatusPositionOutOfRange, t, pos, table_rows);
+    return;
+  }
+  const float* cs = cos_t + (size_t)pos * half;
+  const float* sn = sin_t + (size_t)pos * half;
+  auto turned = [&](Raw raw, int m) -> Raw {
+    if (m >= half) return raw;
+    const float2 v = Pair<T>::get(raw);
+    const float c = cs[m], s = sn[m];
+    return Pair<T>::put(make_float2(fmaf(v.x, c, -v.y * s), fmaf(v.y, c, v.x * s)));
+  };
+  const Raw* low = reinterpret_cast<const Raw*>(low_rows + (size_t)t * low_ld);
+  float2 x[VPT];
+  float ss = 0.f;
+  if (write_cache) {
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int c = threadIdx.x + k * blockDim.x;
+      x[k] = c < low2 ? Pair<T>::get(low[c]) : make_float2(0.f, 0.f);
+    }
+  }
+  const T* q = q_rows + (size_t)t * q_ld;
+  for (int i = threadIdx.x; i < heads * dr2; i += blockDim.x) {
+    const int h = i / dr2, m = i - h * dr2;
+    const Raw v = reinterpret_cast<const Raw*>(q + (size_t)h * (d + dr) + d)[m];
+    reinterpret_cast<Raw*>(qfull + ((size_t)t * heads + h) * wide + rank)[m] = turned(v, m);
+  }
+  if (!write_cache) return;
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) ss = fmaf(x[k].x, x[k].x, fmaf(x[k].y, x[k].y, ss));
+  const float inv = rsqrtf(block_sum(ss, red) / (float)rank + eps);
+  if (pr < 0) return;
+  Raw* dst = reinterpret_cast<Raw*>(pages + (size_t)pr * wide);
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int c = threadIdx.x + k * blockDim.x;
+    if (c < low2) dst[c] = Pair<T>::put(make_float2(x[k].x * inv * w[k].x, x[k].y * inv * w[k].y));
+  }
+  for (int m = threadIdx.x; m < dr2; m += blockDim.x) dst[low2 + m] = turned(low[low2 + m], m);
+}
+
 static int flat_blocks(size_t total, int threads) {
   size_t blocks = (total + threads - 1) / threads;
   if (blocks > (size_t)kSMs * 16) blocks = (size_t)kSMs * 16;
@@ -524,6 +605,20 @@ extern "C" int pe_latent_prepare(int dtype, const void* q, long long q_ld, const
   if (n_tokens <= 0) return PE_OK;
   if (heads <= 0 || d <= 0 || dr < 0 || rank <= 0 || rot < 0 || rot > dr || (rot & 1)) return PE_ERR_BAD_ARGUMENT;
   if (rot > 0 && (!cos_t || !sin_t)) return PE_ERR_BAD_ARGUMENT;
+  const size_t two = dtype == PE_F32 ? 8 : 4;
+  const bool pairs = absorbed == nullptr && d % 2 == 0 && dr % 2 == 0 && rank % 2 == 0 && rank <= 2048 && q_ld % 2 == 0 && low_ld % 2 == 0 &&
+                     (uintptr_t)q % two == 0 && (uintptr_t)low % two == 0 && (uintptr_t)pages % two == 0 && (uintptr_t)qfull % two == 0 &&
+                     (uintptr_t)norm_w % 8 == 0;
+  if (pairs) {
+#define PE_PAIRS(V)                                                                                                             \
+  PE_BY_DTYPE(dtype, pe::launch((pe::latent_prepare_pairs_kernel<T, V>), n_tokens, 256, 0, stream, (const T*)q, q_ld, (const T*)low, \
+                                low_ld, heads, d, dr, rank, norm_w, eps, cos_t, sin_t, rot, table_rows, token_seq, token_pos,        \
+                                seq_slot, page_table, table_stride, num_pages, (T*)pages, (T*)qfull, write_cache, status))
+    if (rank <= 512) { PE_PAIRS(1); } else if (rank <= 1024) { PE_PAIRS(2); } else { PE_PAIRS(4); }
+#undef PE_PAIRS
+    PE_LAUNCH_CHECK();
+    return PE_OK;
+  }
   PE_BY_DTYPE(dtype, pe::launch(pe::latent_prepare_kernel<T>, n_tokens, 256, 0, stream, (const T*)q, q_ld, (const T*)low, low_ld,
                                 heads, d, dr, rank, norm_w, eps, cos_t, sin_t, rot, table_rows, token_seq, token_pos, seq_slot,
                                 page_table, table_stride, num_pages, (T*)pages, (T*)qfull, (const T*)absorbed, n_tokens,
