@@ -88,7 +88,7 @@ __device__ __forceinline__ void ssd_stage_rows(float* dst, int dst_ld, int np, c
 // outputs meet in shuffles); more threads a column hide the walk's latencies and fill the state's loads.  NR == 0: the state
 // lives in shared memory, one thread a column.  CONST: the form with a constant decay per head and silu on x, B and C.
 template <typename T, int MODE, int NR, int SPLIT, bool CONST>
-__global__ void __launch_bounds__(NR == 0 ? 1024 : 512) ssd_kernel(SsdArgs a) {
+__global__ void __launch_bounds__(NR == 0 ? 1024 : 512, NR == 32 ? 2 : 1) ssd_kernel(SsdArgs a) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float s_dt[kSsdBatch], s_a[kSsdBatch], s_log[kSsdBatch];
   const int n = a.n, dv = a.dv, head = blockIdx.x, b = blockIdx.y, c = blockIdx.z;
