@@ -109,7 +109,7 @@ __global__ void moe_route_logits_kernel(const float* logits, const float* __rest
 
 // The choice among groups of neighbours: s = sigmoid(z); the outputs form `n_groups` equal groups, a group's score is the sum
 // of its two largest s (its one s for groups of one), only the `keep` best groups (ties: the lower group) may be chosen from;
-// the `top` largest s among those (ties: the lower index), weighted with s itself.  n_groups <= 1: no groups.  One warp per token.
+// the `top` largest s among those (compared by z; ties: the lower index), weighted with s itself.  n_groups <= 1: no groups.  One warp per token.
 __global__ void moe_route_sigmoid_groups_kernel(const float* logits, int n_tokens, int n_all, int top, int n_groups, int keep,
                                                 int* __restrict__ chosen, float* __restrict__ weight, int* __restrict__ dense_rows,
                                                 int n_real) {
@@ -157,7 +157,7 @@ __global__ void moe_route_sigmoid_groups_kernel(const float* logits, int n_token
     for (int e = lane, i = 0; e < n_all; e += 32, ++i) {
       if ((taken_lo >> i) & 1ull) continue;
       if (n_groups > 1 && gs[e / per] != INFINITY) continue;
-      const float c = 1.f / (1.f + expf(-z[e]));
+      const float c = z[e];      // the sigmoid keeps the order; in float32 it is 1 for every large z
       if (c > best || best_e == 0x7fffffff) { best = c; best_e = e; }
     }
 #pragma unroll
@@ -170,7 +170,7 @@ __global__ void moe_route_sigmoid_groups_kernel(const float* logits, int n_token
     if (lane == 0) {
       const bool any = best_e != 0x7fffffff;
       chosen[(size_t)t * top + j] = any ? best_e : -1;
-      weight[(size_t)t * top + j] = any ? best : 0.f;
+      weight[(size_t)t * top + j] = any ? 1.f / (1.f + expf(-best)) : 0.f;
       if (dense_rows) dense_rows[(size_t)t * top + j] = (any && best_e < n_real) ? t * n_real + best_e : -1;
     }
   }

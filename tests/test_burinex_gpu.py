@@ -421,6 +421,19 @@ def test_experts_weighted_on_their_input(pe, dtype, n, E, top, H, ff):
     assert rel_err(other.double().cpu(), want) > 5e-2
 
 
+def test_the_largest_score_is_chosen_where_the_sigmoid_is_one_or_nothing_in_float32(ops):
+    """Logits so large (or so far below zero) that float32 cannot tell their sigmoids apart, and ordinary ones."""
+    for base in (25.0, 0.0, -120.0):
+        logits = base + torch.tensor([[0.0, 0.002, -0.5, 0.001, 0.5, 0.499]]).repeat(3, 1)
+        logits[1, 0], logits[2, 3] = base + 0.75, base + 0.75
+        chosen = torch.empty(3, 2, dtype=torch.int32, device=DEV)
+        weight = torch.empty(3, 2, device=DEV)
+        ops.moe_route_sigmoid_groups(logits.to(DEV), 2, 1, 1, chosen, weight)
+        assert chosen.tolist() == [[4, 5], [0, 4], [3, 4]]
+        want = torch.sigmoid(logits.double().gather(1, chosen.cpu().long()))
+        assert (weight.double().cpu() - want).abs().max() < 1e-6
+
+
 def _latent_attend(ops, kernel, decode, q, lens, q_lens, nh, row, r, scale, pg, window, sinks, even=True):
     """The step's output rows ``[n, nh * r]`` and the split results of both ways to cut a decode into ranges."""
     n, dtype = sum(q_lens), pg.pages.dtype

@@ -71,7 +71,7 @@ def test_a_configuration_drawn_at_random(pe, seed, dtype):
         if dtype == "float32":
             assert rel_err(got, ref) < 3e-5, (seed, what, cfg)
         else:                     # the median: a rounding may pick another expert here and there
-            limit = 3.0 * max(float(noise.median()), float(noise_long.median()))
+            limit = 4.0 * max(float(noise.median()), float(noise_long.median()))
             assert float((got - ref).pow(2).mean(1).sqrt().median()) < limit, (seed, what, cfg)
 
     s = eng.alloc_slot()
